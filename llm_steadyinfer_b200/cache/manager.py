@@ -1,13 +1,13 @@
 """Cache manager: which pages and which state slot each live request holds.
 
-Layers whose mixers need the same kind of cache (same heads, head size and window) form a
+Layers whose mixers need the same kind of cache (same heads, head size and window or chunk) form a
 *group*; a group has its own page pool and one block table per request, shared by the
 group's layers (the reference has one uniform pool, src/source/scheduler/kv_manager.cpp:41-53).
 Pages are taken when a request grows, given back when it ends, when it is cut back for
-preemption, and, in a windowed group, as soon as the window has passed them. Every request
+preemption, and, in a group with a window or chunks, as soon as no layer that reads them looks back so far. Every request
 also holds one state slot, the index at which mixers with fixed-size state keep theirs.
 
-Prefix reuse (single group without window, no fixed-size state): whole pages are keyed by a
+Prefix reuse (single group without window or chunk, no fixed-size state): whole pages are keyed by a
 hash chained over all tokens before and in them, so equal content at another place or after
 another prefix never matches; the reference hashes a block's own 16 tokens only
 (src/source/scheduler/prefix_cache.cpp:8-18).
@@ -23,7 +23,7 @@ import struct
 from dataclasses import dataclass, field
 from typing import Dict, Hashable, List, Optional, Sequence, Tuple
 
-from ..parts.base import CacheNeed, StateNeed
+from ..parts.base import CacheNeed, StateNeed, first_visible_key
 from .pages import PageError, PagePool, SlotPool
 
 
@@ -40,11 +40,18 @@ class CacheGroup:
     need: CacheNeed
     layers: List[int]                      # layers that own cache in this group, in storage order
     pool: PagePool
+    # the (window, chunk) of every layer that reads the group's pages; empty: some layer reads all of them
+    reach: Tuple[Tuple[Optional[int], Optional[int]], ...] = ()
     tables: Dict[Hashable, List[int]] = field(default_factory=dict)   # request -> page per block, -1 = given back
 
     @property
-    def window(self) -> Optional[int]:
-        return self.need.window
+    def bounded(self) -> bool:
+        """Pages that no later token can read are given back while the request lives."""
+        return bool(self.reach)
+
+    def first_needed(self, length: int) -> int:
+        """The first position whose keys some layer reads once ``length`` tokens are held."""
+        return min((first_visible_key(length, w, c) for w, c in self.reach), default=0)
 
 
 @dataclass
@@ -56,7 +63,8 @@ class RequestCache:
 
 class CacheLayout:
     """Groups the places of the run order ("layers" below) by their cache need.
-    ``cache_from[i]`` names the place whose cache place i reads instead of owning one."""
+    ``cache_from[i]`` names the place whose cache place i reads instead of owning one. How far back the tokens of a
+    place's cache are kept follows from all places that read it, each with its own window or chunk."""
 
     def __init__(self, needs: Sequence[Optional[CacheNeed]], states: Sequence[Optional[StateNeed]],
                  cache_from: Optional[Sequence[Optional[int]]] = None):
@@ -69,17 +77,7 @@ class CacheLayout:
         self.group_layers: List[List[int]] = []
         self.layer_group: List[Optional[int]] = [None] * n
         self.layer_index_in_group: List[Optional[int]] = [None] * n
-        for i, need in enumerate(needs):
-            if cache_from[i] is not None or need is None:
-                continue
-            key = need.group_key()
-            if key not in self.group_keys:
-                self.group_keys.append(key)
-                self.group_layers.append([])
-            g = self.group_keys.index(key)
-            self.layer_group[i] = g
-            self.layer_index_in_group[i] = len(self.group_layers[g])
-            self.group_layers[g].append(i)
+        self.group_reach: List[Tuple] = []
         for i, src in enumerate(cache_from):
             if src is None:
                 continue
@@ -87,9 +85,23 @@ class CacheLayout:
                 raise ValueError(f"layer {i} reads the cache of layer {src}, which owns none")
             if needs[i] is None or needs[i].layout_key() != needs[src].layout_key():
                 raise ValueError(f"layer {i} cannot read layer {src}'s cache: their head layouts differ")
-            sw, rw = needs[src].window, needs[i].window
-            if sw is not None and (rw is None or rw > sw):
-                raise ValueError(f"layer {i} would read further back than layer {src}'s window of {sw} keeps")
+        for i, need in enumerate(needs):
+            if cache_from[i] is not None or need is None:
+                continue
+            reach = {need.reach} | {needs[j].reach for j in range(n) if cache_from[j] == i}
+            reach = () if (None, None) in reach else tuple(sorted(reach, key=lambda r: (r[0] or 0, r[1] or 0)))
+            key = need.layout_key() + (reach,)
+            if key not in self.group_keys:
+                self.group_keys.append(key)
+                self.group_layers.append([])
+                self.group_reach.append(reach)
+            g = self.group_keys.index(key)
+            self.layer_group[i] = g
+            self.layer_index_in_group[i] = len(self.group_layers[g])
+            self.group_layers[g].append(i)
+        for i, src in enumerate(cache_from):
+            if src is None:
+                continue
             self.layer_group[i] = self.layer_group[src]
             self.layer_index_in_group[i] = self.layer_index_in_group[src]
 
@@ -108,13 +120,13 @@ class CacheManager:
             raise ValueError(f"page_size must be positive, got {page_size}")
         self.layout = layout
         self.page_size = int(page_size)
-        self.groups = [CacheGroup(layout.group_need(g), layout.group_layers[g], PagePool(num_pages))
+        self.groups = [CacheGroup(layout.group_need(g), layout.group_layers[g], PagePool(num_pages), layout.group_reach[g])
                        for g in range(layout.num_groups)]
         self.slots = SlotPool(max_requests)
         self.requests: Dict[Hashable, RequestCache] = {}
         has_state = any(s is not None for s in layout.states)
         self.prefix_reuse = bool(prefix_reuse) and len(self.groups) == 1 \
-            and self.groups[0].window is None and not has_state
+            and not self.groups[0].bounded and not has_state
         self._hash_to_page: Dict[bytes, int] = {}
         self._page_to_hash: Dict[int, bytes] = {}
         if self.prefix_reuse:
@@ -196,15 +208,14 @@ class CacheManager:
                 self.versions[req] = next(self._version)
 
     def commit(self, req, new_length: int) -> None:
-        """The request now holds ``new_length`` tokens; windowed groups give back the pages
-        that no later position can read."""
+        """The request now holds ``new_length`` tokens; groups of layers with a window or chunks give back the
+        pages that no later position can read."""
         rc = self.requests[req]
         rc.length = new_length
         for g in self.groups:
-            if g.window is None:
+            if not g.bounded:
                 continue
-            first_needed = new_length - g.window + 1      # the next token reads keys from here on
-            dead = max(0, first_needed) // self.page_size
+            dead = g.first_needed(new_length) // self.page_size      # the next token reads keys from there on
             t = g.tables[req]
             for b in range(min(dead, len(t))):
                 if t[b] >= 0:
@@ -215,7 +226,7 @@ class CacheManager:
     def can_truncate_to(self, keep_length: int) -> int:
         """Preemption keeps a whole number of pages; with windows or fixed-size state nothing
         can be kept, since what the kept part would need is gone or cannot be cut."""
-        if any(g.window is not None for g in self.groups) or any(s is not None for s in self.layout.states):
+        if any(g.bounded for g in self.groups) or any(s is not None for s in self.layout.states):
             return 0
         return (keep_length // self.page_size) * self.page_size
 

@@ -69,6 +69,9 @@ class LayerSpec:
     passes a learned gate: ``h += residual_scale * (sigmoid(W1 x1 + b1) * mixer(x1) + sigmoid(W2 x2 + b2) * ffn(x2))``,
     ``x1 = norm1(h)``, ``x2 = norm2(h)`` (``mixer_gate_name``, ``feed_forward_gate_name``).
 
+    With arrangement "streams" the residual stream has ``ModelSpec.streams`` copies and each sublayer has connections to
+    them (``mixer_streams_prefix``, ``feed_forward_streams_prefix``; see ``StreamConnections``).
+
     ``weight_prefix`` is the checkpoint prefix of this layer ("model.layers.3.").
     ``cache_from`` is None when the layer owns its cache, or the index of the layer
     whose cache it reads (it then writes nothing): that of the latest run of that layer
@@ -95,6 +98,9 @@ class LayerSpec:
     # matrices [hidden, hidden]; their biases are ``<name>.b``
     mixer_gate_name: Optional[str] = None
     feed_forward_gate_name: Optional[str] = None
+    # connections to a stream of several copies (arrangement "streams"): tensor prefixes below weight_prefix
+    mixer_streams_prefix: Optional[str] = None
+    feed_forward_streams_prefix: Optional[str] = None
     residual_scale: float = 1.0                  # what a block adds to the stream is multiplied by it
 
 
@@ -125,6 +131,8 @@ class ModelSpec:
     embedder: Optional[EmbedderSpec] = None      # None: the plain table under ``embed_name``
     stream_adds: tuple = ()                      # StreamAddSpec entries, at most one a place
     stream_vector_shapes: Optional[Dict[str, tuple]] = None   # the tensors that ``stream_adds`` name: name -> shape
+    streams: Optional[int] = None                # copies of the residual stream (arrangement "streams"); None: the one stream
+    logit_scale: float = 1.0                     # logits are multiplied by it (before the soft cap)
     logit_softcap: float = 0.0                   # > 0: logits <- cap * tanh(logits / cap)
 
 

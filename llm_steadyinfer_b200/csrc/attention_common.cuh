@@ -6,6 +6,8 @@
 
 typedef __nv_bfloat16 bf16;
 
+#define LOG2E 1.4426950408889634f      // scores and their maxima are kept in base 2
+
 struct AttnItem { int seq, row0, ntok, pos0; };
 
 // The split decode kernels keep one ticket per (item, kv head) at the START of their scratch, in a
@@ -20,6 +22,12 @@ struct AttnItem { int seq, row0, ntok, pos0; };
 __device__ __forceinline__ int window_first_key(int pos0, int window) {
   return window > 0 && pos0 - window + 1 > 0 ? pos0 - window + 1 : 0;
 }
+// The same with chunks: positions fall into runs of `chunk`, counted from position 0, and a row sees the keys of its
+// own run alone (0: no chunks). It never falls as the position grows, so an item's first row decides for the item.
+__device__ __forceinline__ int first_visible_key(int pos, int window, int chunk) {
+  const int lo = window_first_key(pos, window);
+  return chunk > 0 ? max(lo, pos / chunk * chunk) : lo;
+}
 
 struct AttnParams {
   const bf16* q; long long q_stride;
@@ -33,6 +41,8 @@ struct AttnParams {
   int num_pages, page_size, num_seqs, H, KV, G, hs;
   float scale_log2;         // scale * log2(e)
   int window, nsplit;
+  int chunk;                // rows see keys of their own run of `chunk` positions (0: none); the mma.sync kernels take none
+  const float* sink;        // fp32 [H]: exp(sink[h]) joins the denominator once (nullptr: none); likewise
   int* status;
 };
 

@@ -2,7 +2,7 @@
 // softmax) in the general form of attention_general.cu: key size dk and value size dv of any multiple of 8,
 // values of their own or the first dv entries of the keys (a latent that is key and value), a bias by distance
 // added to the scaled score, an output gate (the result times sigmoid of a row of gate sums), a penalty slope[h] * (i - j) taken off it, a query temperature by position (row i's scale
-// times 1 + coef * ln(floor((i + 1) / every) + 1)), a sink per head in the denominator, a soft limit on the scaled score
+// times 1 + coef * ln(floor((i + 1) / every) + 1)), a window or chunks, a sink per head in the denominator, a soft limit on the scaled score
 // (s <- cap * tanh(s / cap)), key heads that share a value head (v_share neighbouring key heads read one of the
 // KV / v_share value heads), results in fp32 where the caller goes on computing with them. One kernel serves prompt
 // portions and decode rows; for decode the key range of an item can be split over blocks, whose fp32 partial results a second small
@@ -39,12 +39,11 @@ struct FlexParams {
   int warps_are_slices;     // items of at most 16 rows whose values are key columns: every warp takes rows 0..15 and a
                             // value slice of its own, so that a block serves four slices from one key tile
   float scale_log2;         // scale * log2(e)
-  int window, nsplit;
+  int window, chunk, nsplit;
   int* status;
 };
 
 #define FLEX_M 64
-#define LOG2E 1.4426950408889634f
 
 __device__ __forceinline__ bf16* ftile(bf16* base, int pitch_chunks, int row, int chunk) {
   return base + ((size_t)row * pitch_chunks + (chunk ^ (row & 7))) * 8;
@@ -84,7 +83,7 @@ attn_flex_kernel(const FlexParams p) {
   }
   const int* table = p.block_table + (size_t)item.seq * p.table_width;
   const int kv_end_all = item.pos0 + item.ntok;
-  const int kv_lo = window_first_key(item.pos0, p.window);
+  const int kv_lo = first_visible_key(item.pos0, p.window, p.chunk);
   const int kv_begin_all = kv_lo / BLOCK_N * BLOCK_N;
   const int tiles_all = (kv_end_all - kv_begin_all + BLOCK_N - 1) / BLOCK_N;
   const int tiles_per = (tiles_all + p.nsplit - 1) / p.nsplit;
@@ -169,6 +168,7 @@ attn_flex_kernel(const FlexParams p) {
   const int tok_lo = r_lo / p.Gb, tok_hi = r_hi / p.Gb;
   const int pos_lo = tok_lo < item.ntok ? item.pos0 + tok_lo : -1;     // -1: row unused
   const int pos_hi = tok_hi < item.ntok ? item.pos0 + tok_hi : -1;
+  const int first_lo = first_visible_key(pos_lo, p.window, p.chunk), first_hi = first_visible_key(pos_hi, p.window, p.chunk);
   const int hh_lo = r_lo % p.Gb, hh_hi = r_hi % p.Gb;
   const int head_lo = head0 + hh_lo, head_hi = head0 + hh_hi;
   // what a row's raw score is multiplied by beside the scale (its query temperature), and its head's slope (base 2)
@@ -179,7 +179,7 @@ attn_flex_kernel(const FlexParams p) {
   const int warp_first_tok = wrow / p.Gb;
   const bool warp_active = warp_first_tok < item.ntok && v0 < p.dv;
   const int warp_max_pos = item.pos0 + warp_last_tok;
-  const int warp_min_pos = item.pos0 + warp_first_tok;
+  const int warp_first_key = first_visible_key(item.pos0 + warp_first_tok, p.window, p.chunk);
 
   float o[DT][4];
 #pragma unroll
@@ -198,7 +198,7 @@ attn_flex_kernel(const FlexParams p) {
     }
     __syncthreads();
     bool skip = !warp_active || j0 + krow0 > warp_max_pos;
-    if (p.window > 0 && j0 + krow0 + KEYS_W - 1 <= warp_min_pos - p.window) skip = true;
+    if (j0 + krow0 + KEYS_W - 1 < warp_first_key) skip = true;
     if (!skip) {
       float s[NT][4];
 #pragma unroll
@@ -224,7 +224,7 @@ attn_flex_kernel(const FlexParams p) {
         for (int e = 0; e < 4; ++e) {
           const int j = j0 + krow0 + nt * 8 + (lane & 3) * 2 + (e & 1);
           const int pos = (e < 2) ? pos_lo : pos_hi;
-          const bool vis = j >= kv_lo && j <= pos && (p.window <= 0 || j > pos - p.window);
+          const bool vis = j >= ((e < 2) ? first_lo : first_hi) && j <= pos;
           float v = -INFINITY;
           if (vis) {
             // tanh(y) = 1 - 2 / (exp(2 y) + 1): absolute error of some 1e-7, which is what counts for a score
@@ -458,12 +458,12 @@ SI_EXPORT int si_attn_flex(const void* q, long long q_stride, const void* k_cach
                            const int* block_table, int table_width, const int* items, int num_items, void* out,
                            long long out_stride, int num_pages, int page_size, int num_seqs, int H, int KV, int dk,
                            int dv, float scale, int window, const float* dist_bias, int nd, const float* sink,
-                           int nsplit, float* scratch, int max_rows, float softcap, int v_share, int out_is_f32,
+                           int nsplit, float* scratch, int max_rows, float softcap, int v_share, int out_is_f32, int chunk,
                            const float* slopes, float qt_coef, int qt_every, const void* gate, long long gate_stride,
                            int* status, cudaStream_t stream) {
   if (num_items <= 0) return 0;
   if (!si_attn_flex_ok(H, KV, dk, dv, v_cache != nullptr) || nsplit < 1 || nsplit > 64 || (nsplit > 1 && !scratch)) return -2;
-  if (v_share < 1 || KV % v_share || (v_share > 1 && !v_cache) || softcap < 0.f || qt_every < 0) return -2;
+  if (v_share < 1 || KV % v_share || (v_share > 1 && !v_cache) || softcap < 0.f || qt_every < 0 || chunk < 0) return -2;
   FlexParams p;
   p.slopes = slopes; p.qt_coef = qt_coef; p.qt_every = qt_every;
   p.gate = (const bf16*)gate; p.gate_stride = gate_stride;
@@ -480,7 +480,7 @@ SI_EXPORT int si_attn_flex(const void* q, long long q_stride, const void* k_cach
   p.num_pages = num_pages; p.page_size = page_size; p.num_seqs = num_seqs;
   p.H = H; p.KV = KV; p.G = H / KV; p.Gb = flex_heads_per_block(p.G); p.hparts = p.G / p.Gb;
   p.dk = dk; p.dv = dv; p.dk_pitch = (dk + 63) / 64 * 64;
-  p.scale_log2 = scale * LOG2E; p.window = window; p.nsplit = nsplit; p.status = status;
+  p.scale_log2 = scale * LOG2E; p.window = window; p.chunk = chunk; p.nsplit = nsplit; p.status = status;
   const long long slabs = (long long)num_items * KV * p.hparts * nsplit;
   p.part_o = scratch;
   p.part_ml = scratch ? scratch + slabs * FLEX_M * dv : nullptr;

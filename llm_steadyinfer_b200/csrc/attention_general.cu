@@ -5,6 +5,7 @@
 //   * values that are the first dv entries of the keys (v_cache == nullptr: a latent that serves as both),
 //   * a bias by distance: bias[min(i - j, nd - 1), head] (fp32 table [nd, H]) added to the scaled score,
 //   * a sink per head: exp(sink[h]) joins the softmax denominator once, with no key and no value,
+//   * chunks: positions in runs of `chunk` from position 0 on, a query sees keys of its own run,
 //   * a penalty in proportion to the distance: slope[h] * (i - j) taken off the scaled score (fp32 [H]),
 //   * a query temperature by position: the scale of row i is multiplied by 1 + coef * ln(floor((i + 1) / every) + 1),
 //   * an output gate: the result's entry (row, head, d) is multiplied by sigmoid(gate[row, head * dv + d]),
@@ -12,7 +13,7 @@
 //   * key heads that share a value head: `v_share` neighbouring key heads read one value head (the cache then holds
 //     KV / v_share value heads), as the maps of a differential attention do,
 //   * results in fp32 whatever the storage (out_f32), for a caller that goes on subtracting them.
-//     s_j = scale * q_h . K[j, g] + bias[min(pos - j, nd - 1), h],  j in [max(0, pos - window + 1), pos]
+//     s_j = scale * q_h . K[j, g] + bias[min(pos - j, nd - 1), h],  j in [max(0, pos - window + 1, chunk * floor(pos / chunk)), pos]
 //     out_h = sum_j exp(s_j) V[j, g] / (sum_j exp(s_j) + exp(sink_h))
 // One block per (token row, query head); warp w of 4 walks keys j0 + w, j0 + w + 4, ... with a running
 // maximum, the four partial results are merged at the end, so the order of a row's sums depends on its
@@ -34,7 +35,7 @@ attention_general_kernel(const T* __restrict__ q, long long q_row_stride,
                          const int* __restrict__ row_seq, const int* __restrict__ positions,
                          TO* __restrict__ out, long long out_row_stride, int num_pages,
                          int page_size, int num_seqs, int H, int KV, int dk, int dv, float scale,
-                         int window, const float* __restrict__ dist_bias, int nd,
+                         int window, int chunk, const float* __restrict__ dist_bias, int nd,
                          const float* __restrict__ sink, float softcap, int v_share,
                          const float* __restrict__ slopes, float qt_coef, int qt_every,
                          const T* __restrict__ gate, long long gate_row_stride, int* status) {
@@ -65,7 +66,8 @@ attention_general_kernel(const T* __restrict__ q, long long q_row_stride,
   float m = -INFINITY, l = 0.f;
   if (qt_every > 0) scale *= 1.f + qt_coef * logf((float)((pos + 1) / qt_every + 1));
   const float slope = slopes ? slopes[h] : 0.f;
-  const int j0 = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  int j0 = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  if (chunk > 0) j0 = max(j0, pos / chunk * chunk);
   for (int j = j0 + warp; j <= pos; j += GEN_WARPS) {
     const int slot = j / page_size;
     const int page = slot < table_width ? table[slot] : -1;
@@ -133,20 +135,20 @@ SI_EXPORT int si_attention_general(const void* q, int dtype, long long q_row_str
                                    long long out_row_stride, int num_pages, int page_size, int num_tokens,
                                    int num_seqs, int H, int KV, int dk, int dv, float scale, int window,
                                    const float* dist_bias, int nd, const float* sink, float softcap, int v_share,
-                                   int out_f32, const float* slopes, float qt_coef, int qt_every, const void* gate,
+                                   int out_f32, int chunk, const float* slopes, float qt_coef, int qt_every, const void* gate,
                                    long long gate_row_stride, int* status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (dk > 32 * GEN_WIDE_PER_LANE || dv > 32 * GEN_WIDE_PER_LANE || dk <= 0 || dv <= 0 || KV <= 0 || H % KV) return -2;
   if (!v_cache && dv > dk) return -2;
   if (v_share < 1 || KV % v_share || (v_share > 1 && !v_cache)) return -2;
   if (dist_bias && nd <= 0) return -2;
-  if (qt_every < 0) return -2;
+  if (qt_every < 0 || chunk < 0) return -2;
   dim3 grid(num_tokens, H);
   const size_t smem = (size_t)(GEN_WARPS * dv + 2 * GEN_WARPS) * sizeof(float);
 #define GEN_LAUNCH(T, TO, PL)                                                                                          \
   attention_general_kernel<T, TO, PL><<<grid, GEN_WARPS * 32, smem, stream>>>(                                         \
       (const T*)q, q_row_stride, (const T*)k_cache, (const T*)v_cache, block_table, table_width, row_seq, positions,   \
-      (TO*)out, out_row_stride, num_pages, page_size, num_seqs, H, KV, dk, dv, scale, window, dist_bias, nd, sink,     \
+      (TO*)out, out_row_stride, num_pages, page_size, num_seqs, H, KV, dk, dv, scale, window, chunk, dist_bias, nd, sink, \
       softcap, v_share, slopes, qt_coef, qt_every, (const T*)gate, gate_row_stride, status)
   if (dk > 32 * GEN_MAX_PER_LANE || dv > 32 * GEN_MAX_PER_LANE) {        // sizes above 640: the kernel with more entries a lane
     if (dtype == SI_BF16 && out_f32) GEN_LAUNCH(__nv_bfloat16, float, GEN_WIDE_PER_LANE);

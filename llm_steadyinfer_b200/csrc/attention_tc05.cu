@@ -104,7 +104,7 @@ attn_portion_tc05_kernel(const AttnParams p, const __grid_constant__ CUtensorMap
   const int tile_tokens = BM / p.G;                  // tokens of one query tile
   const bool two = item.ntok > tile_tokens;          // the second query tile has rows
   const int kv_end = item.pos0 + item.ntok;
-  const int kv_lo = window_first_key(item.pos0, p.window);
+  const int kv_lo = first_visible_key(item.pos0, p.window, p.chunk);
   const int kv_begin = kv_lo / BN * BN;
   const int ntiles = (kv_end - kv_begin + BN - 1) / BN;
   const int page_rows = 1 << log2_page;
@@ -298,7 +298,8 @@ attn_portion_tc05_kernel(const AttnParams p, const __grid_constant__ CUtensorMap
     const int tok = q * tile_tokens + tl;
     const bool valid = tl < tile_tokens && tok < item.ntok;
     const int pos = valid ? item.pos0 + tok : -1;
-    const int lo = p.window > 0 ? pos - p.window + 1 : INT_MIN;     // visible keys: lo <= j <= pos
+    int lo = p.window > 0 ? pos - p.window + 1 : INT_MIN;           // visible keys: lo <= j <= pos
+    if (p.chunk > 0) lo = max(lo, pos / p.chunk * p.chunk);
     const unsigned lane_base = (unsigned)((warp & 3) * 32) << 16;
     const unsigned ts = tmem + lane_base + TM_S + q * BN, to = tmem + lane_base + TM_O + q * HS;
     float m = -INFINITY, l = 0.f;                    // base of the exponentials (log2 domain), the row's sum
@@ -424,7 +425,11 @@ attn_portion_tc05_kernel(const AttnParams p, const __grid_constant__ CUtensorMap
     if (!alive && lane == 0) { set_status(p.status, SI_WAIT_LIMIT); s_abort = 1; }
     if (alive) {
       tc05_fence_after_sync();
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.sink) {                                          // exp(sink) joins the denominator once
+        const float s2 = p.sink[g * p.G + (hh < p.G ? hh : 0)] * LOG2E, M = fmaxf(m, s2), f = fast_exp2(m - M);
+        inv = f / (l * f + fast_exp2(s2 - M));
+      }
       bf16* dst = p.out + (size_t)(item.row0 + tok) * p.out_stride + (size_t)(g * p.G + hh) * p.hs;
 #pragma unroll
       for (int c = 0; c < HS / 64; ++c) {
@@ -501,9 +506,9 @@ SI_EXPORT int si_attn_portion_tc05(const void* q, long long q_stride, const void
                                    const void* items, int num_items, void* out, long long out_stride, int num_pages,
                                    int page_size, int num_seqs, int H, int KV, int hs, float scale, int window,
                                    const float* slopes, float qt_coef, int qt_every, const void* gate, long long gate_stride,
-                                   int* status, cudaStream_t stream) {
+                                   int chunk, const float* sink, int* status, cudaStream_t stream) {
   if (num_items <= 0) return 0;
-  if (qt_every < 0 || (gate && (gate_stride % 8 || ((uintptr_t)gate % 16)))) return -2;
+  if (qt_every < 0 || chunk < 0 || (gate && (gate_stride % 8 || ((uintptr_t)gate % 16)))) return -2;
   // a temperature below zero would turn the order of the scores round: the plain kernels serve that
   const AttnExtras x{slopes, qt_coef, qt_every, (const bf16*)gate, gate_stride};
   const bool ext = slopes || qt_every > 0 || gate;
@@ -520,7 +525,7 @@ SI_EXPORT int si_attn_portion_tc05(const void* q, long long q_stride, const void
   p.num_pages = num_pages; p.page_size = page_size; p.num_seqs = num_seqs;
   p.H = H; p.KV = KV; p.G = H / KV; p.hs = hs;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = window; p.nsplit = 1; p.status = status;
+  p.window = window; p.chunk = chunk; p.sink = sink; p.nsplit = 1; p.status = status;
   int log2_page = 0;
   while ((1 << log2_page) < page_size) ++log2_page;
   const CUtensorMap& km = *(const CUtensorMap*)kmap;

@@ -79,7 +79,7 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
   }
   const int* table = p.block_table + (size_t)item.seq * p.table_width;
   const int kv_end_all = item.pos0 + item.ntok;
-  const int kv_lo = window_first_key(item.pos0, p.window);
+  const int kv_lo = first_visible_key(item.pos0, p.window, p.chunk);
   const int kv_begin_all = kv_lo / BLOCK_N * BLOCK_N;
   const int tiles_all = (kv_end_all - kv_begin_all + BLOCK_N - 1) / BLOCK_N;
   const int tiles_per = (tiles_all + nsplit - 1) / nsplit;
@@ -172,7 +172,7 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
 #pragma unroll
     for (int i = 0; i < DT; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
   }
-  int pos_of[MT][2];
+  int pos_of[MT][2], first_of[MT][2];                // last and first key a row sees
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -180,11 +180,12 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
       const int r = mt * 16 + (lane >> 2) + 8 * h2;
       const int tok = r / p.G;
       pos_of[mt][h2] = tok < item.ntok ? item.pos0 + tok : -1;
+      first_of[mt][h2] = first_visible_key(pos_of[mt][h2], p.window, p.chunk);
     }
 
   // The query fragments do not change from tile to tile: they are read from shared memory once.
   unsigned qf[MT][KT][4];
-  int pos_min = 0x7fffffff, pos_max = -1;            // over the rows of this lane's fragments
+  int pos_min = 0x7fffffff, first_max = 0;           // over the rows of this lane's fragments
   if constexpr (SWAP) {
     // lane (g, t): B fragment of Q^T, row g, head-dim elements 16kk + 2t, +1 and 16kk + 8 + 2t, +1;
     // the lane's elements of S^T belong to rows 2t and 2t + 1
@@ -199,7 +200,8 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
       for (int i = 0; i < 2; ++i) {
         const int tok = (2 * (lane & 3) + i) / p.G;
         pos_of[0][i] = tok < item.ntok ? item.pos0 + tok : -1;
-        if (pos_of[0][i] >= 0) { pos_min = min(pos_min, pos_of[0][i]); pos_max = max(pos_max, pos_of[0][i]); }
+        first_of[0][i] = first_visible_key(pos_of[0][i], p.window, p.chunk);
+        if (pos_of[0][i] >= 0) { pos_min = min(pos_min, pos_of[0][i]); first_max = max(first_max, first_of[0][i]); }
       }
     }
   } else if (warp < NWARPS) {
@@ -213,7 +215,7 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
       for (int h2 = 0; h2 < 2; ++h2)
-        if (pos_of[mt][h2] >= 0) { pos_min = min(pos_min, pos_of[mt][h2]); pos_max = max(pos_max, pos_of[mt][h2]); }   // rows without a token decide nothing
+        if (pos_of[mt][h2] >= 0) { pos_min = min(pos_min, pos_of[mt][h2]); first_max = max(first_max, first_of[mt][h2]); }   // rows without a token decide nothing
   }
 
   for (int t = 0; warp < NWARPS && t < ntiles; ++t) {
@@ -229,7 +231,7 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
     const int jw = j0 + warp * 16;          // this warp's 16 keys
     if (jw < kv_end) {
       // most tiles lie wholly inside every row's visible range: then nothing is masked
-      const bool masked = __any_sync(0xffffffffu, jw + 15 > pos_min || (p.window > 0 && jw <= pos_max - p.window));
+      const bool masked = __any_sync(0xffffffffu, jw + 15 > pos_min || jw < first_max);
       if constexpr (SWAP) {
         // S^T[16 keys, 8 rows]: the lane holds keys g, g + 8 (elements 0-1, 2-3) of rows 2t, 2t + 1
         float st[4] = {0.f, 0.f, 0.f, 0.f};
@@ -243,8 +245,7 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int j = jw + (lane >> 2) + 8 * (e >> 1);
-            const int pos = pos_of[0][e & 1];
-            if (!(j <= pos && (p.window <= 0 || j > pos - p.window))) st[e] = -INFINITY;
+            if (j > pos_of[0][e & 1] || j < first_of[0][e & 1]) st[e] = -INFINITY;
           }
         }
         float mx[2] = {m[0][0], m[0][1]}, corr[2], base[2];
@@ -294,9 +295,7 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const int j = jw + nt * 8 + (lane & 3) * 2 + (e & 1);
-              const int pos = pos_of[mt][e >> 1];
-              const bool vis = j <= pos && (p.window <= 0 || j > pos - p.window);
-              if (!vis) s[nt][e] = -INFINITY;
+              if (j > pos_of[mt][e >> 1] || j < first_of[mt][e >> 1]) s[nt][e] = -INFINITY;
             }
         }
 #pragma unroll
@@ -407,6 +406,11 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
     }
     if (nsplit == 1) {
       const int tok = r / p.G, hh = r - tok * p.G;
+      if (p.sink) {                          // exp(sink) joins the denominator once
+        const float s2 = p.sink[g * p.G + hh] * LOG2E, Ms = fmaxf(M, s2), f = exp2f(M - Ms);
+        L = L * f + exp2f(s2 - Ms);
+        acc *= f;
+      }
       p.out[(size_t)(item.row0 + tok) * p.out_stride + (size_t)(g * p.G + hh) * p.hs + d] =
           __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
     } else {
@@ -442,9 +446,10 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
   }
   asm volatile("bar.sync 1, 128;\n" ::: "memory");
   for (int r = threadIdx.x; r < rows_used; r += THREADS) {
-    float M = -INFINITY;
+    const float s2 = p.sink ? p.sink[g * p.G + r % p.G] * LOG2E : -INFINITY;
+    float M = s2;
     for (int sp = 0; sp < nsplit; ++sp) M = fmaxf(M, w_s[r * nsplit + sp]);
-    float L = 0.f;
+    float L = p.sink ? exp2f(s2 - M) : 0.f;
     for (int sp = 0; sp < nsplit; ++sp) {
       const float ms = w_s[r * nsplit + sp];
       const float wgt = ms == -INFINITY ? 0.f : exp2f(ms - M);
@@ -557,14 +562,14 @@ SI_EXPORT int si_attn_decode_tma(const void* q, long long q_stride, const void* 
                                  const void* items, int num_items, void* out, long long out_stride, int num_pages,
                                  int page_size, int num_seqs, int H, int KV, int hs, float scale, int window,
                                  int nsplit, const int* work, int num_work, int work_slots, float* scratch,
-                                 int max_rows, int* status, cudaStream_t stream) {
+                                 int max_rows, int chunk, const float* sink, int* status, cudaStream_t stream) {
   if (num_items <= 0) return 0;
   if (!si_attn_decode_tma_ok(H, KV, hs, page_size) || !kmap || !vmap) return -2;
   if (work) {
     if (num_work <= 0 || work_slots <= 0 || !scratch || ((uintptr_t)work % 16)) return -2;
     nsplit = 1;
   }
-  if ((q_stride % 8) || nsplit < 1 || nsplit > 128) return -2;     // the merge stages 2 * rows * nsplit floats in shared memory
+  if ((q_stride % 8) || nsplit < 1 || nsplit > 128 || chunk < 0) return -2;     // the merge stages 2 * rows * nsplit floats in shared memory
   AttnParams p;
   p.q = (const bf16*)q; p.q_stride = q_stride;
   p.k_cache = (const bf16*)k_cache; p.v_cache = (const bf16*)v_cache;
@@ -575,7 +580,7 @@ SI_EXPORT int si_attn_decode_tma(const void* q, long long q_stride, const void* 
   p.num_pages = num_pages; p.page_size = page_size; p.num_seqs = num_seqs;
   p.H = H; p.KV = KV; p.G = H / KV; p.hs = hs;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = window; p.nsplit = nsplit; p.status = status;
+  p.window = window; p.chunk = chunk; p.sink = sink; p.nsplit = nsplit; p.status = status;
   const int rows = rows_for(H, KV);
   if (nsplit > 1 || work) {
     if (!scratch || (long long)num_items * KV > SI_ATTN_TICKETS) return -2;

@@ -1,4 +1,4 @@
-// Embedding gather: out[t, :] = scale * table[tokens[t], :], widened to fp32 (the residual
+// Embedding gather: out[t, :] = scale * table[tokens[t], :] (or its RMS norm times a weight, all fp32), widened to fp32 (the residual
 // stream is fp32 in both precisions; the product with the scale is fp32 too). The reference's kernel
 // (src/source/op/kernels/cuda/emb_kernel.cu:3-21) silently skips token ids outside
 // the vocabulary; here such a row is zeroed and the status word is set.
@@ -7,7 +7,8 @@
 template <typename TW>
 __global__ void embedding_gather_kernel(const int* __restrict__ tokens, const TW* __restrict__ table,
                                         float* __restrict__ out, int hidden, int vocab,
-                                        float scale, int* status) {
+                                        float scale, const float* __restrict__ norm_w, float eps, int* status) {
+  __shared__ float scratch[33];
   pdl_prologue();
   const int t = blockIdx.x;
   const int tok = tokens[t];
@@ -18,20 +19,30 @@ __global__ void embedding_gather_kernel(const int* __restrict__ tokens, const TW
     return;
   }
   const TW* w = table + (size_t)tok * hidden;
+  if (norm_w) {                              // a norm on the embedding's output, in the same launch
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
+      const float x = scale * to_f32<TW>(w[i]);
+      ss = fmaf(x, x, ss);
+    }
+    const float inv = rsqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = norm_w[i] * (scale * to_f32<TW>(w[i]) * inv);
+    return;
+  }
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) o[i] = scale * to_f32<TW>(w[i]);
 }
 
 SI_EXPORT int si_embedding_gather(const int* tokens, const void* table, int table_dtype, float* out,
-                                  int num_tokens, int hidden, int vocab, float scale, int* status,
-                                  cudaStream_t stream) {
+                                  int num_tokens, int hidden, int vocab, float scale, const float* norm_w, float eps,
+                                  int* status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   const int threads = hidden >= 1024 ? 256 : 128;
   if (table_dtype == SI_BF16)
     si_launch(embedding_gather_kernel<__nv_bfloat16>, dim3(num_tokens), dim3(threads), 0, stream,
-              tokens, (const __nv_bfloat16*)table, out, hidden, vocab, scale, status);
+              tokens, (const __nv_bfloat16*)table, out, hidden, vocab, scale, norm_w, eps, status);
   else
     si_launch(embedding_gather_kernel<float>, dim3(num_tokens), dim3(threads), 0, stream,
-              tokens, (const float*)table, out, hidden, vocab, scale, status);
+              tokens, (const float*)table, out, hidden, vocab, scale, norm_w, eps, status);
   return si_last_error();
 }
 

@@ -127,18 +127,20 @@ def _i32(t: Optional[torch.Tensor], name: str) -> None:
 
 # ---------------------------------------------------------------------------------------
 
-def embedding_gather(tokens, table, out, status=None, scale: float = 1.0) -> None:
-    """out[t,:] (fp32) = scale * table[tokens[t],:]."""
-    _cuda(tokens, table, out, status)
+def embedding_gather(tokens, table, out, status=None, scale: float = 1.0, norm_weight=None, eps: float = 0.0) -> None:
+    """out[t,:] (fp32) = x = scale * table[tokens[t],:], or with ``norm_weight`` (fp32 [hidden])
+    norm_weight * x * rsqrt(mean(x^2) + eps)."""
+    _cuda(tokens, table, out, status, norm_weight)
     _i32(tokens, "tokens")
     _need(out.dtype == torch.float32 and out.is_contiguous() and table.is_contiguous(),
           "embedding: out must be contiguous fp32, table contiguous")
     T, d = out.shape
     _need(table.shape[1] == d and tokens.numel() == T, "embedding: shape mismatch")
     f = _fn("embedding", "si_embedding_gather",
-            [_c_p, _c_p, _c_int, _c_p, _c_int, _c_int, _c_int, _c_f, _c_p, _c_p])
-    _check(f(_ptr(tokens), _ptr(table), _dt(table), _ptr(out), T, d, table.shape[0], float(scale),
-             _ptr(status), _stream()), "embedding_gather")
+            [_c_p, _c_p, _c_int, _c_p, _c_int, _c_int, _c_int, _c_f, _c_p, _c_f, _c_p, _c_p])
+    _f32v(norm_weight, "norm_weight", d)
+    _check(f(_ptr(tokens), _ptr(table), _dt(table), _ptr(out), T, d, table.shape[0], float(scale), _ptr(norm_weight),
+             float(eps), _ptr(status), _stream()), "embedding_gather")
 
 
 # Most bytes that one launch fetches ahead into L2. Measured on the 8B shape: 4 to 8 MB, what arrives while
@@ -580,15 +582,18 @@ def attn_decode_tma_work_floats(slots: int, H: int, KV: int, hs: int) -> int:
 
 def attn_decode_tma(q, k_cache, v_cache, block_table, items, out, page_size: int, num_seqs: int, H: int, KV: int,
                     hs: int, scale: float, window: int = 0, nsplit: int = 1, scratch=None, status=None,
-                    max_rows: int = 0, work=None) -> None:
+                    max_rows: int = 0, work=None, chunk: int = 0, sink=None) -> None:
     """``attn_decode`` with the K/V tiles fetched by TMA (head_dim 64 or 128, page sizes 8 to 64);
     items hold at most ``attn_decode_tma_rows // (H // KV)`` tokens. ``max_rows``: the most rows
     (tokens x query heads of a KV head) of any item when the caller knows it (0: unknown); at most 8
     rows run the variant with the products taken the other way round.
     ``work`` (int32 [W, 4], rows of (item, split, splits of that item, first slot of that item); item -1:
     nothing): every item is cut into its own number of shares, ``nsplit`` is not used, and ``scratch``
-    holds ``attn_decode_tma_work_floats(W, ...)`` floats. Made by ``split_work``."""
+    holds ``attn_decode_tma_work_floats(W, ...)`` floats. Made by ``split_work``. ``chunk`` and ``sink`` (fp32 [H]) as in
+    ``attention_general``."""
     _attn_common(q, k_cache, v_cache, block_table, items, out, page_size, H, KV, hs, "attn_decode_tma")
+    _cuda(sink)
+    _f32v(sink, "sink", H)
     if work is not None:
         _cuda(work, scratch)
         _need(work.dtype == torch.int32 and work.dim() == 2 and work.shape[1] == 4 and work.is_contiguous(),
@@ -603,12 +608,12 @@ def attn_decode_tma(q, k_cache, v_cache, block_table, items, out, page_size: int
               f"attn_decode_tma: scratch must hold {need} floats")
     f = _fn("attention_tma", "si_attn_decode_tma",
             [_c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_int, _c_p, _c_ll, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_f, _c_int, _c_int, _c_p, _c_int, _c_int, _c_p, _c_int, _c_p, _c_p])
+             _c_int, _c_int, _c_int, _c_f, _c_int, _c_int, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_p, _c_p, _c_p])
     W = work.shape[0] if work is not None else 0
     _check(f(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _cache_map(k_cache), _cache_map(v_cache),
              _ptr(block_table), block_table.shape[1], _ptr(items), items.shape[0], _ptr(out), out.stride(0),
              k_cache.shape[0], page_size, num_seqs, H, KV, hs, float(scale), int(window or 0), int(nsplit),
-             _ptr(work), W, W, _ptr(scratch), int(max_rows), _ptr(status), _stream()),
+             _ptr(work), W, W, _ptr(scratch), int(max_rows), int(chunk or 0), _ptr(sink), _ptr(status), _stream()),
            f"attn_decode_tma(heads={H}, kv_heads={KV}, head_dim={hs}, page_size={page_size})")
 
 
@@ -898,27 +903,29 @@ def attn_portion_tc05_tokens(H: int, KV: int) -> int:
 
 
 def attn_portion_tc05(q, k_cache, v_cache, block_table, items, out, page_size: int, num_seqs: int, H: int,
-                      KV: int, hs: int, scale: float, window: int = 0, status=None, slopes=None, q_temp=None, gate=None) -> None:
+                      KV: int, hs: int, scale: float, window: int = 0, status=None, slopes=None, q_temp=None, gate=None,
+                      chunk: int = 0, sink=None) -> None:
     """``attn_portion`` on the tcgen05 tensor cores (TMA-fed K/V tiles, S and P V in tensor memory);
     head_dim 64 or 128, page sizes 8 to 64, items of at most ``attn_portion_tc05_tokens`` tokens. ``v_cache`` None: the
-    values are the keys. ``slopes``, ``q_temp`` (a coefficient that is not negative) and ``gate`` as in ``attention_general``
-    (the gate's rows 16-byte aligned)."""
+    values are the keys. ``slopes``, ``q_temp`` (a coefficient that is not negative), ``gate``, ``chunk`` and ``sink`` as in
+    ``attention_general`` (the gate's rows 16-byte aligned)."""
     if v_cache is None:
         v_cache = k_cache
     _attn_common(q, k_cache, v_cache, block_table, items, out, page_size, H, KV, hs, "attn_portion_tc05")
-    _cuda(slopes, gate)
+    _cuda(slopes, gate, sink)
     _f32v(slopes, "slopes", H)
+    _f32v(sink, "sink", H)
     qt_coef, qt_every = _q_temp(q_temp)
     _need(qt_coef >= 0.0, "attn_portion_tc05: a query temperature with a negative coefficient is not supported")
     _need(gate is None or (gate.dtype == torch.bfloat16 and gate.shape == (q.shape[0], H * hs) and gate.stride(1) == 1
                            and gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0), "attn_portion_tc05: gate must be bf16 [T, H*hs], rows 16-byte aligned")
     f = _fn("attention_tc05", "si_attn_portion_tc05",
             [_c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_int, _c_p, _c_ll, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_f, _c_int, _c_p, _c_ll, _c_p, _c_p])
+             _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_f, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_p])
     _check(f(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _cache_map(k_cache), _cache_map(v_cache),
              _ptr(block_table), block_table.shape[1], _ptr(items), items.shape[0], _ptr(out), out.stride(0),
              k_cache.shape[0], page_size, num_seqs, H, KV, hs, float(scale), int(window or 0), _ptr(slopes), qt_coef, qt_every,
-             _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(status),
+             _ptr(gate), gate.stride(0) if gate is not None else 0, int(chunk or 0), _ptr(sink), _ptr(status),
              _stream()), f"attn_portion_tc05(heads={H}, kv_heads={KV}, head_dim={hs}, page_size={page_size})")
 
 
@@ -963,7 +970,8 @@ def _q_temp(q_temp):
 
 def attention_general(q, k_cache, v_cache, block_table, row_seq, positions, out, page_size: int, num_seqs: int,
                       H: int, KV: int, dk: int, dv: int, scale: float, window: int = 0, dist_bias=None, sink=None,
-                      status=None, softcap: float = 0.0, v_share: int = 1, slopes=None, q_temp=None, gate=None) -> None:
+                      status=None, softcap: float = 0.0, v_share: int = 1, slopes=None, q_temp=None, gate=None,
+                      chunk: int = 0) -> None:
     """fp32-arithmetic attention over the paged cache with key size ``dk``, value size ``dv``, values from
     ``v_cache`` or (None) the first ``dv`` entries of the keys, a bias by distance ``dist_bias`` (fp32 [nd, H],
     row min(distance, nd - 1)) and a sink per head (fp32 [H]) in the softmax denominator. ``softcap`` > 0: the scaled
@@ -971,7 +979,7 @@ def attention_general(q, k_cache, v_cache, block_table, row_seq, positions, out,
     (``v_cache`` holds KV / v_share heads). ``slopes`` (fp32 [H]): ``slopes[h] * (i - j)`` is taken off the scaled score of
     query i and key j. ``q_temp`` ``(coef, every)``: row i's scale is multiplied by 1 + coef * ln(floor((i + 1) / every) + 1).
     ``gate`` ([T, H*dv] like ``q``, rows with a stride): the result is multiplied entry by entry with sigmoid(gate).
-    ``out`` may be fp32 whatever the storage."""
+    ``chunk`` > 0: a query sees keys of its own run of ``chunk`` positions alone (runs are counted from position 0). ``out`` may be fp32 whatever the storage."""
     _cuda(q, k_cache, v_cache, block_table, row_seq, positions, out, dist_bias, sink, slopes, gate, status)
     _need(gate is None or (gate.dtype == q.dtype and gate.shape == (q.shape[0], H * dv) and gate.stride(1) == 1),
           "attention_general: gate must be [T, H*dv] in q's dtype")
@@ -997,12 +1005,12 @@ def attention_general(q, k_cache, v_cache, block_table, row_seq, positions, out,
     _f32v(sink, "sink", H)
     f = _fn("attention_general", "si_attention_general",
             [_c_p, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_p, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_int, _c_p, _c_f, _c_int, _c_int, _c_p, _c_f, _c_int,
+             _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_int, _c_p, _c_f, _c_int, _c_int, _c_int, _c_p, _c_f, _c_int,
              _c_p, _c_ll, _c_p, _c_p])
     _check(f(_ptr(q), _dt(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
              _ptr(row_seq), _ptr(positions), _ptr(out), out.stride(0), k_cache.shape[0], page_size, T, num_seqs,
              H, KV, dk, dv, float(scale), int(window or 0), _ptr(dist_bias), nd, _ptr(sink), float(softcap or 0.0),
-             int(v_share), 1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0, _ptr(slopes), qt_coef,
+             int(v_share), 1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0, int(chunk or 0), _ptr(slopes), qt_coef,
              qt_every, _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(status), _stream()),
            f"attention_general(dk={dk}, dv={dv})")
 
@@ -1189,13 +1197,14 @@ def attn_flex_scratch_floats(num_items: int, H: int, KV: int, dv: int, nsplit: i
 
 def attn_flex(q, k_cache, v_cache, block_table, items, out, page_size: int, num_seqs: int, H: int, KV: int, dk: int,
               dv: int, scale: float, window: int = 0, dist_bias=None, sink=None, nsplit: int = 1, scratch=None,
-              status=None, max_rows: int = 0, softcap: float = 0.0, v_share: int = 1, slopes=None, q_temp=None, gate=None) -> None:
+              status=None, max_rows: int = 0, softcap: float = 0.0, v_share: int = 1, slopes=None, q_temp=None, gate=None,
+              chunk: int = 0) -> None:
     """``attention_general`` on the tensor cores for bfloat16. ``items``: int32 [n, 4] rows (sequence, first row,
     tokens, first position) of at most ``attn_flex_tokens`` tokens. ``nsplit`` > 1 cuts every item's keys into that
     many shares (decode rows over long contexts); ``scratch`` then holds ``attn_flex_scratch_floats`` floats.
     ``max_rows``: the most rows (tokens x query heads of a key head served together) of any item when the caller knows it
     (0: unknown); at most 16 rows over keys that are their own values let a block's warps take a value slice each.
-    ``softcap``, ``v_share``, ``slopes``, ``q_temp``, ``gate`` as in ``attention_general``; ``out`` may be fp32."""
+    ``softcap``, ``v_share``, ``slopes``, ``q_temp``, ``gate``, ``chunk`` as in ``attention_general``; ``out`` may be fp32."""
     _cuda(q, k_cache, v_cache, block_table, items, out, dist_bias, sink, scratch, slopes, gate, status)
     _need(gate is None or (gate.dtype == torch.bfloat16 and gate.shape == (q.shape[0], H * dv) and gate.stride(1) == 1
                            and gate.stride(0) % 2 == 0 and gate.data_ptr() % 4 == 0), "attn_flex: gate must be bf16 [T, H*dv], rows 4-byte aligned")
@@ -1227,12 +1236,12 @@ def attn_flex(q, k_cache, v_cache, block_table, items, out, page_size: int, num_
               f"attn_flex: scratch must hold {need} floats")
     f = _fn("attention_flex", "si_attn_flex",
             [_c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_p, _c_int, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_f, _c_int, _c_p, _c_int, _c_p, _c_int, _c_p, _c_int, _c_f, _c_int, _c_int, _c_p, _c_f, _c_int,
+             _c_int, _c_int, _c_f, _c_int, _c_p, _c_int, _c_p, _c_int, _c_p, _c_int, _c_f, _c_int, _c_int, _c_int, _c_p, _c_f, _c_int,
              _c_p, _c_ll, _c_p, _c_p])
     _check(f(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(items),
              items.shape[0], _ptr(out), out.stride(0), k_cache.shape[0], page_size, num_seqs, H, KV, dk, dv,
              float(scale), int(window or 0), _ptr(dist_bias), nd, _ptr(sink), int(nsplit), _ptr(scratch), int(max_rows),
-             float(softcap or 0.0), int(v_share), 1 if out.dtype == torch.float32 else 0, _ptr(slopes), qt_coef, qt_every,
+             float(softcap or 0.0), int(v_share), 1 if out.dtype == torch.float32 else 0, int(chunk or 0), _ptr(slopes), qt_coef, qt_every,
              _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(status), _stream()), f"attn_flex(heads={H}, kv_heads={KV}, dk={dk}, dv={dv})", kernels=2 if nsplit > 1 else 1)
 
 
@@ -1726,3 +1735,78 @@ def gated_add(resid, z1, b1, a, z2=None, b2=None, f=None, mult: float = 1.0) -> 
     fn = _fn("norm", "si_gated_add", [_c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_f, _c_p])
     _check(fn(_ptr(resid), _ptr(z1), _ptr(b1), _ptr(a), _ptr(z2), _ptr(b2), _ptr(f), _dt(z1), T, d, float(mult), _stream()),
            f"gated_add(hidden={d})")
+
+
+# ---- a residual stream in several copies --------------------------------------------------------------------------
+
+def stream_norm(src, weight, eps: float, out, streams: int, dst=None, y=None, mix=None, write=None, read=None, rows=None,
+                ahead=None) -> None:
+    """The connections between two sublayers of a model whose residual stream has S copies, and the norm of what the next
+    one reads (all fp32 but ``y`` and ``out``):
+        x'_t = sum_s mix[s, t] x_s + write[t] y;   u = sum_s read[s] x'_s;   out = weight * u * rsqrt(mean(u^2) + eps)
+    ``src`` [T, S, d] fp32 (S = ``streams``), or [T, d] where all copies are the same row. ``dst``
+    [T, S, d]: where x' goes (``src`` itself for an update in place; None: nowhere). ``y`` None: x' = x. ``read`` None: the
+    plain sum. ``rows`` (int32 [R]): output row r comes from row rows[r], and nothing is stored. ``ahead``: as in ``add_rmsnorm``."""
+    _cuda(src, weight, out, dst, y, mix, write, read, rows, ahead)
+    _i32(rows, "rows")
+    d = src.shape[-1]
+    spread = src.dim() == 2
+    S = int(streams)
+    _need(spread or src.shape[1] == S, "stream_norm: src must be [T, streams, d] or [T, d]")
+    _need(src.dtype == torch.float32 and src.is_contiguous() and out.is_contiguous() and out.dim() == 2 and out.shape[1] == d
+          and weight.is_contiguous() and weight.numel() == d, "stream_norm: src must be contiguous fp32, out and weight of its width")
+    _need(out.shape[0] == (rows.numel() if rows is not None else src.shape[0]), "stream_norm: row count mismatch")
+    _need(dst is None or (rows is None and y is not None and dst.dtype == torch.float32 and dst.is_contiguous()
+                          and tuple(dst.shape) == (src.shape[0], S, d)), "stream_norm: dst goes with y, without rows, and is fp32 [T, S, d]")
+    if y is not None:
+        _need(y.is_contiguous() and tuple(y.shape) == (src.shape[0], d) and y.dtype == out.dtype and mix is not None and write is not None,
+              "stream_norm: y must be [T, d] in out's dtype, with mix and write")
+    _f32v(mix, "mix", S * S); _f32v(write, "write", S); _f32v(read, "read", S)
+    ahead_bytes = 0
+    if ahead is not None:
+        ahead_bytes = min(ahead.numel() * ahead.element_size(), AHEAD_BYTES) if ahead.is_contiguous() else 0
+    f = _fn("streams", "si_stream_norm",
+            [_c_p, _c_ll, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_int, _c_int, _c_int, _c_int, _c_f,
+             _c_p, _c_ll, _c_p])
+    _check(f(_ptr(src), d if spread else S * d, 0 if spread else d, _ptr(dst), _ptr(y), _ptr(mix), _ptr(write), _ptr(read),
+             _ptr(rows), _ptr(weight), _dt(weight), _ptr(out), _dt(out), out.shape[0], S, d, float(eps),
+             _ptr(ahead) if ahead_bytes else None, ahead_bytes, _stream()), f"stream_norm(streams={S}, width={d})")
+
+
+# ---- short convolutions over q, k and v ---------------------------------------------------------------------------
+
+def qkv_conv(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, block_table, k_cache, v_cache, page_size: int,
+             num_seqs: int, NQ: int, NK: int, NV: int, dk: int, dv: int, q_out, norm: bool, eps: float, q_weight=None,
+             k_weight=None, longest: int = 0, status=None) -> None:
+    """Rows ``u`` = [q: NQ*dk | k: NK*dk | v: NV*dv | ...] of a stacked projection, plus ``bias`` (fp32 [C] or None), through a
+    causal convolution over time per channel (``taps`` fp32 [K, C]; zeros before the sequence), then with ``norm`` every q and
+    k vector divided by its root mean square (times ``q_weight`` / ``k_weight``, fp32 [dk], where given); q into ``q_out``
+    [T, NQ*dk], k and v into their pages (``k_cache`` None: the queries alone are kept). ``state`` (fp32 [slots, >= (K-1)*C];
+    None for K = 1) holds each request's last K - 1 values of every channel and is renewed. ``longest``: the most rows that a
+    sequence of the step brings (1: a decode step, one launch; 0: not known)."""
+    _cuda(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, block_table, k_cache, v_cache, q_out, q_weight, k_weight, status)
+    for t, nm in ((positions, "positions"), (row_seq, "row_seq"), (q_start, "q_start"), (ctx_len, "ctx_len"), (slots, "slots"),
+                  (block_table, "block_table")):
+        _i32(t, nm)
+    T = u.shape[0]
+    C = (NQ + NK) * dk + NV * dv
+    K = taps.shape[0]
+    _need(u.stride(1) == 1 and u.shape[1] >= C and tuple(taps.shape) == (K, C), "qkv_conv: u must hold C channels, taps [K, C]")
+    _f32v(taps, "taps"); _f32v(bias, "bias", C); _f32v(q_weight, "q_weight", dk); _f32v(k_weight, "k_weight", dk)
+    _need(q_out.dtype == u.dtype and q_out.stride(1) == 1 and tuple(q_out.shape) == (T, NQ * dk), "qkv_conv: q_out must be [T, NQ*dk] in u's dtype")
+    _need(K == 1 or (state is not None and state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
+                     and state.shape[1] >= (K - 1) * C), "qkv_conv: state must be fp32 [slots, >= (K-1)*C]")
+    if k_cache is not None:
+        _need(k_cache.dtype == u.dtype and k_cache.is_contiguous() and tuple(k_cache.shape[1:]) == (NK, page_size, dk),
+              "qkv_conv: keys must be [pages, NK, page_size, dk]")
+        _need(v_cache is not None and v_cache.dtype == u.dtype and v_cache.is_contiguous()
+              and tuple(v_cache.shape) == (k_cache.shape[0], NV, page_size, dv), "qkv_conv: values must be [pages, NV, page_size, dv]")
+    f = _fn("qkv_conv", "si_qkv_conv",
+            [_c_p, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_p, _c_int, _c_int,
+             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_f, _c_int, _c_p, _c_p])
+    _check(f(_ptr(u), _dt(u), u.stride(0), _ptr(bias), _ptr(taps), _ptr(state), state.stride(0) if state is not None else 0,
+             _ptr(positions), _ptr(row_seq), _ptr(q_start), _ptr(ctx_len), _ptr(slots), _ptr(block_table),
+             block_table.shape[1] if block_table is not None else 0, _ptr(k_cache), _ptr(v_cache),
+             k_cache.shape[0] if k_cache is not None else 0, page_size, T, num_seqs, NQ, NK, NV, dk, dv, K, _ptr(q_out),
+             q_out.stride(0), 1 if norm else 0, _ptr(q_weight), _ptr(k_weight), float(eps), int(longest), _ptr(status), _stream()),
+           f"qkv_conv(dk={dk}, dv={dv}, taps={K})", kernels=2 if K > 1 and longest != 1 else 1)

@@ -14,7 +14,7 @@ import torch
 
 from ..config.base import EmbedderSpec, ModelConfig, ModelSpec
 from ..csrc import ops
-from ..parts import Block, NormedDelta, SublayerGate, SummedDelta, embedder_class, feed_forward_class, mixer_class, norm_class, position_class
+from ..parts import Block, NormedDelta, StreamConnections, StreamDelta, SublayerGate, SummedDelta, embedder_class, feed_forward_class, mixer_class, norm_class, position_class
 from ..parts.linear import configure_library_gemm, linear
 from ..engine import tracing
 
@@ -50,8 +50,21 @@ class Model:
                 g1 = SublayerGate({"size": self.spec.hidden_size}, dtype, self.device)
             if ffn is not None and ls.feed_forward_gate_name is not None:
                 g2 = SublayerGate({"size": self.spec.hidden_size}, dtype, self.device)
-            self.blocks.append(Block(mixer, ffn, n1, n2, ls.arrangement, n1b, n2b, g1, g2, ls.residual_scale))
-        self.final_norm = norm_class(self.spec.final_norm.kind)(self.spec.final_norm.params, dtype, self.device)
+            c1 = c2 = None                            # connections to the streams, where the residual stream has several copies
+            if (ls.mixer_streams_prefix is not None) != (self.spec.streams is not None):
+                raise ValueError("a layer has connections to several streams exactly where the model has streams")
+            if ls.mixer_streams_prefix is not None:
+                c1 = StreamConnections({"streams": self.spec.streams}, dtype, self.device)
+                if ffn is not None:
+                    c2 = StreamConnections({"streams": self.spec.streams}, dtype, self.device)
+            self.blocks.append(Block(mixer, ffn, n1, n2, ls.arrangement, n1b, n2b, g1, g2, ls.residual_scale, c1, c2))
+        if self.spec.streams is not None and self.spec.stream_adds:
+            raise ValueError("additions between layers go with a single residual stream")
+        # a scale on the logits is a gain of the final norm, so that it costs nothing and rounds nothing twice
+        fparams = dict(self.spec.final_norm.params)
+        if self.spec.logit_scale != 1.0:
+            fparams["gain"] = float(fparams.get("gain", 1.0)) * float(self.spec.logit_scale)
+        self.final_norm = norm_class(self.spec.final_norm.kind)(fparams, dtype, self.device)
         # the embedder: by default the plain table under the spec's embedding name
         es = self.spec.embedder or EmbedderSpec("table", {})
         self._embed_prefix, _, last = self.spec.embed_name.rpartition(".")
@@ -85,6 +98,10 @@ class Model:
                 yield p + ls.mixer_gate_name, b.mixer_gate
             if b.feed_forward_gate is not None:
                 yield p + ls.feed_forward_gate_name, b.feed_forward_gate
+            if b.mixer_streams is not None:
+                yield p + ls.mixer_streams_prefix, b.mixer_streams
+            if b.feed_forward_streams is not None:
+                yield p + ls.feed_forward_streams_prefix, b.feed_forward_streams
             if b.feed_forward is not None:
                 yield p + ls.feed_forward_prefix, b.feed_forward
                 if b.feed_forward_norm is not None:
@@ -124,6 +141,13 @@ class Model:
         for prefix, part in self._named_parts():
             if name.startswith(prefix) and name[len(prefix):] in part.weight_shapes():
                 return part.norm_like(name[len(prefix):])
+        return False
+
+    def identity_like(self, name: str) -> bool:
+        """True for square matrices that random weights draw around the identity (``Part.identity_like``)."""
+        for prefix, part in self._named_parts():
+            if name.startswith(prefix) and name[len(prefix):] in part.weight_shapes():
+                return part.identity_like(name[len(prefix):])
         return False
 
     def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -173,13 +197,16 @@ class Model:
         ``ctx.logit_rows`` or None when no row is wanted. ``caches[o]`` is the view of the o-th
         place in the run order (a layer that runs twice has a cache per run)."""
         T, d = ctx.num_tokens, self.spec.hidden_size
-        resid = ctx.buf("resid", (T, d), torch.float32)
-        self.embedder.forward(ctx, resid, caches[len(self.spec.order)].state)
+        S = self.spec.streams
+        resid = ctx.buf("resid", (T, d) if S is None else (T, S, d), torch.float32)
+        # several streams: all start as the embedder's rows, which stand for them until the first result is written
+        first = resid if S is None else ctx.buf("embed_out", (T, d), torch.float32)
+        self.embedder.forward(ctx, first, caches[len(self.spec.order)].state)
         embed_out = None
         if self._keeps_embedding:
             embed_out = ctx.buf("embed_out", (T, d), torch.float32)
             embed_out.copy_(resid)
-        delta = None
+        delta = None if S is None else StreamDelta(None, None, first)
         for o, i in enumerate(self.spec.order):
             add = self.stream_adds.get(o)
             if add is not None:                       # the pending delta goes in with what the stream gains here
@@ -192,13 +219,16 @@ class Model:
             else:
                 delta = self.blocks[i].forward(resid, delta, ctx, caches[o])
             if self._layer_hook is not None:
-                self._layer_hook(o, resid if delta is None else resid + (
+                self._layer_hook(o, delta.value(resid) if S is not None else resid if delta is None else resid + (
                     delta.value() if isinstance(delta, (NormedDelta, SummedDelta)) else delta.float()))
         R = ctx.num_logit_rows
         if R == 0:
             return None
         x = ctx.buf("final_x", (R, d), self.dtype)
-        self.final_norm.forward(resid, delta, x, rows=ctx.logit_rows)
+        if S is None:
+            self.final_norm.forward(resid, delta, x, rows=ctx.logit_rows)
+        else:                                         # the norm of the streams' sum
+            self.final_norm.forward_streams(resid, delta, None, x, rows=ctx.logit_rows)
         logits = ctx.buf("logits", (R, self.spec.vocab_size), torch.float32)
         linear(x, self.lm_head, logits, ctx.status)
         if self.spec.logit_softcap > 0:

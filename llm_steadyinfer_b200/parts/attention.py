@@ -25,10 +25,22 @@ Options beyond the reference's block, all parameters of the part:
 ``output_gate``    name of a matrix [heads * value_dim, hidden]: the heads' results are multiplied entry by entry with
                    ``sigmoid(W_g x)`` before the output projection; its rows are stacked behind q, k, v in one product, and the
                    attention kernels apply the gate when they store their results.
-With any option but ``names`` the mixer runs the general attention kernels (``attention_general.cu`` in 32-bit,
-``attention_flex.cu`` on the tensor cores in bfloat16) instead of the rotary ones. Sequences that bring a full work item of
+``biases``         the projections of q, k and v have biases (tensor names: the matrix's + ``bias_suffix``).
+``conv_taps``      K: every channel of q, k and v passes a causal convolution over time of K taps (tensor names: the matrix's +
+                   ``conv_suffix``, [channels, K], the last tap the current token's); the last K - 1 projected values of a request
+                   are its state.
+``qk_norm``        ``{"eps": e}``: every query and key head is divided by its root mean square (after the convolution).
+``sink_score``     a number s: exp(s) joins every row's softmax denominator once, without a value.
+``chunk``          positions fall into runs of so many, counted from position 0; a query sees keys of its own run alone.
+``own_keys``       False: the layer has no key and value projections and reads the cache of another one (its spec's
+                   ``cache_from``), whose keys lie there as that layer stored them.
+With any option but ``names`` the mixer runs its general form. Biases, convolution and norm are one launch behind the stacked
+projection (``qkv_conv.cu``), which also stores keys and values. The attention itself: where scores are plain but for the sink
+and the chunk and the layout is one that the fast kernels take (key size 64 or 128, values of the same size), decode rows go to
+``attention_tma.cu`` and prompt portions to ``attention_tc05.cu`` as in the reference's block; else the general kernels
+(``attention_general.cu`` in 32-bit, ``attention_flex.cu`` on the tensor cores in bfloat16). Sequences that bring a full work item of
 rows to a bfloat16 step go to the tcgen05 prompt kernel (``attention_tc05.cu``) where its layout fits (key size 64 or 128,
-values of the same size or the keys themselves, no bias table): it takes slopes, temperature and gate as well.
+values of the same size or the keys themselves, no bias table): it takes slopes, temperature, gate, chunks and sink as well.
 """
 from __future__ import annotations
 
@@ -38,7 +50,7 @@ import numpy as np
 import torch
 
 from ..csrc import ops
-from .base import CacheNeed, Mixer, register_mixer
+from .base import CacheNeed, Mixer, StateNeed, first_visible_key, register_mixer
 from . import flex_plan
 from . import linear as linear_mod
 from .linear import linear
@@ -66,8 +78,6 @@ class Attention(Mixer):
         self.window = params.get("window") or None
         if self.H % self.KV:
             raise ValueError(f"attention: {self.H} heads are not a multiple of {self.KV} kv heads")
-        if self.hs > 256:
-            raise ValueError(f"attention: head_dim {self.hs} above 256 is not supported")
         self.vs = int(params.get("value_dim") or self.hs)
         self.names = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight"}
         self.names.update(params.get("names") or {})
@@ -88,26 +98,64 @@ class Attention(Mixer):
         qt = params.get("query_temperature") or None
         self.q_temp = None if qt is None else (float(qt["coef"]), qt["every"])
         self.gate_name = params.get("output_gate") or None
-        self.general = (self.bias_spec is not None or self.vs != self.hs or not self.own_v or self.slopes is not None
-                        or self.q_temp is not None or self.gate_name is not None)
+        self.chunk = params.get("chunk") or None
+        self.sink_score = params.get("sink_score")
+        self.sink = None                 # fp32 [H] on the device
+        if self.sink_score is not None:
+            self.sink = torch.full((self.H,), float(self.sink_score), dtype=torch.float32, device=device)
+        self.biases = bool(params.get("biases", False))
+        self.bias_suffix = params.get("bias_suffix", ".bias")
+        self.taps = int(params.get("conv_taps") or 1)
+        self.has_conv = params.get("conv_taps") is not None
+        self.conv_suffix = params.get("conv_suffix", ".conv")
+        qkn = params.get("qk_norm") or None
+        self.qk_norm = qkn is not None
+        self.qk_eps = float(qkn["eps"]) if self.qk_norm else 0.0
+        self.own_keys = bool(params.get("own_keys", True))
+        self.prepared = self.biases or self.has_conv or self.qk_norm or not self.own_keys     # a launch behind the projection
+        # scores that the fast kernels know: q . k times the scale, a window or chunks, a sink
+        self.plain_scores = (self.bias_spec is None and self.vs == self.hs and self.own_v and self.slopes is None
+                             and self.q_temp is None and self.gate_name is None)
+        self.general = not self.plain_scores or self.prepared or self.chunk is not None or self.sink is not None
+        if self.hs > (1024 if self.general else 256) or self.vs > 1024:
+            raise ValueError(f"attention: head_dim {self.hs} is not supported (at most 256, 1,024 in the general form)")
+        if self.taps < 1:
+            raise ValueError(f"attention: {self.taps} convolution taps")
+        if self.prepared and (not self.own_v or self.gate_name is not None):
+            raise ValueError("attention: values that are the keys and an output gate go without biases, convolution, query/key "
+                             "norm and another layer's keys")
         if self.general and position is not None:
             raise ValueError("attention: the general form (a distance bias, slopes, a value size of its own, values that are "
                              "the keys, a query temperature, an output gate) goes without a position encoding")
         # columns of the stacked projection: q, k, v (if the layer has values of its own), the gate (if it has one)
-        self.kv_cols = self.KV * (self.hs + (self.vs if self.own_v else 0))
+        self.kv_cols = self.KV * (self.hs + (self.vs if self.own_v else 0)) if self.own_keys else 0
+        self.channels = self.H * self.hs + self.kv_cols
         self.gate_off = self.H * self.hs + self.kv_cols
         self.proj_cols = -(-(self.gate_off + (self.H * self.vs if self.gate_name else 0)) // 8) * 8 if self.general else 0
         self.dist_bias = None            # fp32 [distances, H], made at load
         self.qkv = None
+        self.qkv_bias = self.qkv_taps = None        # fp32 [channels], fp32 [taps, channels]
         self.o = None
+
+    def _projections(self):
+        """(name, rows) of the matrices in the stacked projection that biases and convolutions belong to."""
+        n = self.names
+        out = [(n["q"], self.H * self.hs)]
+        if self.own_keys:
+            out.append((n["k"], self.KV * self.hs))
+            if self.own_v:
+                out.append((n["v"], self.KV * self.vs))
+        return out
 
     def weight_shapes(self):
         n = self.names
-        shapes = {n["q"]: (self.H * self.hs, self.hidden),
-                  n["k"]: (self.KV * self.hs, self.hidden),
-                  n["o"]: (self.hidden, self.H * self.vs)}
-        if self.own_v:
-            shapes[n["v"]] = (self.KV * self.vs, self.hidden)
+        shapes = {n["o"]: (self.hidden, self.H * self.vs)}
+        for name, rows in self._projections():
+            shapes[name] = (rows, self.hidden)
+            if self.biases:
+                shapes[name + self.bias_suffix] = (rows,)
+            if self.has_conv:
+                shapes[name + self.conv_suffix] = (rows, self.taps)
         if self.gate_name:
             shapes[self.gate_name] = (self.H * self.vs, self.hidden)
         if self.bias_spec is not None:
@@ -115,15 +163,24 @@ class Attention(Mixer):
         return shapes
 
     def keeps_dtype(self, name):
-        return self.bias_spec is not None and name == self.bias_name
+        if self.bias_spec is not None and name == self.bias_name:
+            return True
+        return any((self.biases and name == p + self.bias_suffix) or (self.has_conv and name == p + self.conv_suffix)
+                   for p, _ in self._projections())
 
     def norm_like(self, name):
         return False
 
     def load_weights(self, tensors):
         n = self.names
-        parts = [tensors[n["q"]], tensors[n["k"]]] + ([tensors[n["v"]]] if self.own_v else []) \
-            + ([tensors[self.gate_name]] if self.gate_name else [])
+        parts = [tensors[name] for name, _ in self._projections()] + ([tensors[self.gate_name]] if self.gate_name else [])
+        stacked = lambda suffix: torch.cat([tensors[name + suffix].float() for name, _ in self._projections()], 0)
+        if self.biases:
+            self.qkv_bias = stacked(self.bias_suffix).contiguous()
+        if self.has_conv:
+            self.qkv_taps = stacked(self.conv_suffix).t().contiguous()
+        elif self.prepared:                                  # one tap of one: the value itself
+            self.qkv_taps = torch.ones(1, self.channels, dtype=torch.float32, device=parts[0].device)
         rows = sum(p.shape[0] for p in parts)
         if self.general and rows < self.proj_cols:           # rows of the product's result stay 16-byte aligned
             parts.append(torch.zeros(self.proj_cols - rows, self.hidden, dtype=parts[0].dtype, device=parts[0].device))
@@ -134,8 +191,14 @@ class Attention(Mixer):
 
     def cache_need(self):
         if not self.own_v:
-            return CacheNeed(self.KV, self.hs, self.window, 0)
-        return CacheNeed(self.KV, self.hs, self.window, None if self.vs == self.hs else self.vs)
+            return CacheNeed(self.KV, self.hs, self.window, 0, chunk=self.chunk)
+        return CacheNeed(self.KV, self.hs, self.window, None if self.vs == self.hs else self.vs, chunk=self.chunk)
+
+    def state_need(self):
+        if self.taps == 1:
+            return None
+        # rows of a multiple of four entries: a slot starts on a 16-byte boundary
+        return StateNeed((-(-(self.taps - 1) * self.channels // 4) * 4,), torch.float32)
 
     @property
     def capturable(self):
@@ -149,8 +212,18 @@ class Attention(Mixer):
 
     def kernel_files(self, page_size):
         if self.general:
-            return ("attention_general",) + (("attention_tc05", "attention_tma") if self.dtype == torch.bfloat16 and self.general_tc05_ok(page_size) else ()) + (
-                ("gemm_f32",) if self.dtype == torch.float32 else ("attention_flex", "gemm_skinny", "gemm_rows", "gemm_tc05"))
+            names = ["qkv_conv"] if self.prepared else ["attention_general"]          # what stores keys and values
+            if self.dtype == torch.float32:
+                return tuple(names + ["attention_general", "gemm_f32"])
+            names += ["gemm_skinny", "gemm_rows", "gemm_tc05"]
+            if self.uses_fast(page_size):
+                return tuple(names + ["attention_tma", "attention_tc05"])
+            names.append("attention_flex")
+            if self.hs % 8 or self.vs % 8:                                             # sizes that kernel does not take
+                names.append("attention_general")
+            if self.general_tc05_ok(page_size):
+                names += ["attention_tma", "attention_tc05"]
+            return tuple(names)
         names = ["rope_kv"] + (["gemm_f32"] if self.dtype == torch.float32 else ["gemm_skinny", "gemm_rows", "gemm_tc05"])
         if not self.uses_tensor_cores():
             return tuple(names + ["attention_ref"])
@@ -202,7 +275,7 @@ class Attention(Mixer):
     def _plan_general_tc05(self, ctx, page_size: int) -> dict:
         """Which sequences of the step go to the tcgen05 prompt kernel (those that bring at least one full item of rows),
         and their work items; the others are the general tensor-core kernel's."""
-        key = ("attention_general_tc05", self.H, self.KV, self.hs, self.window)
+        key = ("attention_general_tc05", self.H, self.KV, self.hs, self.window, self.chunk)
         got = ctx.plans.get(key)
         if got is not None:
             return got
@@ -220,39 +293,53 @@ class Attention(Mixer):
                 items += [(s, row0 + b, min(per, n - b), pos0 + b) for b in range(0, n, per)]
             if chosen:
                 out = {"skip": frozenset(chosen), "all": len(chosen) == ctx.num_seqs,
-                       "items": ctx.upload_ints(f"attn_gen_tc05_{self.H}_{self.KV}_{self.hs}_{self.window}",
+                       "items": ctx.upload_ints(f"attn_gen_tc05_{self._tag()}",
                                                 np.asarray(items, dtype=np.int32)).view(-1, 4)}
         ctx.plans[key] = out
         return out
 
     def forward_general(self, x, ctx, cache):
-        """No rotation; keys (and values of their own size, where the layer has them) into the pages as they are; scores with
-        the bias, the slopes and the query temperature; the gate on the heads' results."""
+        """No rotation; keys (and values of their own size, where the layer has them) into the pages as they are, or behind
+        biases, convolution and norm; scores with the bias, the slopes and the query temperature, the sink in the denominator;
+        the gate on the heads' results."""
         T = x.shape[0]
         H, KV, hs, vs = self.H, self.KV, self.hs, self.vs
         qkv = ctx.buf("attn_qkv", (T, self.proj_cols), self.dtype)
         linear(x, self.qkv, qkv, ctx.status)
         v_cache = cache.v if self.own_v else None
-        if cache.writes:
+        q = qkv[:, :H * hs]
+        if self.prepared:
+            q = ctx.buf("attn_q", (T, H * hs), self.dtype)
+            stores = cache.writes and self.own_keys
+            kv = KV if self.own_keys else 0
+            longest = 1 if ctx.seq_cap is not None else int(np.diff(ctx.h_q_start).max())
+            ops.qkv_conv(qkv, self.qkv_bias, self.qkv_taps, cache.state, ctx.positions, ctx.row_seq, ctx.q_start, ctx.ctx_len,
+                         ctx.slots, cache.block_table, cache.k if stores else None, cache.v if stores else None, cache.page_size,
+                         ctx.seq_slots, H, kv, kv, hs, vs, q, self.qk_norm, self.qk_eps, longest=longest, status=ctx.status)
+        elif cache.writes:
             ops.kv_store(qkv, ctx.positions, ctx.row_seq, cache.block_table, cache.k, v_cache, cache.page_size,
                          ctx.seq_slots, H, KV, hs, vs if self.own_v else 0, status=ctx.status)
         attn = ctx.buf("attn_out", (T, H * vs), self.dtype)
         gate = qkv[:, self.gate_off:self.gate_off + H * vs] if self.gate_name else None      # applied in the attention's epilogue
-        if self.uses_flex():
+        if self.uses_fast(cache.page_size):
+            self.attend(q, cache, ctx, attn)
+        elif self.uses_flex():
             big = self._plan_general_tc05(ctx, cache.page_size)
             if not big["all"]:
-                flex_plan.attend(flex_plan.plan(ctx, self.device, H, KV, hs, vs, self.own_v, self.window, skip=big["skip"]),
-                                 qkv[:, :H * hs], cache.k, v_cache, cache.block_table, attn, cache.page_size, ctx.seq_slots, H, KV,
-                                 hs, vs, self.scale, self.window, dist_bias=self.dist_bias, status=ctx.status, slopes=self.slopes,
-                                 q_temp=self.q_temp, gate=gate)
+                flex_plan.attend(flex_plan.plan(ctx, self.device, H, KV, hs, vs, self.own_v, self.window, skip=big["skip"],
+                                                chunk=self.chunk),
+                                 q, cache.k, v_cache, cache.block_table, attn, cache.page_size, ctx.seq_slots, H, KV,
+                                 hs, vs, self.scale, self.window, dist_bias=self.dist_bias, sink=self.sink, status=ctx.status,
+                                 slopes=self.slopes, q_temp=self.q_temp, gate=gate, chunk=self.chunk)
             if big["items"] is not None:
-                ops.attn_portion_tc05(qkv[:, :H * hs], cache.k, v_cache, cache.block_table, big["items"], attn, cache.page_size,
+                ops.attn_portion_tc05(q, cache.k, v_cache, cache.block_table, big["items"], attn, cache.page_size,
                                       ctx.seq_slots, H, KV, hs, self.scale, self.window or 0, status=ctx.status,
-                                      slopes=self.slopes, q_temp=self.q_temp, gate=gate)
+                                      slopes=self.slopes, q_temp=self.q_temp, gate=gate, chunk=self.chunk or 0, sink=self.sink)
         else:
-            ops.attention_general(qkv[:, :H * hs], cache.k, v_cache, cache.block_table, ctx.row_seq, ctx.positions, attn,
+            ops.attention_general(q, cache.k, v_cache, cache.block_table, ctx.row_seq, ctx.positions, attn,
                                   cache.page_size, ctx.seq_slots, H, KV, hs, vs, self.scale, self.window or 0,
-                                  dist_bias=self.dist_bias, status=ctx.status, slopes=self.slopes, q_temp=self.q_temp, gate=gate)
+                                  dist_bias=self.dist_bias, sink=self.sink, status=ctx.status, slopes=self.slopes,
+                                  q_temp=self.q_temp, gate=gate, chunk=self.chunk or 0)
         out = ctx.buf("delta", (T, self.hidden), self.dtype)
         linear(attn, self.o, out, ctx.status)
         return out
@@ -267,6 +354,17 @@ class Attention(Mixer):
         return (self.general and self.dtype == torch.bfloat16 and USE_TENSOR_CORES
                 and ops.attn_flex_ok(self.H, self.KV, self.hs, self.vs, self.own_v))
 
+    def uses_fast(self, page_size: int) -> bool:
+        """The general form whose scores the fast kernels know (the TMA-fed decode kernel, the tcgen05 prompt kernel)."""
+        return (self.general and self.plain_scores and self.dtype == torch.bfloat16 and USE_TENSOR_CORES and USE_TMA and USE_TC05
+                and self.hs in (64, 128) and page_size in (8, 16, 32, 64) and self.H // self.KV <= 32
+                and ops.attn_decode_tma_ok(self.H, self.KV, self.hs, page_size)
+                and ops.attn_portion_tc05_ok(self.H, self.KV, self.hs, page_size))
+
+    def _tag(self) -> str:
+        """Names the buffers of a plan: what layers that share it have in common."""
+        return f"{self.H}_{self.KV}_{self.hs}_{self.window}" + (f"_c{self.chunk}" if self.chunk else "")
+
     def uses_tensor_cores(self) -> bool:
         return not self.general and self.dtype == torch.bfloat16 and USE_TENSOR_CORES and self.hs % 16 == 0
 
@@ -274,15 +372,16 @@ class Attention(Mixer):
         """Cut the step's sequences into work items for the tensor-core kernels: runs of few
         tokens (decode rows) for the decode kernel, longer portions in runs of the portion
         kernel's item size. One plan serves every layer with the same head layout and window."""
-        if self.general:
+        if self.general and not self.uses_fast(cache.page_size):
             if self.uses_flex() and cache.k is not None:
                 big = self._plan_general_tc05(ctx, cache.page_size)
                 if not big["all"]:
-                    flex_plan.plan(ctx, self.device, self.H, self.KV, self.hs, self.vs, self.own_v, self.window, skip=big["skip"])
+                    flex_plan.plan(ctx, self.device, self.H, self.KV, self.hs, self.vs, self.own_v, self.window, skip=big["skip"],
+                                   chunk=self.chunk)
             return
-        if not self.uses_tensor_cores():
+        if not self.general and not self.uses_tensor_cores():
             return
-        key = ("attention", self.H, self.KV, self.hs, self.window)
+        key = ("attention", self.H, self.KV, self.hs, self.window, self.chunk)
         if key in ctx.plans or cache.k is None:
             return
         G = self.H // self.KV
@@ -316,7 +415,7 @@ class Attention(Mixer):
             # sequence beside short ones is cut into more of them; a second wave of blocks would wait.
             tiles = []
             for (_, _, n, pos0) in dec:
-                first = max(0, pos0 - self.window + 1) // 64 * 64 if self.window else 0
+                first = first_visible_key(pos0, self.window, self.chunk) // 64 * 64
                 tiles.append(-(-(pos0 + n - first) // 64) if n > 0 else 0)
             # Entries: every item whole, the shares that run at once, and room for finer cuts when items outnumber
             # those (entries without work are blocks that start and leave, so not more room than pays)
@@ -325,7 +424,7 @@ class Attention(Mixer):
             work = ops.split_work(tiles, budget, entries, MAX_SPLITS, MIN_TILES_PER_SPLIT)
             if ctx.seq_cap is None:                    # shapes are free: only the entries with work
                 work = work[:max(1, int((work[:, 0] >= 0).sum()))]
-            both = ctx.upload_ints(f"attn_dec_{self.H}_{self.KV}_{self.hs}_{self.window}",
+            both = ctx.upload_ints(f"attn_dec_{self._tag()}",
                                    np.concatenate([np.asarray(dec, dtype=np.int32).reshape(-1), work.reshape(-1)]))
             plan["dec"] = both[:4 * len(dec)].view(-1, 4)
             plan["work"] = both[4 * len(dec):].view(-1, 4)
@@ -338,34 +437,36 @@ class Attention(Mixer):
                 longest = max(d[3] + d[2] for d in dec)
                 nsplit = min(nsplit, max(1, -(-longest // (64 * MIN_TILES_PER_SPLIT))))
             plan["nsplit"] = nsplit
-            plan["dec"] = ctx.upload_ints(f"attn_dec_{self.H}_{self.KV}_{self.hs}_{self.window}",
+            plan["dec"] = ctx.upload_ints(f"attn_dec_{self._tag()}",
                                           np.asarray(dec, dtype=np.int32)).view(-1, 4)
             if nsplit > 1:
                 n = ops.attn_decode_scratch_floats(len(dec), self.H, self.KV, self.hs, nsplit)
                 plan["scratch"] = ctx.buf("attn_split", (n,), torch.float32)
         if por:
-            plan["por"] = ctx.upload_ints(f"attn_por_{self.H}_{self.KV}_{self.hs}_{self.window}",
+            plan["por"] = ctx.upload_ints(f"attn_por_{self._tag()}",
                                           np.asarray(por, dtype=np.int32)).view(-1, 4)
         ctx.plans[key] = plan
 
     def attend(self, q, cache, ctx, out):
-        if not self.uses_tensor_cores():
+        if not self.general and not self.uses_tensor_cores():
             ops.paged_attention_ref(q, cache.k, cache.v, cache.block_table, ctx.row_seq, ctx.positions,
                                     out, cache.page_size, ctx.seq_slots, self.H, self.KV, self.hs,
                                     self.scale, self.window or 0, status=ctx.status)
             return
-        plan = ctx.plans[("attention", self.H, self.KV, self.hs, self.window)]
+        plan = ctx.plans[("attention", self.H, self.KV, self.hs, self.window, self.chunk)]
+        # the fast kernels take chunks and a sink; a layout that has neither may run the others
+        extra = {"chunk": self.chunk, "sink": self.sink} if self.general else {}
         args = (cache.page_size, ctx.seq_slots, self.H, self.KV, self.hs, self.scale, self.window or 0)
         if plan["dec"] is not None:
             if plan["tma"]:
                 ops.attn_decode_tma(q, cache.k, cache.v, cache.block_table, plan["dec"], out, *args, work=plan["work"],
-                                    scratch=plan["scratch"], status=ctx.status, max_rows=plan["dec_rows"])
+                                    scratch=plan["scratch"], status=ctx.status, max_rows=plan["dec_rows"], **extra)
             else:
                 ops.attn_decode(q, cache.k, cache.v, cache.block_table, plan["dec"], out, *args,
                                 nsplit=plan["nsplit"], scratch=plan["scratch"], status=ctx.status)
         if plan["por"] is not None:
             portion = ops.attn_portion_tc05 if plan["tc05"] else ops.attn_portion
-            portion(q, cache.k, cache.v, cache.block_table, plan["por"], out, *args, status=ctx.status)
+            portion(q, cache.k, cache.v, cache.block_table, plan["por"], out, *args, status=ctx.status, **extra)
 
 
 def distance_bucket(n: int, rows: int, max_distance: float) -> int:

@@ -5,6 +5,7 @@ know which model or layer it sits in. Four kinds exist:
 
 ``Norm``              ``forward(resid, delta, out, rows=None)``: add ``delta`` into the fp32
                       residual stream and normalise it into ``out``.
+                      (on a stream of several copies: ``forward_streams``.)
 ``PositionEncoding``  gives a mixer what it needs to encode positions: ``rotary()`` returns
                       ``(inv_freq, rot_dim)`` for mixers that fuse the rotation, or None, in
                       which case the mixer calls ``apply(q, k, ctx)`` on unfused views.
@@ -36,11 +37,19 @@ from typing import Any, Callable, Dict, Optional, Tuple
 import torch
 
 
+def first_visible_key(pos: int, window: Optional[int], chunk: Optional[int]) -> int:
+    """The first key that the token at position ``pos`` sees: within the last ``window`` positions, and not before its run
+    of ``chunk`` positions (counted from position 0); None: no such limit."""
+    lo = max(0, pos - window + 1) if window else 0
+    return max(lo, pos // chunk * chunk) if chunk else lo
+
+
 @dataclass(frozen=True)
 class CacheNeed:
     """Paged keys and values of one layer: pages of [num_kv_heads, page_size, head_dim] for keys and
-    [num_kv_heads, page_size, value_dim] for values. ``window`` None keeps every token; otherwise pages
-    that lie wholly before ``position - window + 1`` are given back. ``value_dim`` None: as ``head_dim``;
+    [num_kv_heads, page_size, value_dim] for values. ``window`` and ``chunk`` None keep every token; otherwise pages
+    that lie wholly before the next token's ``first_visible_key`` are given back (as far as no layer that reads this
+    layer's cache still sees them). ``value_dim`` None: as ``head_dim``;
     0: the layer keeps no values of their own (a latent that serves as key and value). ``num_value_heads`` None:
     as many value heads as key heads; otherwise the value pages hold that many heads (several key heads that read
     one value head, as the maps of a differential attention do)."""
@@ -49,6 +58,7 @@ class CacheNeed:
     window: Optional[int] = None
     value_dim: Optional[int] = None
     num_value_heads: Optional[int] = None
+    chunk: Optional[int] = None
 
     @property
     def v_dim(self) -> int:
@@ -62,8 +72,10 @@ class CacheNeed:
         """What two layers must share for one to read the other's pages."""
         return ("paged_kv", self.num_kv_heads, self.head_dim, self.v_dim, self.v_heads)
 
-    def group_key(self) -> Tuple:
-        return self.layout_key() + (self.window,)
+    @property
+    def reach(self) -> Tuple[Optional[int], Optional[int]]:
+        """(window, chunk): how far back a token reads."""
+        return (self.window or None, self.chunk or None)
 
 
 @dataclass(frozen=True)
@@ -103,6 +115,25 @@ class SummedDelta:
         return self.a.float() + self.b.float()
 
 
+@dataclass
+class StreamDelta:
+    """What a sublayer leaves to be done to a residual stream kept in S copies: ``y`` [T, d] in the compute dtype, the
+    sublayer's result, and ``connections`` (``StreamConnections``) with the numbers that write it back; the next norm's
+    launch does it. ``spread`` [T, d] fp32: the streams are still one row each, this one, and have not been stored yet.
+    ``y`` None (with ``spread``): the state before the first sublayer."""
+    y: Optional[torch.Tensor]
+    connections: Optional["Part"]
+    spread: Optional[torch.Tensor] = None
+
+    def value(self, resid: torch.Tensor) -> torch.Tensor:
+        """The sum of the streams once this is done, from the stored streams ``resid`` [T, S, d] (hooks and tests)."""
+        x = resid if self.spread is None else self.spread.unsqueeze(1).expand(resid.shape)
+        if self.y is None:
+            return x.sum(1)
+        c = self.connections
+        return torch.einsum("s,tsd->td", c.mix.sum(1), x) + c.write.sum() * self.y.float()
+
+
 class Part:
     # True if ``forward`` reads nothing on the host that changes from step to step: whatever depends on
     # the step comes from device tensors of ``ctx`` or is planned in ``prepare``, and nothing waits for
@@ -134,6 +165,10 @@ class Part:
         """True for tensors that random weights should draw around one instead of around zero (norm weights)."""
         return self.keeps_dtype(name)
 
+    def identity_like(self, name: str) -> bool:
+        """True for square matrices that random weights should draw around the identity."""
+        return False
+
     def streams_first(self, rows: int) -> Optional[torch.Tensor]:
         """The weights that ``forward`` on ``rows`` rows reads first, if it streams them from memory once
         (few rows); the launch before it may fetch them into L2 ahead. None: nothing to fetch ahead."""
@@ -152,6 +187,13 @@ class Norm(Part):
 
     def forward(self, resid: torch.Tensor, delta: Optional[torch.Tensor], out: torch.Tensor,
                 rows: Optional[torch.Tensor] = None) -> None:
+        raise NotImplementedError
+
+    def forward_streams(self, resid: torch.Tensor, delta: "StreamDelta", connections: Optional["Part"], out: torch.Tensor,
+                        rows: Optional[torch.Tensor] = None, ahead: Optional[torch.Tensor] = None) -> None:
+        """The norm on a residual stream of several copies (``resid`` [T, S, d]): do what ``delta`` leaves to be done,
+        read the row that ``connections`` make of the streams (None: their sum) and normalise it into ``out``. With
+        ``rows`` the streams stay as they are. Kinds that have no such form leave this unimplemented."""
         raise NotImplementedError
 
     def normalize(self, x: torch.Tensor, out: Optional[torch.Tensor] = None) -> None:

@@ -22,6 +22,11 @@ The add is one kernel in fp32 on the stream itself (``ops.gated_add``), so the b
 What it hands on is a ``SummedDelta``: the next norm's launch adds both results in fp32 before its own statistics. While the
 feed-forward runs, the scratch key "delta" (where parts put their results) stands for a second buffer, so that the mixer's
 result stays alive beside it.
+"streams" runs both sublayers, one after the other, on a residual stream kept in several copies: each reads a row made of
+all of them and writes its result back into all of them through numbers of its own (``StreamConnections``):
+    u = sum_s in1[s] x_s;  y = mixer(norm1(u));  x_t <- sum_s mix1[s, t] x_s + out1[t] y;  likewise the feed-forward
+``resid`` is [T, S, d] then, and what a sublayer hands on is a ``StreamDelta``: the next norm's launch writes the streams,
+reads for its own sublayer and normalises.
 Another arrangement (post-norm, ...) is added with ``register_arrangement`` and needs no change here.
 """
 from __future__ import annotations
@@ -31,8 +36,9 @@ from typing import Callable, Dict, Optional
 import torch
 
 from ..csrc import ops
-from .base import FeedForward, Mixer, Norm, NormedDelta, Part, SummedDelta
+from .base import FeedForward, Mixer, Norm, NormedDelta, Part, StreamDelta, SummedDelta
 from .linear import linear
+from .streams import StreamConnections
 
 _ARRANGEMENTS: Dict[str, Callable] = {}
 _CAPTURABLE: Dict[str, bool] = {}
@@ -92,7 +98,8 @@ class Block:
                  feed_forward_norm: Optional[Norm], arrangement_name: str = "pre_norm",
                  mixer_post_norm: Optional[Norm] = None, feed_forward_post_norm: Optional[Norm] = None,
                  mixer_gate: Optional[SublayerGate] = None, feed_forward_gate: Optional[SublayerGate] = None,
-                 residual_scale: float = 1.0):
+                 residual_scale: float = 1.0, mixer_streams: Optional[StreamConnections] = None,
+                 feed_forward_streams: Optional[StreamConnections] = None):
         self.mixer = mixer
         self.feed_forward = feed_forward
         self.mixer_norm = mixer_norm
@@ -102,6 +109,8 @@ class Block:
         self.mixer_gate = mixer_gate
         self.feed_forward_gate = feed_forward_gate
         self.residual_scale = float(residual_scale)
+        self.mixer_streams = mixer_streams
+        self.feed_forward_streams = feed_forward_streams
         self.arrangement = arrangement_name
         self._run = arrangement(arrangement_name)
         self.capturable = _CAPTURABLE[arrangement_name]
@@ -205,3 +214,21 @@ def parallel_gated(block: Block, resid, delta, ctx, cache):
 
 
 register_arrangement("parallel_gated", parallel_gated, capturable=True)
+
+
+def streams(block: Block, resid, delta, ctx, cache):
+    if block.mixer_streams is None or (block.feed_forward is not None and block.feed_forward_streams is None):
+        raise ValueError("arrangement 'streams' needs the connections of each sublayer to the streams")
+    T, _, d = resid.shape
+    x = ctx.buf("block_x", (T, d), block.mixer.dtype)
+    block.mixer_norm.forward_streams(resid, delta, block.mixer_streams, x, ahead=block.mixer.streams_first(T))
+    # before the first sublayer the streams are one row each; they are stored when the first result is written
+    spread = delta.spread if delta.y is None else None
+    a = StreamDelta(block.mixer.forward(x, ctx, cache), block.mixer_streams, spread)
+    if block.feed_forward is None:
+        return a
+    block.feed_forward_norm.forward_streams(resid, a, block.feed_forward_streams, x, ahead=block.feed_forward.streams_first(T))
+    return StreamDelta(block.feed_forward.forward(x, ctx), block.feed_forward_streams)
+
+
+register_arrangement("streams", streams, capturable=True)

@@ -1,7 +1,8 @@
 """Embedders: the step's tokens into rows of the fp32 residual stream.
 
 ``table``        ``x = scale * table[token]`` (``scale`` 1 unless given): the reference's embedding
-                 (src/source/op/kernels/cuda/emb_kernel.cu:3-21) has no scale.
+                 (src/source/op/kernels/cuda/emb_kernel.cu:3-21) has no scale. With ``norm`` ``{"eps": e, "name": tensor}``
+                 the row passes an RMS norm with that weight, in the same launch.
 ``table_pair``   ``x = table[token] + pair[r]`` with a hashed embedding of the pair (previous token, token):
                  ``r = (previous * mul_prev + token * mul_cur) mod buckets``; the first token of a sequence takes
                  the pair table's extra last row, number ``buckets``. The previous token of a portion's first row is
@@ -25,18 +26,31 @@ class TableEmbedder(Embedder):
         self.hidden = int(params["hidden_size"])
         self.name = params.get("name", "weight")
         self.scale = float(params.get("scale", 1.0))
+        norm = params.get("norm") or None
+        self.norm_name = norm["name"] if norm else None
+        self.norm_eps = float(norm["eps"]) if norm else 0.0
+        self.norm_weight = None
 
     def weight_shapes(self):
-        return {self.name: (self.vocab, self.hidden)}
+        shapes = {self.name: (self.vocab, self.hidden)}
+        if self.norm_name is not None:
+            shapes[self.norm_name] = (self.hidden,)
+        return shapes
+
+    def keeps_dtype(self, name):
+        return self.norm_name is not None and name == self.norm_name
 
     def load_weights(self, tensors):
         self.table = tensors[self.name].contiguous()
+        if self.norm_name is not None:
+            self.norm_weight = tensors[self.norm_name].float().contiguous()
 
     def kernel_files(self, page_size):
         return ("embedding",)
 
     def forward(self, ctx, out, state):
-        ops.embedding_gather(ctx.tokens, self.table, out, status=ctx.status, scale=self.scale)
+        ops.embedding_gather(ctx.tokens, self.table, out, status=ctx.status, scale=self.scale, norm_weight=self.norm_weight,
+                             eps=self.norm_eps)
 
 
 class TablePairEmbedder(TableEmbedder):
@@ -46,8 +60,8 @@ class TablePairEmbedder(TableEmbedder):
         self.mul_prev = int(params["mul_prev"])
         self.mul_cur = int(params["mul_cur"])
         self.pair_name = params.get("pair_name", "pair")
-        if self.scale != 1.0:
-            raise ValueError("table_pair: a scale on the embedding is not supported")
+        if self.scale != 1.0 or self.norm_name is not None:
+            raise ValueError("table_pair: a scale or a norm on the embedding is not supported")
         if self.buckets <= 0 or self.mul_prev < 0 or self.mul_cur < 0:
             raise ValueError("table_pair: buckets must be positive and the multipliers not negative")
         self.pair = None

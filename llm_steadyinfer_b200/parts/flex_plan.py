@@ -11,15 +11,16 @@ import numpy as np
 import torch
 
 from ..csrc import ops
+from .base import first_visible_key
 
 MAX_SPLITS = 32
 MIN_KEYS_PER_SPLIT = 256
 BLOCKS_PER_SM = 2
 
 
-def plan(ctx, device, H: int, KV: int, dk: int, dv: int, own_v: bool, window, skip=frozenset()) -> dict:
-    """``skip``: sequences of the step that get no items (another path serves them)."""
-    key = ("flex", H, KV, dk, dv, own_v, window, tuple(sorted(skip)))
+def plan(ctx, device, H: int, KV: int, dk: int, dv: int, own_v: bool, window, skip=frozenset(), chunk=None) -> dict:
+    """``skip``: sequences of the step that get no items (another path serves them). ``window``, ``chunk``: what a row sees."""
+    key = ("flex", H, KV, dk, dv, own_v, window, chunk, tuple(sorted(skip)))
     got = ctx.plans.get(key)
     if got is not None:
         return got
@@ -40,7 +41,7 @@ def plan(ctx, device, H: int, KV: int, dk: int, dv: int, own_v: bool, window, sk
     if fixed:                                         # fixed shapes: pad with empty items, shares by the shape alone
         dec += [(0, 0, 0, 0)] * (ctx.seq_cap - len(dec))
     out = {"dec": None, "por": None, "nsplit": 1, "scratch": None, "dec_rows": 0}
-    tag = f"{H}_{KV}_{dk}_{dv}_{int(own_v)}_{window}" + ("_rest" if skip else "")
+    tag = f"{H}_{KV}_{dk}_{dv}_{int(own_v)}_{window}" + (f"_c{chunk}" if chunk else "") + ("_rest" if skip else "")
     if dec:
         # blocks one item gets without shares: kv heads x parts of the query heads x slices of the value columns
         gb = max(g for g in range(1, min(H // KV, 64) + 1) if (H // KV) % g == 0)
@@ -52,8 +53,10 @@ def plan(ctx, device, H: int, KV: int, dk: int, dv: int, own_v: bool, window, sk
         per = KV * ((H // KV) // gb) * slices
         nsplit = max(1, min(MAX_SPLITS, BLOCKS_PER_SM * ops.sm_count(device) // (len(dec) * per)))
         if not fixed:
-            longest = max(d[3] + d[2] for d in dec)
+            longest = max(d[3] + d[2] - first_visible_key(d[3], window, chunk) for d in dec)
             nsplit = min(nsplit, max(1, longest // MIN_KEYS_PER_SPLIT))
+        elif chunk:
+            nsplit = min(nsplit, max(1, chunk // MIN_KEYS_PER_SPLIT))
         out["nsplit"] = nsplit
         out["dec"] = ctx.upload_ints("flex_dec_" + tag, np.asarray(dec, dtype=np.int32)).view(-1, 4)
         if nsplit > 1:
@@ -67,12 +70,12 @@ def plan(ctx, device, H: int, KV: int, dk: int, dv: int, own_v: bool, window, sk
 
 def attend(pl: dict, q, k_cache, v_cache, block_table, out, page_size, seq_slots, H, KV, dk, dv, scale, window,
            dist_bias=None, sink=None, status=None, softcap: float = 0.0, v_share: int = 1, slopes=None, q_temp=None,
-           gate=None) -> None:
+           gate=None, chunk=None) -> None:
     args = (page_size, seq_slots, H, KV, dk, dv, scale, window or 0)
     if pl["dec"] is not None:
         ops.attn_flex(q, k_cache, v_cache, block_table, pl["dec"], out, *args, dist_bias=dist_bias, sink=sink,
                       nsplit=pl["nsplit"], scratch=pl["scratch"], status=status, max_rows=pl["dec_rows"], softcap=softcap,
-                      v_share=v_share, slopes=slopes, q_temp=q_temp, gate=gate)
+                      v_share=v_share, slopes=slopes, q_temp=q_temp, gate=gate, chunk=chunk or 0)
     if pl["por"] is not None:
         ops.attn_flex(q, k_cache, v_cache, block_table, pl["por"], out, *args, dist_bias=dist_bias, sink=sink, status=status,
-                      softcap=softcap, v_share=v_share, slopes=slopes, q_temp=q_temp, gate=gate)
+                      softcap=softcap, v_share=v_share, slopes=slopes, q_temp=q_temp, gate=gate, chunk=chunk or 0)

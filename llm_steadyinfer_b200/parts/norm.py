@@ -4,7 +4,8 @@ written back to the fp32 residual stream. Formula of the reference's
 constant in the kernel; here it is a parameter of the part. With ``scalar`` the checkpoint holds one number
 for all coordinates (a tensor without dimensions), which is spread over the width when the weights are loaded.
 With ``offset`` c the checkpoint's vector is stored around zero and the norm multiplies by ``c + weight`` (summed in fp32
-when the weights are loaded, and kept in fp32).
+when the weights are loaded, and kept in fp32). With ``gain`` g the result is multiplied by g (the weight is, in fp32, when it
+is loaded).
 """
 from __future__ import annotations
 
@@ -27,6 +28,7 @@ class RMSNorm(Norm):
         self.name = params.get("weight_name", "weight")      # "" where the checkpoint names the vector by the prefix alone
         self.scalar = bool(params.get("scalar", False))     # one number for all coordinates
         self.offset = float(params.get("offset", 0.0))      # added to the stored vector
+        self.gain = float(params.get("gain", 1.0))          # what the result is multiplied by
         self.weight: Optional[torch.Tensor] = None
 
     def weight_shapes(self):
@@ -39,6 +41,8 @@ class RMSNorm(Norm):
         w = tensors[self.name]
         if self.offset:
             w = w.float() + self.offset
+        if self.gain != 1.0:
+            w = w.float() * self.gain
         self.weight = (w.reshape(1).expand(self.size) if self.scalar else w).contiguous()
 
     def norm_like(self, name):
@@ -55,6 +59,13 @@ class RMSNorm(Norm):
             ops.add_rmsnorm(resid, delta.a, self.weight, self.eps, out, rows=rows, ahead=ahead, delta2=delta.b)
         else:
             ops.add_rmsnorm(resid, delta, self.weight, self.eps, out, rows=rows, ahead=ahead)
+
+    def forward_streams(self, resid, delta, connections, out, rows=None, ahead=None):
+        c = delta.connections
+        ops.stream_norm(resid if delta.spread is None else delta.spread, self.weight, self.eps, out,
+                        dst=resid if rows is None and delta.y is not None else None, y=delta.y,
+                        mix=None if delta.y is None else c.mix, write=None if delta.y is None else c.write,
+                        read=None if connections is None else connections.read, rows=rows, ahead=ahead, streams=resid.shape[1])
 
     def add(self, resid, delta: NormedDelta, extra=None, vec=None):
         """``resid += norm(delta) (+ extra) (+ vec)`` with no norm of the stream behind it."""

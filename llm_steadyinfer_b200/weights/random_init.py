@@ -1,5 +1,5 @@
 """Random weights from a configuration and a seed: matrices and embeddings with mean 0 and
-standard deviation 0.02, norm weights 1 + 0.1 z. Every element is a function of (seed, tensor
+standard deviation 0.02, norm weights 1 + 0.1 z, the few matrices drawn around the identity I + 0.02 z. Every element is a function of (seed, tensor
 name, index of the element) alone, made of 64-bit integer arithmetic and one multiplication, so
 that the same values come out on the CPU and on a GPU, bit for bit, and a tensor's values do not
 depend on which other tensors exist: z is the sum of twelve uniform draws minus six (variance
@@ -58,7 +58,7 @@ def standard_draws(key: int, first: int, count: int, device) -> torch.Tensor:
     return (total.to(torch.float64) + (6.0 - 6.0 * 2097152.0)) * (1.0 / 2097152.0)
 
 
-def _draw(name: str, shape, is_norm: bool, seed: int, device, store_dtype: torch.dtype) -> torch.Tensor:
+def _draw(name: str, shape, is_norm: bool, seed: int, device, store_dtype: torch.dtype, identity: bool = False) -> torch.Tensor:
     n = 1
     for s in shape:
         n *= int(s)
@@ -67,6 +67,9 @@ def _draw(name: str, shape, is_norm: bool, seed: int, device, store_dtype: torch
     for a in range(0, n, _CHUNK):
         z = standard_draws(key, a, min(_CHUNK, n - a), device)
         z = 1.0 + NORM_STD * z if is_norm else MATRIX_STD * z      # float64, rounded once below
+        if identity:
+            at = torch.arange(a, a + z.numel(), dtype=torch.int64, device=z.device)
+            z = z + (at // int(shape[1]) == at % int(shape[1]))
         out[a:a + z.numel()] = z.to(store_dtype)
     return out.view(tuple(shape))
 
@@ -76,7 +79,7 @@ def random_tensors(model, seed: int, store_dtype: torch.dtype, device="cpu") -> 
     for name, shape in sorted(model.weight_shapes().items()):
         if any(s < 0 for s in shape):
             raise ValueError(f"random weights: the configuration leaves the shape of {name!r} to the checkpoint {list(shape)}")
-        out[name] = _draw(name, shape, model.norm_like(name), seed, device, store_dtype)
+        out[name] = _draw(name, shape, model.norm_like(name), seed, device, store_dtype, model.identity_like(name))
     return out
 
 
@@ -100,6 +103,6 @@ def init_random(model, seed: int, store_dtype: torch.dtype = torch.bfloat16) -> 
     checkpoint would be."""
     tensors = {}
     for name, shape in sorted(model.weight_shapes().items()):
-        t = _draw(name, shape, model.norm_like(name), seed, model.device, store_dtype)
+        t = _draw(name, shape, model.norm_like(name), seed, model.device, store_dtype, model.identity_like(name))
         tensors[name] = place(t, model.keeps_dtype(name), model.dtype, model.device)
     model.load_weights(tensors)
