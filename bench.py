@@ -316,6 +316,19 @@ def _fevosun_config(size="base"):
             "layers": [first] + one[1:] + one}, {"attention": att, "latent": lat, "latent_2": lat2, "feed_forward": routed}
 
 
+# ---- the Risizen design beside the closest existing models ---------------------------------------------------
+# Sizes as the Vibunex section's (--design-size): attention of `heads` heads of 128 over `kv` key/value heads (the Llama twin's),
+# convolutions of four taps, chunks of 8,192 (longer than the contexts here, so that both models read as many keys), every
+# fourth layer reading the keys of the layer before it; four streams; the Llama twin's feed-forward size.
+def _risizen_config(size="base"):
+    width, ff, heads, kv = _VIBUNEX_SIZES[size][:4]
+    own = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "conv": 4, "scale": 128 ** -0.5, "mask": {"size": 8192}}
+    mlp = {"kind": "dense", "ff": ff, "limit": 7.0}
+    layers = [{"type": "attention", "mixer": dict(own, kv_from=i - 1) if i % 4 == 3 else own, "mlp": mlp} for i in range(8)]
+    return {"architecture": "Risizen", "vocab": MIVORAX_VOCAB, "width": width, "streams": 4, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+            "layers": layers}, {"attention": own, "feed_forward": mlp, "streams": 4}
+
+
 def mivorax_section(args, section="mivorax") -> int:
     """Prefill of 2,048 tokens and decode (batch 8, context 4,096) of an 8-layer Mivorax model (2 latent attention,
     4 attention with distance bias, 2 state-space layers; width 2,048) and of a Llama model of the same width, depth,
@@ -336,7 +349,14 @@ def mivorax_section(args, section="mivorax") -> int:
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda:0")        # larger than L2: written between timed steps
     results = {}
     width, ff = MIVORAX_WIDTH, MIVORAX_FF
-    if section == "fevosun":
+    if section == "risizen":
+        # 8 layers (6 with keys of their own, 2 that read them; four streams) beside the Llama model of the same width, depth, heads,
+        # feed-forward size and vocabulary, its closest in the attention, and the Nufasun model, its closest in the feed-forward
+        width, ff, heads, kv = _VIBUNEX_SIZES[args.design_size][:4]
+        ris, mixers = _risizen_config(args.design_size)
+        designs = (("risizen", ris),) + ((("nufasun", _nufasun_config()),) if args.design_size == "base" else ()) \
+            + (("llama", _llama_twin(width, ff, heads, kv)),)
+    elif section == "fevosun":
         # 8 layers (4 attention whose values are its keys, 2 + 2 latent attention; one dense and 7 routed feed-forwards with 5,632
         # active entries a token, as the other models' feed-forwards) beside the Mivorax model (its closest in the mixers), the
         # Vibunex model (its closest in the feed-forward) and the Llama model of the same width, depth and vocabulary
@@ -480,16 +500,17 @@ def main() -> int:
     ap.add_argument("--profiler-range", action="store_true",
                     help="bracket the timed region of --section with cudaProfilerStart/Stop "
                          "(for ncu --profile-from-start off)")
-    ap.add_argument("--section", default="all", choices=["all", "decode", "prefill", "mivorax", "nufasun", "vibunex", "fevosun"],
+    ap.add_argument("--section", default="all", choices=["all", "decode", "prefill", "mivorax", "nufasun", "vibunex", "fevosun", "risizen"],
                     help="run only the device-timed decode steps or only the prefill (for profiling); 'mivorax': prefill "
                          "and decode of a Mivorax model at layer sizes of a real model beside a Llama model of equal "
                          "width, with time per kind of kernel (its own JSON line; the default workload is not run); "
                          "'nufasun': the same for a Nufasun model beside the Mivorax and Llama models; 'vibunex': the same for a "
                          "Vibunex model beside the Nufasun and Llama models; 'fevosun': the same for a Fevosun model beside the "
-                         "Mivorax, Vibunex and Llama models")
+                         "Mivorax, Vibunex and Llama models; 'risizen': the same for a Risizen model beside the Nufasun and Llama "
+                         "models")
     ap.add_argument("--design-size", default="base", choices=["narrow", "base", "wide"],
-                    help="--section vibunex / fevosun: width 1,024 / 2,048 / 4,096 with heads, experts and feed-forward to match")
-    ap.add_argument("--only-design", default=None, help="--section mivorax / nufasun / vibunex / fevosun: run this model alone (for profiling)")
+                    help="--section vibunex / fevosun / risizen: width 1,024 / 2,048 / 4,096 with heads, experts and feed-forward to match")
+    ap.add_argument("--only-design", default=None, help="--section mivorax / nufasun / vibunex / fevosun / risizen: run this model alone (for profiling)")
     args = ap.parse_args()
 
     if args.gpus != 1:
@@ -498,7 +519,7 @@ def main() -> int:
     if args.impl == "reference":
         return reference_arm(args)
     K, W = args.steps, max(3, args.warmup)
-    if args.section in ("mivorax", "nufasun", "vibunex", "fevosun"):
+    if args.section in ("mivorax", "nufasun", "vibunex", "fevosun", "risizen"):
         return mivorax_section(args, args.section)
 
     import torch

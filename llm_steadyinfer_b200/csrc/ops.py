@@ -1777,13 +1777,14 @@ def stream_norm(src, weight, eps: float, out, streams: int, dst=None, y=None, mi
 
 def qkv_conv(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, block_table, k_cache, v_cache, page_size: int,
              num_seqs: int, NQ: int, NK: int, NV: int, dk: int, dv: int, q_out, norm: bool, eps: float, q_weight=None,
-             k_weight=None, longest: int = 0, status=None) -> None:
+             k_weight=None, portions: int = 3, status=None) -> None:
     """Rows ``u`` = [q: NQ*dk | k: NK*dk | v: NV*dv | ...] of a stacked projection, plus ``bias`` (fp32 [C] or None), through a
     causal convolution over time per channel (``taps`` fp32 [K, C]; zeros before the sequence), then with ``norm`` every q and
     k vector divided by its root mean square (times ``q_weight`` / ``k_weight``, fp32 [dk], where given); q into ``q_out``
     [T, NQ*dk], k and v into their pages (``k_cache`` None: the queries alone are kept). ``state`` (fp32 [slots, >= (K-1)*C];
-    None for K = 1) holds each request's last K - 1 values of every channel and is renewed. ``longest``: the most rows that a
-    sequence of the step brings (1: a decode step, one launch; 0: not known)."""
+    None for K = 1) holds each request's last K - 1 values of every channel and is renewed. ``portions``: what the step
+    holds beside sequences of one row: 1 portions of several rows from position 0, 2 such portions from a later position (a second
+    launch), 3 both, 0 neither."""
     _cuda(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, block_table, k_cache, v_cache, q_out, q_weight, k_weight, status)
     for t, nm in ((positions, "positions"), (row_seq, "row_seq"), (q_start, "q_start"), (ctx_len, "ctx_len"), (slots, "slots"),
                   (block_table, "block_table")):
@@ -1803,10 +1804,11 @@ def qkv_conv(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, 
               and tuple(v_cache.shape) == (k_cache.shape[0], NV, page_size, dv), "qkv_conv: values must be [pages, NV, page_size, dv]")
     f = _fn("qkv_conv", "si_qkv_conv",
             [_c_p, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_p, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_f, _c_int, _c_p, _c_p])
+             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_f, _c_int, _c_p, _c_p, _c_p])
+    launches = ctypes.c_int(1)
     _check(f(_ptr(u), _dt(u), u.stride(0), _ptr(bias), _ptr(taps), _ptr(state), state.stride(0) if state is not None else 0,
              _ptr(positions), _ptr(row_seq), _ptr(q_start), _ptr(ctx_len), _ptr(slots), _ptr(block_table),
              block_table.shape[1] if block_table is not None else 0, _ptr(k_cache), _ptr(v_cache),
              k_cache.shape[0] if k_cache is not None else 0, page_size, T, num_seqs, NQ, NK, NV, dk, dv, K, _ptr(q_out),
-             q_out.stride(0), 1 if norm else 0, _ptr(q_weight), _ptr(k_weight), float(eps), int(longest), _ptr(status), _stream()),
-           f"qkv_conv(dk={dk}, dv={dv}, taps={K})", kernels=2 if K > 1 and longest != 1 else 1)
+             q_out.stride(0), 1 if norm else 0, _ptr(q_weight), _ptr(k_weight), float(eps), int(portions), ctypes.addressof(launches),
+             _ptr(status), _stream()), f"qkv_conv(dk={dk}, dv={dv}, taps={K})", kernels=launches.value)

@@ -7,13 +7,14 @@
 //   q into `q_out`; k and v into their pages [pages, NK or NV, page_size, size].
 // A layer that reads another layer's cache has NK = NV = 0: the queries alone.
 // Per request the slot of the state keeps the last K - 1 values p of every channel, [K - 1, C] fp32, oldest first; a
-// portion starts from them (from zeros at position 0) and leaves its own behind, so a sequence may be cut anywhere. A
-// sequence that brings one row (decode) has its slot renewed by the thread that read it; longer portions by a second small
-// launch, since other blocks read the old values. All arithmetic is fp32.
+// portion starts from them (from zeros at position 0) and leaves its own behind, so a sequence may be cut anywhere. The slot
+// of a sequence that brings one row (decode) is renewed by the threads that read it, that of a sequence from its start by the
+// threads of its last row (nobody reads the old values); the other portions' by a second small launch, since other blocks
+// read the old values. All arithmetic is fp32.
 //
 // The fast kernel: a thread holds eight neighbouring channels (16 bytes of bfloat16) with their taps, their last K - 1
-// inputs and their bias in registers and walks up to a few dozen rows, so that every input is read once; the threads of a
-// vector (a group of 2^n lanes) add their squares with shuffles. Sizes that are no multiples of 8, vectors above 256
+// inputs and their bias in registers and walks a few dozen rows (prompts; one row in decode steps), so that every input and
+// tap is read once; the threads of a vector (a group of 2^n lanes) add their squares with shuffles. Sizes that are no multiples of 8, vectors above 256
 // entries and more than four taps take the plain kernel: a warp a vector, every tap read where it lies.
 #include "common.cuh"
 
@@ -27,7 +28,8 @@ struct ConvArgs {
   int num_pages, page_size, num_tokens, num_seqs, NQ, NK, NV, dk, dv, C, K;
   void* q_out; long long q_out_stride;
   int norm; const float* q_w; const float* k_w; float eps;
-  int rows_per_block, lanes_qk, trigger;                 // fast kernel: rows a block walks, lanes a q or k vector
+  int lanes_qk, rows_per_block, trigger;                 // fast kernel: lanes a q or k vector, rows a block walks
+  int state_from_start;                                  // second launch: portions from position 0 as well (plain kernel)
   int* status;
 };
 
@@ -69,9 +71,26 @@ __device__ __forceinline__ long long conv_page(const ConvArgs& p, int seq, int p
   return page;
 }
 
-template <typename T, int K>
-__global__ void __launch_bounds__(256) qkv_conv_vec_kernel(const ConvArgs p) {
-  constexpr int HIST = K > 1 ? K - 1 : 1;
+// What a row needs beside its channels: looked up once by a thread each and shared by the block.
+struct ConvRow {
+  int seq, leaves, page, at;                             // seq -1: nothing to do; it renews the slot; its page (-1: no store), place there
+  int back, pos;                                         // rows of its portion before it
+  float* state;                                          // its sequence's slot
+};
+#define CONV_FROM_START 1
+#define CONV_CONTINUED 2
+#define CONV_ROWS 128                                    // most rows a block walks
+
+// R: 1 (a block has one row) or 4 (it walks rows_per_block rows, the loads of four of them in flight together). The last
+// values of the thread's channels stand in a ring of four, the row's place in it being a compile-time number, in pairs for
+// the packed fp32 instructions.
+template <typename T, int K, int R>
+__global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) {
+  static_assert(K >= 1 && K <= 4 && (R == 1 || R == 4), "");
+  constexpr int PACK = (int)sizeof(T) / 2;               // 16-byte pieces that hold eight channels
+  constexpr bool STAGED = R > 1 && PACK == 1;            // rows come through shared memory, four rows ahead of the sums
+  __shared__ ConvRow rows[R == 1 ? 1 : CONV_ROWS];
+  __shared__ uint4 stage[STAGED ? 2 * R * 256 : 1];      // [half][row][thread]: every thread reads what it fetched itself
   const int lane = threadIdx.x & 31;
   const int id = blockIdx.y * blockDim.x + threadIdx.x;
   // threads of the q and k vectors first (lanes_qk each, those beyond dk / 8 idle), then one for every 8 channels of v
@@ -85,100 +104,226 @@ __global__ void __launch_bounds__(256) qkv_conv_vec_kernel(const ConvArgs p) {
     const int e = (id - qk_threads) * 8;
     if (e < p.NV * p.dv) { vec = e / p.dv; off = e % p.dv; c = (p.NQ + p.NK) * p.dk + e; }
   }
-  const bool is_v = id >= qk_threads;
+  const bool is_v = id >= qk_threads, is_q = !is_v && vec < p.NQ;
   const bool on = c >= 0;
+  const bool norm = !is_v && p.norm;
   // the lanes of this thread's vector
   const unsigned group = p.lanes_qk >= 32 ? 0xffffffffu : ((1u << p.lanes_qk) - 1u) << (lane & ~(p.lanes_qk - 1));
-  float w[K][8], b[8], g[8], hist[HIST][8];              // hist[j]: the value j + 1 rows back
+  float2 w[K][4], b[4], ring[4][4];
 #pragma unroll
-  for (int e = 0; e < 8; ++e) { b[e] = 0.f; g[e] = 1.f; }
+  for (int e = 0; e < 4; ++e) b[e] = make_float2(0.f, 0.f);
+  auto load_pairs = [](const float* src, float2 (&v)[4]) {
+    const float4 lo = *reinterpret_cast<const float4*>(src), hi = *reinterpret_cast<const float4*>(src + 4);
+    v[0] = make_float2(lo.x, lo.y); v[1] = make_float2(lo.z, lo.w);
+    v[2] = make_float2(hi.x, hi.y); v[3] = make_float2(hi.z, hi.w);
+  };
   if (on) {                                              // weights: read before the wait for the kernel before this one
 #pragma unroll
-    for (int j = 0; j < K; ++j) load8<float>(p.w + (size_t)j * p.C + c, w[j]);
-    if (p.bias) load8<float>(p.bias + c, b);
-    if (!is_v && p.norm) {
-      const float* gw = vec < p.NQ ? p.q_w : p.k_w;
-      if (gw) load8<float>(gw + off, g);
+    for (int j = 0; j < K; ++j) load_pairs(p.w + (size_t)j * p.C + c, w[j]);
+    if (p.bias) load_pairs(p.bias + c, b);
+  }
+  const float* gw = !norm ? nullptr : is_q ? p.q_w : p.k_w;
+  const int t0 = blockIdx.x * p.rows_per_block, nrows = min(p.rows_per_block, p.num_tokens - t0);
+  if (threadIdx.x < nrows) {                             // the step's integers: copied in before any of its kernels began
+    const int t = t0 + threadIdx.x;
+    ConvRow r;
+    r.seq = p.row_seq[t];
+    r.pos = p.positions[t];
+    r.back = r.leaves = r.at = 0;
+    r.page = -1;
+    r.state = nullptr;
+    if (r.seq >= p.num_seqs) {
+      set_status(p.status, SI_BAD_SEQ);
+      r.seq = -1;
     }
+    if (r.seq >= 0) {
+      const int start = p.q_start[r.seq];
+      r.back = t - start;
+      const int end = p.q_start[r.seq + 1];
+      r.leaves = end - start == 1 || (t == end - 1 && r.pos == r.back);
+      if (p.state) r.state = p.state + (size_t)p.slots[r.seq] * p.state_stride;
+      if (p.k_cache) { r.page = (int)conv_page(p, r.seq, r.pos, true); r.at = r.pos % p.page_size; }
+    }
+    rows[threadIdx.x] = r;
   }
   if (p.trigger) pdl_trigger();
+  __syncthreads();
   pdl_wait();
-  const T* u = (const T*)p.u;
-  const int t0 = blockIdx.x * p.rows_per_block, t1 = min(p.num_tokens, t0 + p.rows_per_block);
+  const T* u = (const T*)p.u + (size_t)t0 * p.u_stride + c;
+  T* qo = (T*)p.q_out + (size_t)t0 * p.q_out_stride + c;
+  auto unpack = [](const uint4* src, float2 (&v)[4]) {
+    float f[8];
+    load8<T>(reinterpret_cast<const T*>(src), f);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = make_float2(f[2 * e], f[2 * e + 1]);
+  };
+  // row r of the four at hand: its values join the ring, y = the convolution; returns the sum of y^2
+  auto sums = [&](int r, int half, const uint4* raw, float2 (&y)[4]) {
+    float2 (&x)[4] = ring[r & 3];
+    if (STAGED) {
+      const uint4 mine = stage[(half * R + r) * 256 + threadIdx.x];
+      unpack(&mine, x);
+    } else {
+      unpack(raw + r * PACK, x);
+    }
+    float2 s2 = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      x[e] = __fadd2_rn(x[e], b[e]);
+      y[e] = __fmul2_rn(w[0][e], ring[(r - K + 1) & 3][e]);
+#pragma unroll
+      for (int j = 1; j < K; ++j) y[e] = __ffma2_rn(w[j][e], ring[(r - K + 1 + j) & 3][e], y[e]);
+      s2 = __ffma2_rn(y[e], y[e], s2);
+    }
+    return s2.x + s2.y;
+  };
+  const float inv_dk = 1.f / (float)p.dk;
+  auto normalise = [&](float ss, float2 (&y)[4]) {       // ss: over the whole vector
+    const float inv = rsqrtf(fmaf(ss, inv_dk, p.eps));
+#pragma unroll
+    for (int e = 0; e < 4; ++e) y[e] = __fmul2_rn(y[e], make_float2(inv, inv));
+    if (gw && on) {
+      float2 g[4];
+      load_pairs(gw + off, g);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[e] = __fmul2_rn(y[e], g[e]);
+    }
+  };
+  // where this thread's entries of a row go: q by rows, k and v by page and place in it
+  const int heads = is_v ? p.NV : p.NK, size = is_v ? p.dv : p.dk, head = is_v ? vec : vec - p.NQ;
+  const long long page_step = (long long)heads * p.page_size * size;
+  T* kv = is_q ? nullptr : (is_v ? (T*)p.v_cache : (T*)p.k_cache);
+  if (kv) kv += (long long)head * p.page_size * size + off;
+  auto put = [&](int i, const float2 (&y)[4]) {
+    T* dst;
+    if (is_q) {
+      dst = qo + (size_t)i * p.q_out_stride;
+    } else {
+      if (!kv || rows[i].page < 0) return;
+      dst = kv + rows[i].page * page_step + rows[i].at * size;
+    }
+    const float out[8] = {y[0].x, y[0].y, y[1].x, y[1].y, y[2].x, y[2].y, y[3].x, y[3].y};
+    store8<T>(dst, out);
+  };
+  auto fetch = [&](int i0, int half) {
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+      if (on && i0 + r < nrows)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(
+            &stage[(half * R + r) * 256 + threadIdx.x])), "l"(u + (size_t)(i0 + r) * p.u_stride));
+    asm volatile("cp.async.commit_group;\n" ::);
+  };
+  if (STAGED) fetch(0, 0);
   int seq_before = -1;
-  for (int t = t0; t < t1; ++t) {
-    const int seq = p.row_seq[t];
-    if (seq < 0 || seq >= p.num_seqs) {                  // a padding row of a fixed-shape step, or a fault
-      if (seq >= 0 && id == 0) set_status(p.status, SI_BAD_SEQ);
-      seq_before = -1;
-      continue;
+  for (int i0 = 0; i0 < nrows; i0 += R) {
+    uint4 raw[STAGED ? 1 : R * PACK];                    // the thread's channels of R rows
+    const int half = (i0 / R) & 1;
+    if (STAGED) {
+      fetch(i0 + R, half ^ 1);
+      asm volatile("cp.async.wait_group 1;\n" ::: "memory");      // the rows at i0 have arrived
     }
-    const int pos = p.positions[t];
-    const int start = p.q_start[seq];
-    float* st = p.state ? p.state + (size_t)p.slots[seq] * p.state_stride : nullptr;
-    if (on && K > 1 && seq != seq_before) {              // the block's first row, or a sequence's first row: its past
-      const int back = t - start;
 #pragma unroll
-      for (int j = 0; j < K - 1; ++j) {
-        const int d = j + 1;                             // rows back
-        if (d > pos) {
+    for (int r = 0; r < R && !STAGED; ++r)
+      if (on && i0 + r < nrows) {
 #pragma unroll
-          for (int e = 0; e < 8; ++e) hist[j][e] = 0.f;
-        } else if (d <= back) {
-          load8<T>(u + (size_t)(t - d) * p.u_stride + c, hist[j]);
+        for (int h = 0; h < PACK; ++h) raw[r * PACK + h] = reinterpret_cast<const uint4*>(u + (size_t)(i0 + r) * p.u_stride)[h];
+      }
+    if (R > 1) {
+      // four rows that go on from the row before them, none of which renews the slot: in pairs, so that their sums overlap
+      bool run = i0 + R <= nrows && seq_before >= 0;
 #pragma unroll
-          for (int e = 0; e < 8; ++e) hist[j][e] += b[e];
-        } else {
-          load8<float>(st + (size_t)(K - 1 - (d - back)) * p.C + c, hist[j]);
+      for (int r = 0; r < R; ++r) run = run && rows[i0 + r].seq == seq_before && !rows[i0 + r].leaves;
+      if (run) {
+#pragma unroll
+        for (int r = 0; r < R; r += 2) {                 // two at a time: what the registers hold
+          float2 y0[4], y1[4];
+          float s0 = 0.f, s1 = 0.f;
+          if (on) {
+            s0 = sums(r, half, raw, y0);
+            s1 = sums(r + 1, half, raw, y1);
+          }
+          if (norm) {
+            for (int o = 1; o < p.lanes_qk; o <<= 1) {
+              s0 += __shfl_xor_sync(group, s0, o);
+              s1 += __shfl_xor_sync(group, s1, o);
+            }
+            normalise(s0, y0);
+            normalise(s1, y1);
+          }
+          if (on) {
+            put(i0 + r, y0);
+            put(i0 + r + 1, y1);
+          }
+        }
+        continue;
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int i = i0 + r;
+      if (i >= nrows) break;
+      const int seq = rows[i].seq;
+      if (K > 1 && on && seq >= 0 && seq != seq_before) {          // the block's first row, or a sequence's: its past
+        const int pos = rows[i].pos, back = rows[i].back;
+        const float* st = rows[i].state + c;
+#pragma unroll
+        for (int d = 1; d < K; ++d) {                    // d rows back
+          float2 (&h)[4] = ring[(r - d) & 3];
+          if (d > pos) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) h[e] = make_float2(0.f, 0.f);
+          } else if (d <= back) {
+            uint4 old[PACK];
+#pragma unroll
+            for (int q = 0; q < PACK; ++q) old[q] = reinterpret_cast<const uint4*>(u + (ptrdiff_t)(i - d) * p.u_stride)[q];
+            unpack(old, h);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) h[e] = __fadd2_rn(h[e], b[e]);
+          } else {
+            load_pairs(st + (size_t)(K - 1 - (d - back)) * p.C, h);
+          }
         }
       }
-    }
-    seq_before = seq;
-    float y[8];
-    float ss = 0.f;
+      seq_before = seq;
+      if (seq < 0) continue;                             // a padding row of a fixed-shape step, or a fault
+      float2 y[4];
+      float ss = 0.f;
+      if (on) {
+        ss = sums(r, half, raw, y);
+        if (K > 1 && rows[i].leaves) {                   // nobody else reads or writes its slot in this launch
 #pragma unroll
-    for (int e = 0; e < 8; ++e) y[e] = 0.f;
-    if (on) {
-      float x[8];
-      load8<T>(u + (size_t)t * p.u_stride + c, x);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] += b[e];
-#pragma unroll
-      for (int e = 0; e < 8; ++e) {
-#pragma unroll
-        for (int j = 0; j < K - 1; ++j) y[e] = fmaf(w[j][e], hist[K - 2 - j][e], y[e]);
-        y[e] = fmaf(w[K - 1][e], x[e], y[e]);
-        ss = fmaf(y[e], y[e], ss);
-      }
-      if (K > 1) {
-#pragma unroll
-        for (int j = HIST - 1; j > 0; --j)
-#pragma unroll
-          for (int e = 0; e < 8; ++e) hist[j][e] = hist[j - 1][e];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) hist[0][e] = x[e];
-        if (p.q_start[seq + 1] - start == 1) {           // the sequence's only row: nobody else reads or writes its slot here
-#pragma unroll
-          for (int j = 0; j < K - 1; ++j) store8<float>(st + (size_t)(K - 2 - j) * p.C + c, hist[j]);
+          for (int d = 0; d < K - 1; ++d) {
+            const float2 (&h)[4] = ring[(r - d) & 3];
+            float* dst = rows[i].state + (size_t)(K - 2 - d) * p.C + c;
+            *reinterpret_cast<float4*>(dst) = make_float4(h[0].x, h[0].y, h[1].x, h[1].y);
+            *reinterpret_cast<float4*>(dst + 4) = make_float4(h[2].x, h[2].y, h[3].x, h[3].y);
+          }
         }
       }
+      if (norm) {                                        // whole groups of lanes are q and k, or not
+        for (int o = 1; o < p.lanes_qk; o <<= 1) ss += __shfl_xor_sync(group, ss, o);
+        normalise(ss, y);
+      }
+      if (on) put(i, y);
     }
-    if (!is_v && p.norm) {                               // whole groups of lanes are q and k, or not
-      for (int o = 1; o < p.lanes_qk; o <<= 1) ss += __shfl_xor_sync(group, ss, o);
-      const float inv = rsqrtf(ss / (float)p.dk + p.eps);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) y[e] *= inv * g[e];
-    }
-    if (!on) continue;
-    if (!is_v && vec < p.NQ) {
-      store8<T>((T*)p.q_out + (size_t)t * p.q_out_stride + c, y);
-    } else if (p.k_cache) {
-      const long long page = conv_page(p, seq, pos, lane == 0);
-      if (page < 0) continue;
-      const int at = pos % p.page_size;
-      if (is_v) store8<T>((T*)p.v_cache + (((size_t)page * p.NV + vec) * p.page_size + at) * p.dv + off, y);
-      else store8<T>((T*)p.k_cache + (((size_t)page * p.NK + (vec - p.NQ)) * p.page_size + at) * p.dk + off, y);
-    }
+  }
+}
+
+template <typename T, int R>
+static void conv_launch_vec(ConvArgs& p, int yb, int threads, cudaStream_t stream) {
+  p.rows_per_block = 1;
+  if (R > 1) {                                           // as many rows as let all blocks run at once (two a multiprocessor)
+    const long long blocks = 2LL * si_sm_count() / yb > 0 ? 2LL * si_sm_count() / yb : 1;
+    const long long per = (p.num_tokens + blocks - 1) / blocks;
+    p.rows_per_block = (int)(per > CONV_ROWS ? CONV_ROWS : (per + R - 1) / R * R);
+  }
+  const dim3 grid((p.num_tokens + p.rows_per_block - 1) / p.rows_per_block, yb);
+  p.trigger = si_pdl_trigger_mode((long long)grid.x * grid.y, 2LL * si_sm_count()) == 1;
+  switch (p.K) {
+    case 1: si_launch(qkv_conv_vec_kernel<T, 1, R>, grid, dim3(threads), 0, stream, p); break;
+    case 2: si_launch(qkv_conv_vec_kernel<T, 2, R>, grid, dim3(threads), 0, stream, p); break;
+    case 3: si_launch(qkv_conv_vec_kernel<T, 3, R>, grid, dim3(threads), 0, stream, p); break;
+    default: si_launch(qkv_conv_vec_kernel<T, 4, R>, grid, dim3(threads), 0, stream, p); break;
   }
 }
 
@@ -242,27 +387,35 @@ __global__ void __launch_bounds__(128) qkv_conv_kernel(const ConvArgs p) {
 // (sequence, channel); entry i is the value at row n - K + 1 + i of the portion, an old entry where that lies before it.
 template <typename T>
 __global__ void qkv_conv_state_kernel(const ConvArgs p) {
-  pdl_prologue();
   const int s = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= p.C) return;
+  // the step's integers and the weights do not depend on the kernel before this one
   const int row0 = p.q_start[s], n = p.q_start[s + 1] - row0;
-  if (n <= 1) return;
   const int pos0 = p.ctx_len[s] - n, H = p.K - 1;
   const float b = p.bias ? p.bias[c] : 0.f;
   const T* u = (const T*)p.u;
   float* st = p.state + (size_t)p.slots[s] * p.state_stride + c;
-  for (int i = 0; i < H; ++i) {                          // in order: an entry is read before a later turn overwrites it
+  pdl_wait();
+  if (n <= 1 || (pos0 == 0 && !p.state_from_start)) return;
+  auto entry = [&](int i) {
     const int r = n - H + i;
-    float x;
-    if (r >= 0) x = to_f32<T>(u[(size_t)(row0 + r) * p.u_stride + c]) + b;
-    else if (pos0 + r < 0) x = 0.f;
-    else x = st[(size_t)(H + r) * p.C];
-    st[(size_t)i * p.C] = x;
+    if (r >= 0) return to_f32<T>(u[(size_t)(row0 + r) * p.u_stride + c]) + b;
+    return pos0 + r < 0 ? 0.f : st[(size_t)(H + r) * p.C];
+  };
+  if (H <= 4) {                                          // all loads before the first store
+    float x[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) x[i] = i < H ? entry(i) : 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (i < H) st[(size_t)i * p.C] = x[i];
+    return;
   }
+  for (int i = 0; i < H; ++i) st[(size_t)i * p.C] = entry(i);      // in order: an entry is read before a later turn overwrites it
 }
 
 template <typename T>
-static int conv_launch(ConvArgs p, int longest, cudaStream_t stream) {
+static int conv_launch(ConvArgs p, int portions, int* launches, cudaStream_t stream) {
   const auto al = [](const void* q) { return ((uintptr_t)q % 16) == 0; };
   const int elem = 16 / (int)sizeof(T);
   bool vec = p.K <= 4 && p.dk % 8 == 0 && p.dk <= 256 && (p.NV == 0 || p.dv % 8 == 0) && p.u_stride % elem == 0 &&
@@ -274,33 +427,31 @@ static int conv_launch(ConvArgs p, int longest, cudaStream_t stream) {
     const long long want = (long long)(p.NQ + p.NK) * p.lanes_qk + (long long)p.NV * p.dv / 8;
     const int threads = want <= 128 ? 128 : 256;
     const int yb = (int)((want + threads - 1) / threads);
-    long long rows = (long long)p.num_tokens * yb / (8LL * si_sm_count());
-    p.rows_per_block = rows < 1 ? 1 : (rows > 16 ? 16 : (int)rows);
-    const dim3 grid((p.num_tokens + p.rows_per_block - 1) / p.rows_per_block, yb);
-    p.trigger = si_pdl_trigger_mode((long long)grid.x * grid.y, 2LL * si_sm_count()) == 1 && longest == 1;
-    switch (p.K) {
-      case 1: si_launch(qkv_conv_vec_kernel<T, 1>, grid, dim3(threads), 0, stream, p); break;
-      case 2: si_launch(qkv_conv_vec_kernel<T, 2>, grid, dim3(threads), 0, stream, p); break;
-      case 3: si_launch(qkv_conv_vec_kernel<T, 3>, grid, dim3(threads), 0, stream, p); break;
-      default: si_launch(qkv_conv_vec_kernel<T, 4>, grid, dim3(threads), 0, stream, p); break;
-    }
+    // a row a block while all of them run at once, else several rows whose loads overlap
+    if ((long long)p.num_tokens * yb <= 2LL * si_sm_count()) conv_launch_vec<T, 1>(p, yb, threads, stream);
+    else conv_launch_vec<T, 4>(p, yb, threads, stream);
   } else {
     const dim3 grid(p.num_tokens, (p.NQ + p.NK + p.NV + 3) / 4);
     si_launch(qkv_conv_kernel<T>, grid, dim3(128), 0, stream, p);
+    p.state_from_start = 1;
   }
-  if (p.K > 1 && longest != 1)
+  if (launches) *launches = 1;
+  if (p.K > 1 && (portions & (vec ? CONV_CONTINUED : CONV_CONTINUED | CONV_FROM_START))) {
+    if (launches) *launches = 2;
     si_launch(qkv_conv_state_kernel<T>, dim3((p.C + 127) / 128, p.num_seqs), dim3(128), 0, stream, p);
+  }
   return si_last_error();
 }
 
-// Most rows that one call's sequence brings: `longest` (1: a decode step, no second launch; 0: not known).
+// `portions`: what the step holds beside sequences of one row: 1 portions of several rows that begin at position 0, 2 such
+// portions that begin later, 3 both (or not known); 0 neither (a decode step). `launches` (may be null): kernels launched.
 // Returns 0, a CUDA error code, or -2 (size refused).
 SI_EXPORT int si_qkv_conv(const void* u, int dtype, long long u_stride, const float* bias, const float* w, float* state,
                           long long state_stride, const int* positions, const int* row_seq, const int* q_start,
                           const int* ctx_len, const int* slots, const int* block_table, int table_width, void* k_cache,
                           void* v_cache, int num_pages, int page_size, int num_tokens, int num_seqs, int NQ, int NK, int NV,
                           int dk, int dv, int K, void* q_out, long long q_out_stride, int norm, const float* q_w,
-                          const float* k_w, float eps, int longest, int* status, cudaStream_t stream) {
+                          const float* k_w, float eps, int portions, int* launches, int* status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (NQ < 0 || NK < 0 || NV < 0 || dk <= 0 || dv < 0 || K < 1 || num_seqs > 65535 || (K > 1 && !state)) return -2;
   if ((NK > 0 || NV > 0) && k_cache && (!block_table || page_size <= 0 || (NV > 0 && !v_cache))) return -2;
@@ -308,6 +459,6 @@ SI_EXPORT int si_qkv_conv(const void* u, int dtype, long long u_stride, const fl
   if (C > (1LL << 30) || state_stride < (long long)(K - 1) * C) return -2;
   ConvArgs p{u, u_stride, bias, w, state, state_stride, positions, row_seq, q_start, ctx_len, slots, block_table, table_width,
              k_cache, v_cache, num_pages, page_size, num_tokens, num_seqs, NQ, NK, NV, dk, dv, (int)C, K, q_out, q_out_stride,
-             norm, q_w, k_w, eps, 1, 1, 0, status};
-  return dtype == SI_BF16 ? conv_launch<__nv_bfloat16>(p, longest, stream) : conv_launch<float>(p, longest, stream);
+             norm, q_w, k_w, eps, 1, 1, 0, 0, status};
+  return dtype == SI_BF16 ? conv_launch<__nv_bfloat16>(p, portions, launches, stream) : conv_launch<float>(p, portions, launches, stream);
 }

@@ -125,7 +125,7 @@ __global__ void __launch_bounds__(512) stream_norm_vec_kernel(const StreamArgs p
     cluster.sync();
     ss = 0.f;
     for (int b = 0; b < parts; ++b) ss += *cluster.map_shared_rank(&part, b);
-    cluster.sync();                                      // no block leaves while another may still read its part
+    cluster.barrier_arrive();                            // this block has read the others' parts
   }
   const float inv = rsqrtf(ss / (float)p.width + p.eps);
   T* out = (T*)p.out + (size_t)r * p.width;
@@ -138,6 +138,7 @@ __global__ void __launch_bounds__(512) stream_norm_vec_kernel(const StreamArgs p
       store4<T>(out + 4 * c, make_float4(w.x * (u[v].x * inv), w.y * (u[v].y * inv), w.z * (u[v].z * inv), w.w * (u[v].w * inv)));
     }
   }
+  if (parts > 1) cluster.barrier_wait();                 // no block leaves while another may still read its part
 }
 
 // Any width and any number of streams: a column at a time, the column's streams and the row of u in shared memory.

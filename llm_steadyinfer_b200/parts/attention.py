@@ -312,10 +312,9 @@ class Attention(Mixer):
             q = ctx.buf("attn_q", (T, H * hs), self.dtype)
             stores = cache.writes and self.own_keys
             kv = KV if self.own_keys else 0
-            longest = 1 if ctx.seq_cap is not None else int(np.diff(ctx.h_q_start).max())
             ops.qkv_conv(qkv, self.qkv_bias, self.qkv_taps, cache.state, ctx.positions, ctx.row_seq, ctx.q_start, ctx.ctx_len,
                          ctx.slots, cache.block_table, cache.k if stores else None, cache.v if stores else None, cache.page_size,
-                         ctx.seq_slots, H, kv, kv, hs, vs, q, self.qk_norm, self.qk_eps, longest=longest, status=ctx.status)
+                         ctx.seq_slots, H, kv, kv, hs, vs, q, self.qk_norm, self.qk_eps, portions=_portions(ctx), status=ctx.status)
         elif cache.writes:
             ops.kv_store(qkv, ctx.positions, ctx.row_seq, cache.block_table, cache.k, v_cache, cache.page_size,
                          ctx.seq_slots, H, KV, hs, vs if self.own_v else 0, status=ctx.status)
@@ -467,6 +466,19 @@ class Attention(Mixer):
         if plan["por"] is not None:
             portion = ops.attn_portion_tc05 if plan["tc05"] else ops.attn_portion
             portion(q, cache.k, cache.v, cache.block_table, plan["por"], out, *args, status=ctx.status, **extra)
+
+
+def _portions(ctx) -> int:
+    """What the step holds beside sequences of one row, as ``ops.qkv_conv`` takes it: 1 portions from position 0, 2 portions
+    that go on, 3 both, 0 neither."""
+    if ctx.seq_cap is not None:                          # fixed shapes hold single rows
+        return 0
+    got = ctx.plans.get("portions")
+    if got is None:
+        n = np.diff(ctx.h_q_start)
+        fresh = np.asarray(ctx.h_ctx_len) == n
+        got = ctx.plans["portions"] = (1 if (fresh & (n > 1)).any() else 0) | (2 if (~fresh & (n > 1)).any() else 0)
+    return got
 
 
 def distance_bucket(n: int, rows: int, max_distance: float) -> int:
