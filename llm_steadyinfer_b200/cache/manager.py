@@ -45,6 +45,10 @@ class CacheGroup:
     tables: Dict[Hashable, List[int]] = field(default_factory=dict)   # request -> page per block, -1 = given back
 
     @property
+    def window(self) -> Optional[int]:
+        return self.need.window
+
+    @property
     def bounded(self) -> bool:
         """Pages that no later token can read are given back while the request lives."""
         return bool(self.reach)

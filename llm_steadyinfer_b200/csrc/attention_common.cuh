@@ -39,6 +39,7 @@ struct AttnParams {
   float* part_ml;           // [item][kv head][split][row][2]
   int* counters;            // [item][kv head] tickets of the split merge, zero between launches
   int num_pages, page_size, num_seqs, H, KV, G, hs;
+  int vs;                   // value size (the mma.sync kernels: hs)
   float scale_log2;         // scale * log2(e)
   int window, nsplit;
   int chunk;                // rows see keys of their own run of `chunk` positions (0: none); the mma.sync kernels take none

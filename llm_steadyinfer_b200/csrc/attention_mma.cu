@@ -475,7 +475,7 @@ static bool fill_params(AttnParams& p, const void* q, long long q_stride, const 
   p.num_pages = num_pages; p.page_size = page_size; p.num_seqs = num_seqs;
   p.H = H; p.KV = KV; p.G = H / KV; p.hs = hs;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.chunk = 0; p.sink = nullptr;
+  p.chunk = 0; p.sink = nullptr; p.vs = hs;
   p.window = window; p.nsplit = 1; p.status = status;
   return true;
 }

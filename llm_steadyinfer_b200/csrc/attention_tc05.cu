@@ -22,8 +22,12 @@
 // simple: S of the next key tile is issued behind P V of the current one, so it overwrites P only
 // after P has been read, and when S is complete so is every earlier product into O.
 //
+// Keys and values narrower than a tile's columns (multiples of 8): the tensor maps end at their sizes, so the boxes' further
+// columns arrive as zeros; the queries are padded likewise and results beyond the value size are not stored.
+//
 // The reference computes prompt attention row by row with its scalar split kernel
-// (src/source/op/kernels/cuda/paged_kernels.cu:96-206). Conditions here: head_dim 64 or 128, page size
+// (src/source/op/kernels/cuda/paged_kernels.cu:96-206). Conditions here: key and value sizes up to 128, multiples of 8
+// (the extended instance: 64 or 128, both alike), page size
 // a power of two from 8 to 64, G <= 128; other layouts use the mma.sync kernel. Every mbarrier wait
 // is bounded; when one runs out the block sets SI_WAIT_LIMIT and leaves without storing.
 #include "attention_common.cuh"
@@ -158,7 +162,7 @@ attn_portion_tc05_kernel(const AttnParams p, const __grid_constant__ CUtensorMap
       const int tl = r / p.G, hh = r - tl * p.G;
       const int tok = q * tile_tokens + tl;
       v[i] = make_uint4(0, 0, 0, 0);
-      if (row < rows && tl < tile_tokens && tok < item.ntok)
+      if (row < rows && tl < tile_tokens && tok < item.ntok && c * 8 < p.hs)
         v[i] = *reinterpret_cast<const uint4*>(p.q + (size_t)(item.row0 + tok) * p.q_stride + (size_t)(g * p.G + hh) * p.hs + c * 8);
     }
 #pragma unroll
@@ -430,7 +434,7 @@ attn_portion_tc05_kernel(const AttnParams p, const __grid_constant__ CUtensorMap
         const float s2 = p.sink[g * p.G + (hh < p.G ? hh : 0)] * LOG2E, M = fmaxf(m, s2), f = fast_exp2(m - M);
         inv = f / (l * f + fast_exp2(s2 - M));
       }
-      bf16* dst = p.out + (size_t)(item.row0 + tok) * p.out_stride + (size_t)(g * p.G + hh) * p.hs;
+      bf16* dst = p.out + (size_t)(item.row0 + tok) * p.out_stride + (size_t)(g * p.G + hh) * p.vs;
 #pragma unroll
       for (int c = 0; c < HS / 64; ++c) {
         float v[64];
@@ -459,7 +463,7 @@ attn_portion_tc05_kernel(const AttnParams p, const __grid_constant__ CUtensorMap
             raw.y = pack_bf16(v[8 * q8 + 2] * inv, v[8 * q8 + 3] * inv);
             raw.z = pack_bf16(v[8 * q8 + 4] * inv, v[8 * q8 + 5] * inv);
             raw.w = pack_bf16(v[8 * q8 + 6] * inv, v[8 * q8 + 7] * inv);
-            *reinterpret_cast<uint4*>(dst + c * 64 + q8 * 8) = raw;
+            if (c * 64 + q8 * 8 < p.vs) *reinterpret_cast<uint4*>(dst + c * 64 + q8 * 8) = raw;
           }
         }
       }
@@ -472,9 +476,9 @@ attn_portion_tc05_kernel(const AttnParams p, const __grid_constant__ CUtensorMap
 
 // ---- host side --------------------------------------------------------------------------------
 // 1 when this kernel takes the layout.
-SI_EXPORT int si_attn_portion_tc05_ok(int H, int KV, int hs, int page_size) {
+SI_EXPORT int si_attn_portion_tc05_ok(int H, int KV, int hs, int vs, int page_size) {
   if (KV <= 0 || H % KV || H / KV > 128) return 0;
-  if (hs != 64 && hs != 128) return 0;
+  if (hs <= 0 || vs <= 0 || hs > 128 || vs > 128 || hs % 8 || vs % 8) return 0;
   if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64) return 0;
   return si_encode_fn() != nullptr;
 }
@@ -504,7 +508,7 @@ static int launch(const AttnParams& p, const CUtensorMap& km, const CUtensorMap&
 SI_EXPORT int si_attn_portion_tc05(const void* q, long long q_stride, const void* k_cache, const void* v_cache,
                                    const void* kmap, const void* vmap, const int* block_table, int table_width,
                                    const void* items, int num_items, void* out, long long out_stride, int num_pages,
-                                   int page_size, int num_seqs, int H, int KV, int hs, float scale, int window,
+                                   int page_size, int num_seqs, int H, int KV, int hs, int vs, float scale, int window,
                                    const float* slopes, float qt_coef, int qt_every, const void* gate, long long gate_stride,
                                    int chunk, const float* sink, int* status, cudaStream_t stream) {
   if (num_items <= 0) return 0;
@@ -513,7 +517,7 @@ SI_EXPORT int si_attn_portion_tc05(const void* q, long long q_stride, const void
   const AttnExtras x{slopes, qt_coef, qt_every, (const bf16*)gate, gate_stride};
   const bool ext = slopes || qt_every > 0 || gate;
   if (num_items > 65535) return -2;                  // the grid's second dimension
-  if (!si_attn_portion_tc05_ok(H, KV, hs, page_size) || !kmap || !vmap) return -2;
+  if (!si_attn_portion_tc05_ok(H, KV, hs, vs, page_size) || !kmap || !vmap) return -2;
   if ((q_stride % 8) || (out_stride % 8) || ((uintptr_t)q % 16) || ((uintptr_t)out % 16)) return -2;
   AttnParams p;
   p.q = (const bf16*)q; p.q_stride = q_stride;
@@ -523,13 +527,15 @@ SI_EXPORT int si_attn_portion_tc05(const void* q, long long q_stride, const void
   p.out = (bf16*)out; p.out_stride = out_stride;
   p.part_o = nullptr; p.part_ml = nullptr; p.counters = nullptr;
   p.num_pages = num_pages; p.page_size = page_size; p.num_seqs = num_seqs;
-  p.H = H; p.KV = KV; p.G = H / KV; p.hs = hs;
+  p.H = H; p.KV = KV; p.G = H / KV; p.hs = hs; p.vs = vs;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.window = window; p.chunk = chunk; p.sink = sink; p.nsplit = 1; p.status = status;
   int log2_page = 0;
   while ((1 << log2_page) < page_size) ++log2_page;
   const CUtensorMap& km = *(const CUtensorMap*)kmap;
   const CUtensorMap& vm = *(const CUtensorMap*)vmap;
-  if (ext) return hs == 64 ? launch<1, true>(p, km, vm, num_items, log2_page, stream, x) : launch<2, true>(p, km, vm, num_items, log2_page, stream, x);
-  return hs == 64 ? launch<1, false>(p, km, vm, num_items, log2_page, stream, x) : launch<2, false>(p, km, vm, num_items, log2_page, stream, x);
+  if (ext && (hs != vs || (hs != 64 && hs != 128))) return -2;
+  const bool narrow = hs <= 64 && vs <= 64;
+  if (ext) return narrow ? launch<1, true>(p, km, vm, num_items, log2_page, stream, x) : launch<2, true>(p, km, vm, num_items, log2_page, stream, x);
+  return narrow ? launch<1, false>(p, km, vm, num_items, log2_page, stream, x) : launch<2, false>(p, km, vm, num_items, log2_page, stream, x);
 }

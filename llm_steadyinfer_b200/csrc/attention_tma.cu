@@ -13,7 +13,10 @@
 // addresses, which the cp.async version pays about 400 of per thread and tile, and never meet
 // at a block-wide barrier inside the loop.
 //
-// Conditions: head_dim 64 or 128, page_size a power of two from 8 to 64, at most 32 rows per
+// Keys and values narrower than a tile's 64 or 128 columns: the tensor maps end at their sizes, so the boxes' further columns
+// arrive as zeros, and results beyond the value size are not stored.
+//
+// Conditions: key and value sizes up to 128, multiples of 8, page_size a power of two from 8 to 64, at most 32 rows per
 // item. Everything else stays with the cp.async kernel. Every wait on an mbarrier is bounded:
 // when it runs out the block reports SI_WAIT_LIMIT in the status word and leaves.
 #include "attention_common.cuh"
@@ -391,8 +394,8 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
   // partial results: [slot0 + split][kv head][row]
   const size_t slab0 = ((size_t)slot0 * p.KV + g) * ROWS;
   const size_t slab_step = (size_t)p.KV * ROWS;                       // from one split to the next
-  for (int idx = threadIdx.x; idx < rows_used * p.hs; idx += THREADS) {
-    const int r = idx / p.hs, d = idx - r * p.hs;
+  for (int idx = threadIdx.x; idx < rows_used * p.vs; idx += THREADS) {
+    const int r = idx / p.vs, d = idx - r * p.vs;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < NWARPS; ++w) M = fmaxf(M, fm[w * ROWS + r]);
@@ -411,11 +414,11 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
         L = L * f + exp2f(s2 - Ms);
         acc *= f;
       }
-      p.out[(size_t)(item.row0 + tok) * p.out_stride + (size_t)(g * p.G + hh) * p.hs + d] =
+      p.out[(size_t)(item.row0 + tok) * p.out_stride + (size_t)(g * p.G + hh) * p.vs + d] =
           __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
     } else {
       const size_t slab = slab0 + (size_t)split * slab_step + r;
-      __stcg(p.part_o + slab * p.hs + d, acc);
+      __stcg(p.part_o + slab * p.vs + d, acc);
       if (d == 0) { __stcg(p.part_ml + slab * 2, M); __stcg(p.part_ml + slab * 2 + 1, L); }
     }
   }
@@ -461,11 +464,11 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
   asm volatile("bar.sync 1, 128;\n" ::: "memory");
   // four outputs a thread, sixteen 16-byte loads in flight: with a few rows (a decode step) every thread has
   // one turn, and the splits cost two round trips to L2 instead of one for every eight scalar loads
-  const int hs4 = p.hs >> 2;
-  for (int idx = threadIdx.x; idx < rows_used * hs4; idx += THREADS) {
-    const int r = idx / hs4, d = (idx - r * hs4) << 2;
-    const float* src = p.part_o + (slab0 + r) * p.hs + d;       // split sp lies sp * slab_step * hs further
-    const size_t step = slab_step * p.hs;
+  const int vs4 = p.vs >> 2;
+  for (int idx = threadIdx.x; idx < rows_used * vs4; idx += THREADS) {
+    const int r = idx / vs4, d = (idx - r * vs4) << 2;
+    const float* src = p.part_o + (slab0 + r) * p.vs + d;       // split sp lies sp * slab_step * vs further
+    const size_t step = slab_step * p.vs;
     const float* wr = w_s + r * nsplit;
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int sp = 0; sp < nsplit; sp += 16) {
@@ -483,7 +486,7 @@ attn_decode_tma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k
     }
     const float L = L_s[r];
     const int tok = r / p.G, hh = r - tok * p.G;
-    bf16* dst = p.out + (size_t)(item.row0 + tok) * p.out_stride + (size_t)(g * p.G + hh) * p.hs + d;
+    bf16* dst = p.out + (size_t)(item.row0 + tok) * p.out_stride + (size_t)(g * p.G + hh) * p.vs + d;
     dst[0] = __float2bfloat16_rn(L > 0.f ? acc.x / L : 0.f);
     dst[1] = __float2bfloat16_rn(L > 0.f ? acc.y / L : 0.f);
     dst[2] = __float2bfloat16_rn(L > 0.f ? acc.z / L : 0.f);
@@ -499,9 +502,9 @@ static int rows_for(int H, int KV) {
 }
 
 // 1 when the TMA decode kernel takes this layout.
-SI_EXPORT int si_attn_decode_tma_ok(int H, int KV, int hs, int page_size) {
+SI_EXPORT int si_attn_decode_tma_ok(int H, int KV, int hs, int vs, int page_size) {
   if (KV <= 0 || H % KV) return 0;
-  if (hs != 64 && hs != 128) return 0;
+  if (hs <= 0 || vs <= 0 || hs > 128 || vs > 128 || hs % 8 || vs % 8) return 0;
   if (page_size != 8 && page_size != 16 && page_size != 32 && page_size != 64) return 0;
   return rows_for(H, KV) > 0 && si_encode_fn() != nullptr;
 }
@@ -518,16 +521,17 @@ SI_EXPORT int si_attn_encode_cache_map(void* map_out, const void* cache, long lo
                            (unsigned)page_size);
 }
 
-SI_EXPORT long long si_attn_decode_tma_scratch_floats(int num_items, int H, int KV, int hs, int nsplit) {
+// Floats of scratch for partial results of value size `vs`.
+SI_EXPORT long long si_attn_decode_tma_scratch_floats(int num_items, int H, int KV, int vs, int nsplit) {
   if (nsplit <= 1) return 0;
   const long long rows = rows_for(H, KV);
-  return SI_ATTN_TICKETS + (long long)num_items * KV * nsplit * rows * (hs + 2);
+  return SI_ATTN_TICKETS + (long long)num_items * KV * nsplit * rows * (vs + 2);
 }
 
 // Scratch of the launch with a work list: the tickets, then `slots` partial results (one per work entry).
-SI_EXPORT long long si_attn_decode_tma_work_floats(int slots, int H, int KV, int hs) {
+SI_EXPORT long long si_attn_decode_tma_work_floats(int slots, int H, int KV, int vs) {
   const long long rows = rows_for(H, KV);
-  return SI_ATTN_TICKETS + (long long)slots * KV * rows * (hs + 2);
+  return SI_ATTN_TICKETS + (long long)slots * KV * rows * (vs + 2);
 }
 
 template <int NH, int MT, bool SWAP = false>
@@ -560,11 +564,11 @@ static int launch(const AttnParams& p, const CUtensorMap& km, const CUtensorMap&
 SI_EXPORT int si_attn_decode_tma(const void* q, long long q_stride, const void* k_cache, const void* v_cache,
                                  const void* kmap, const void* vmap, const int* block_table, int table_width,
                                  const void* items, int num_items, void* out, long long out_stride, int num_pages,
-                                 int page_size, int num_seqs, int H, int KV, int hs, float scale, int window,
+                                 int page_size, int num_seqs, int H, int KV, int hs, int vs, float scale, int window,
                                  int nsplit, const int* work, int num_work, int work_slots, float* scratch,
                                  int max_rows, int chunk, const float* sink, int* status, cudaStream_t stream) {
   if (num_items <= 0) return 0;
-  if (!si_attn_decode_tma_ok(H, KV, hs, page_size) || !kmap || !vmap) return -2;
+  if (!si_attn_decode_tma_ok(H, KV, hs, vs, page_size) || !kmap || !vmap) return -2;
   if (work) {
     if (num_work <= 0 || work_slots <= 0 || !scratch || ((uintptr_t)work % 16)) return -2;
     nsplit = 1;
@@ -578,7 +582,7 @@ SI_EXPORT int si_attn_decode_tma(const void* q, long long q_stride, const void* 
   p.out = (bf16*)out; p.out_stride = out_stride;
   p.part_o = nullptr; p.part_ml = nullptr; p.counters = nullptr;
   p.num_pages = num_pages; p.page_size = page_size; p.num_seqs = num_seqs;
-  p.H = H; p.KV = KV; p.G = H / KV; p.hs = hs;
+  p.H = H; p.KV = KV; p.G = H / KV; p.hs = hs; p.vs = vs;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.window = window; p.chunk = chunk; p.sink = sink; p.nsplit = nsplit; p.status = status;
   const int rows = rows_for(H, KV);
@@ -587,17 +591,18 @@ SI_EXPORT int si_attn_decode_tma(const void* q, long long q_stride, const void* 
     const size_t slots = work ? (size_t)work_slots : (size_t)num_items * nsplit;
     p.counters = reinterpret_cast<int*>(scratch);
     p.part_o = scratch + SI_ATTN_TICKETS;
-    p.part_ml = p.part_o + slots * KV * rows * hs;
+    p.part_ml = p.part_o + slots * KV * rows * vs;
   }
   const int4* wl = reinterpret_cast<const int4*>(work);
   int log2_page = 0;
   while ((1 << log2_page) < page_size) ++log2_page;
   const CUtensorMap& km = *(const CUtensorMap*)kmap;
   const CUtensorMap& vm = *(const CUtensorMap*)vmap;
+  const bool narrow = hs <= 64 && vs <= 64;
   if (rows == 16 && max_rows >= 1 && max_rows <= 8)
-    return hs == 64 ? launch<1, 1, true>(p, km, vm, num_items, log2_page, wl, num_work, stream)
+    return narrow ? launch<1, 1, true>(p, km, vm, num_items, log2_page, wl, num_work, stream)
                     : launch<2, 1, true>(p, km, vm, num_items, log2_page, wl, num_work, stream);
-  if (hs == 64) return rows == 16 ? launch<1, 1>(p, km, vm, num_items, log2_page, wl, num_work, stream)
+  if (narrow) return rows == 16 ? launch<1, 1>(p, km, vm, num_items, log2_page, wl, num_work, stream)
                                   : launch<1, 2>(p, km, vm, num_items, log2_page, wl, num_work, stream);
   return rows == 16 ? launch<2, 1>(p, km, vm, num_items, log2_page, wl, num_work, stream)
                     : launch<2, 2>(p, km, vm, num_items, log2_page, wl, num_work, stream);

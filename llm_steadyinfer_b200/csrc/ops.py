@@ -386,15 +386,16 @@ def attn_decode_scratch_floats(num_items: int, H: int, KV: int, hs: int, nsplit:
     return lib.si_attn_decode_scratch_floats(_c_int(num_items), _c_int(H), _c_int(KV), _c_int(hs), _c_int(nsplit))
 
 
-def _attn_common(q, k_cache, v_cache, block_table, items, out, page_size, H, KV, hs, what):
+def _attn_common(q, k_cache, v_cache, block_table, items, out, page_size, H, KV, hs, what, vs=None):
+    vs = hs if vs is None else vs
     _cuda(q, k_cache, v_cache, block_table, items, out)
     _i32(block_table, "block_table"); _i32(items, "items")
     _need(q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16
           and v_cache.dtype == torch.bfloat16, f"{what}: bfloat16 tensors only")
-    _need(q.stride(1) == 1 and out.stride(1) == 1 and q.shape[1] == H * hs and out.shape[1] == H * hs,
+    _need(q.stride(1) == 1 and out.stride(1) == 1 and q.shape[1] == H * hs and out.shape[1] == H * vs,
           f"{what}: q/out must be [T, H*hs] rows")
-    _need(tuple(k_cache.shape[1:]) == (KV, page_size, hs) and k_cache.is_contiguous() and v_cache.is_contiguous(),
-          f"{what}: cache must be [pages, KV, page_size, hs]")
+    _need(tuple(k_cache.shape[1:]) == (KV, page_size, hs) and k_cache.is_contiguous() and v_cache.is_contiguous()
+          and tuple(v_cache.shape) == (k_cache.shape[0], KV, page_size, vs), f"{what}: cache must be [pages, KV, page_size, hs]")
     _need(items.dim() == 2 and items.shape[1] == 4, f"{what}: items must be int32 [n, 4]")
     _need(q.data_ptr() % 16 == 0 and k_cache.data_ptr() % 16 == 0 and v_cache.data_ptr() % 16 == 0,
           f"{what}: q and cache must be 16-byte aligned")
@@ -452,11 +453,14 @@ def _keep_map(table: dict, key, ent) -> None:
 _tensor_maps = {}
 
 
-def attn_decode_tma_ok(H: int, KV: int, hs: int, page_size: int) -> bool:
-    """True when the TMA decode kernel takes this head layout and page size."""
+def attn_decode_tma_ok(H: int, KV: int, hs: int, page_size: int, vs: Optional[int] = None) -> bool:
+    """True when the TMA decode kernel takes this head layout and page size: heads of 64 or 128, or, for callers that name
+    the value size ``vs``, key and value sizes of any multiple of 8 up to 128 (padded inside the kernel)."""
+    if vs is None and hs not in (64, 128):
+        return False
     lib = build.load("attention_tma")
     lib.si_attn_decode_tma_ok.restype = _c_int
-    return bool(lib.si_attn_decode_tma_ok(_c_int(H), _c_int(KV), _c_int(hs), _c_int(page_size)))
+    return bool(lib.si_attn_decode_tma_ok(_c_int(H), _c_int(KV), _c_int(hs), _c_int(hs if vs is None else vs), _c_int(page_size)))
 
 
 def attn_decode_tma_rows(H: int, KV: int) -> int:
@@ -582,7 +586,7 @@ def attn_decode_tma_work_floats(slots: int, H: int, KV: int, hs: int) -> int:
 
 def attn_decode_tma(q, k_cache, v_cache, block_table, items, out, page_size: int, num_seqs: int, H: int, KV: int,
                     hs: int, scale: float, window: int = 0, nsplit: int = 1, scratch=None, status=None,
-                    max_rows: int = 0, work=None, chunk: int = 0, sink=None) -> None:
+                    max_rows: int = 0, work=None, chunk: int = 0, sink=None, vs: Optional[int] = None) -> None:
     """``attn_decode`` with the K/V tiles fetched by TMA (head_dim 64 or 128, page sizes 8 to 64);
     items hold at most ``attn_decode_tma_rows // (H // KV)`` tokens. ``max_rows``: the most rows
     (tokens x query heads of a KV head) of any item when the caller knows it (0: unknown); at most 8
@@ -590,29 +594,30 @@ def attn_decode_tma(q, k_cache, v_cache, block_table, items, out, page_size: int
     ``work`` (int32 [W, 4], rows of (item, split, splits of that item, first slot of that item); item -1:
     nothing): every item is cut into its own number of shares, ``nsplit`` is not used, and ``scratch``
     holds ``attn_decode_tma_work_floats(W, ...)`` floats. Made by ``split_work``. ``chunk`` and ``sink`` (fp32 [H]) as in
-    ``attention_general``."""
-    _attn_common(q, k_cache, v_cache, block_table, items, out, page_size, H, KV, hs, "attn_decode_tma")
+    ``attention_general``. ``vs``: size of the values where it is not the keys' (scratch is counted in it)."""
+    vs = hs if vs is None else vs
+    _attn_common(q, k_cache, v_cache, block_table, items, out, page_size, H, KV, hs, "attn_decode_tma", vs)
     _cuda(sink)
     _f32v(sink, "sink", H)
     if work is not None:
         _cuda(work, scratch)
         _need(work.dtype == torch.int32 and work.dim() == 2 and work.shape[1] == 4 and work.is_contiguous(),
               "attn_decode_tma: work must be int32 [W, 4]")
-        need = attn_decode_tma_work_floats(work.shape[0], H, KV, hs)
+        need = attn_decode_tma_work_floats(work.shape[0], H, KV, vs)
         _need(scratch is not None and scratch.dtype == torch.float32 and scratch.numel() >= need,
               f"attn_decode_tma: scratch must hold {need} floats")
     elif nsplit > 1:
         _cuda(scratch)
-        need = attn_decode_tma_scratch_floats(items.shape[0], H, KV, hs, nsplit)
+        need = attn_decode_tma_scratch_floats(items.shape[0], H, KV, vs, nsplit)
         _need(scratch is not None and scratch.dtype == torch.float32 and scratch.numel() >= need,
               f"attn_decode_tma: scratch must hold {need} floats")
     f = _fn("attention_tma", "si_attn_decode_tma",
             [_c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_int, _c_p, _c_ll, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_f, _c_int, _c_int, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_p, _c_p, _c_p])
+             _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_int, _c_p, _c_int, _c_int, _c_p, _c_int, _c_int, _c_p, _c_p, _c_p])
     W = work.shape[0] if work is not None else 0
     _check(f(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _cache_map(k_cache), _cache_map(v_cache),
              _ptr(block_table), block_table.shape[1], _ptr(items), items.shape[0], _ptr(out), out.stride(0),
-             k_cache.shape[0], page_size, num_seqs, H, KV, hs, float(scale), int(window or 0), int(nsplit),
+             k_cache.shape[0], page_size, num_seqs, H, KV, hs, vs, float(scale), int(window or 0), int(nsplit),
              _ptr(work), W, W, _ptr(scratch), int(max_rows), int(chunk or 0), _ptr(sink), _ptr(status), _stream()),
            f"attn_decode_tma(heads={H}, kv_heads={KV}, head_dim={hs}, page_size={page_size})")
 
@@ -889,10 +894,13 @@ def gemm_rows_swiglu(a, w, out, status=None) -> None:
 
 # ---- prompt-portion attention on tcgen05 ---------------------------------------------------------
 
-def attn_portion_tc05_ok(H: int, KV: int, hs: int, page_size: int) -> bool:
+def attn_portion_tc05_ok(H: int, KV: int, hs: int, page_size: int, vs: Optional[int] = None) -> bool:
+    """As ``attn_decode_tma_ok``, for the tcgen05 prompt kernel."""
+    if vs is None and hs not in (64, 128):
+        return False
     lib = build.load("attention_tc05")
     lib.si_attn_portion_tc05_ok.restype = _c_int
-    return bool(lib.si_attn_portion_tc05_ok(_c_int(H), _c_int(KV), _c_int(hs), _c_int(page_size)))
+    return bool(lib.si_attn_portion_tc05_ok(_c_int(H), _c_int(KV), _c_int(hs), _c_int(hs if vs is None else vs), _c_int(page_size)))
 
 
 def attn_portion_tc05_tokens(H: int, KV: int) -> int:
@@ -904,14 +912,15 @@ def attn_portion_tc05_tokens(H: int, KV: int) -> int:
 
 def attn_portion_tc05(q, k_cache, v_cache, block_table, items, out, page_size: int, num_seqs: int, H: int,
                       KV: int, hs: int, scale: float, window: int = 0, status=None, slopes=None, q_temp=None, gate=None,
-                      chunk: int = 0, sink=None) -> None:
+                      chunk: int = 0, sink=None, vs: Optional[int] = None) -> None:
     """``attn_portion`` on the tcgen05 tensor cores (TMA-fed K/V tiles, S and P V in tensor memory);
     head_dim 64 or 128, page sizes 8 to 64, items of at most ``attn_portion_tc05_tokens`` tokens. ``v_cache`` None: the
     values are the keys. ``slopes``, ``q_temp`` (a coefficient that is not negative), ``gate``, ``chunk`` and ``sink`` as in
-    ``attention_general`` (the gate's rows 16-byte aligned)."""
+    ``attention_general`` (the gate's rows 16-byte aligned). ``vs``: size of the values where it is not the keys'."""
     if v_cache is None:
         v_cache = k_cache
-    _attn_common(q, k_cache, v_cache, block_table, items, out, page_size, H, KV, hs, "attn_portion_tc05")
+    vs = hs if vs is None else vs
+    _attn_common(q, k_cache, v_cache, block_table, items, out, page_size, H, KV, hs, "attn_portion_tc05", vs)
     _cuda(slopes, gate, sink)
     _f32v(slopes, "slopes", H)
     _f32v(sink, "sink", H)
@@ -921,10 +930,10 @@ def attn_portion_tc05(q, k_cache, v_cache, block_table, items, out, page_size: i
                            and gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0), "attn_portion_tc05: gate must be bf16 [T, H*hs], rows 16-byte aligned")
     f = _fn("attention_tc05", "si_attn_portion_tc05",
             [_c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_int, _c_p, _c_ll, _c_int, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_f, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_p])
+             _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_p, _c_f, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_p])
     _check(f(_ptr(q), q.stride(0), _ptr(k_cache), _ptr(v_cache), _cache_map(k_cache), _cache_map(v_cache),
              _ptr(block_table), block_table.shape[1], _ptr(items), items.shape[0], _ptr(out), out.stride(0),
-             k_cache.shape[0], page_size, num_seqs, H, KV, hs, float(scale), int(window or 0), _ptr(slopes), qt_coef, qt_every,
+             k_cache.shape[0], page_size, num_seqs, H, KV, hs, vs, float(scale), int(window or 0), _ptr(slopes), qt_coef, qt_every,
              _ptr(gate), gate.stride(0) if gate is not None else 0, int(chunk or 0), _ptr(sink), _ptr(status),
              _stream()), f"attn_portion_tc05(heads={H}, kv_heads={KV}, head_dim={hs}, page_size={page_size})")
 

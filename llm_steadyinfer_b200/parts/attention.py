@@ -36,7 +36,7 @@ Options beyond the reference's block, all parameters of the part:
                    ``cache_from``), whose keys lie there as that layer stored them.
 With any option but ``names`` the mixer runs its general form. Biases, convolution and norm are one launch behind the stacked
 projection (``qkv_conv.cu``), which also stores keys and values. The attention itself: where scores are plain but for the sink
-and the chunk and the layout is one that the fast kernels take (key size 64 or 128, values of the same size), decode rows go to
+and the chunk and the sizes are ones that the fast kernels take (multiples of 8 up to 128), decode rows go to
 ``attention_tma.cu`` and prompt portions to ``attention_tc05.cu`` as in the reference's block; else the general kernels
 (``attention_general.cu`` in 32-bit, ``attention_flex.cu`` on the tensor cores in bfloat16). Sequences that bring a full work item of
 rows to a bfloat16 step go to the tcgen05 prompt kernel (``attention_tc05.cu``) where its layout fits (key size 64 or 128,
@@ -114,9 +114,9 @@ class Attention(Mixer):
         self.own_keys = bool(params.get("own_keys", True))
         self.prepared = self.biases or self.has_conv or self.qk_norm or not self.own_keys     # a launch behind the projection
         # scores that the fast kernels know: q . k times the scale, a window or chunks, a sink
-        self.plain_scores = (self.bias_spec is None and self.vs == self.hs and self.own_v and self.slopes is None
-                             and self.q_temp is None and self.gate_name is None)
-        self.general = not self.plain_scores or self.prepared or self.chunk is not None or self.sink is not None
+        self.plain_scores = (self.bias_spec is None and self.own_v and self.slopes is None and self.q_temp is None
+                             and self.gate_name is None)
+        self.general = not self.plain_scores or self.vs != self.hs or self.prepared or self.chunk is not None or self.sink is not None
         if self.hs > (1024 if self.general else 256) or self.vs > 1024:
             raise ValueError(f"attention: head_dim {self.hs} is not supported (at most 256, 1,024 in the general form)")
         if self.taps < 1:
@@ -356,13 +356,17 @@ class Attention(Mixer):
     def uses_fast(self, page_size: int) -> bool:
         """The general form whose scores the fast kernels know (the TMA-fed decode kernel, the tcgen05 prompt kernel)."""
         return (self.general and self.plain_scores and self.dtype == torch.bfloat16 and USE_TENSOR_CORES and USE_TMA and USE_TC05
-                and self.hs in (64, 128) and page_size in (8, 16, 32, 64) and self.H // self.KV <= 32
-                and ops.attn_decode_tma_ok(self.H, self.KV, self.hs, page_size)
-                and ops.attn_portion_tc05_ok(self.H, self.KV, self.hs, page_size))
+                and max(self.hs, self.vs) <= 128 and self.hs % 8 == 0 and self.vs % 8 == 0 and page_size in (8, 16, 32, 64)
+                and self.H // self.KV <= 32 and ops.attn_decode_tma_ok(self.H, self.KV, self.hs, page_size, self.vs)
+                and ops.attn_portion_tc05_ok(self.H, self.KV, self.hs, page_size, self.vs))
+
+    def _plan_key(self) -> tuple:
+        return ("attention", self.H, self.KV, self.hs, self.vs, self.window, self.chunk)
 
     def _tag(self) -> str:
         """Names the buffers of a plan: what layers that share it have in common."""
-        return f"{self.H}_{self.KV}_{self.hs}_{self.window}" + (f"_c{self.chunk}" if self.chunk else "")
+        return f"{self.H}_{self.KV}_{self.hs}_{self.window}" + (f"_v{self.vs}" if self.vs != self.hs else "") \
+            + (f"_c{self.chunk}" if self.chunk else "")
 
     def uses_tensor_cores(self) -> bool:
         return not self.general and self.dtype == torch.bfloat16 and USE_TENSOR_CORES and self.hs % 16 == 0
@@ -380,14 +384,15 @@ class Attention(Mixer):
             return
         if not self.general and not self.uses_tensor_cores():
             return
-        key = ("attention", self.H, self.KV, self.hs, self.window, self.chunk)
+        key = self._plan_key()
         if key in ctx.plans or cache.k is None:
             return
         G = self.H // self.KV
-        tma = USE_TMA and ops.attn_decode_tma_ok(self.H, self.KV, self.hs, cache.page_size)
+        sizes = (self.H, self.KV, self.hs, cache.page_size) + ((self.vs,) if self.general else ())
+        tma = USE_TMA and ops.attn_decode_tma_ok(*sizes)
         dec_rows = ops.attn_decode_tma_rows(self.H, self.KV) if tma else ops.attn_decode_rows(self.H, self.KV, self.hs)
         dec_tokens = dec_rows // G
-        tc05 = USE_TC05 and ops.attn_portion_tc05_ok(self.H, self.KV, self.hs, cache.page_size)
+        tc05 = USE_TC05 and ops.attn_portion_tc05_ok(*sizes)
         por_tokens = (ops.attn_portion_tc05_tokens(self.H, self.KV) if tc05
                       else ops.attn_portion_tokens(self.H, self.KV, self.hs))
         if por_tokens <= 0:
@@ -427,7 +432,7 @@ class Attention(Mixer):
                                    np.concatenate([np.asarray(dec, dtype=np.int32).reshape(-1), work.reshape(-1)]))
             plan["dec"] = both[:4 * len(dec)].view(-1, 4)
             plan["work"] = both[4 * len(dec):].view(-1, 4)
-            plan["scratch"] = ctx.buf("attn_split", (ops.attn_decode_tma_work_floats(entries, self.H, self.KV, self.hs),),
+            plan["scratch"] = ctx.buf("attn_split", (ops.attn_decode_tma_work_floats(entries, self.H, self.KV, self.vs),),
                                       torch.float32)
         elif dec:
             # as many blocks as run at once (two per SM), not more: a second wave would wait
@@ -452,9 +457,9 @@ class Attention(Mixer):
                                     out, cache.page_size, ctx.seq_slots, self.H, self.KV, self.hs,
                                     self.scale, self.window or 0, status=ctx.status)
             return
-        plan = ctx.plans[("attention", self.H, self.KV, self.hs, self.window, self.chunk)]
+        plan = ctx.plans[self._plan_key()]
         # the fast kernels take chunks and a sink; a layout that has neither may run the others
-        extra = {"chunk": self.chunk, "sink": self.sink} if self.general else {}
+        extra = {"chunk": self.chunk, "sink": self.sink, "vs": self.vs} if self.general else {}
         args = (cache.page_size, ctx.seq_slots, self.H, self.KV, self.hs, self.scale, self.window or 0)
         if plan["dec"] is not None:
             if plan["tma"]:

@@ -294,7 +294,8 @@ def _paged(rows, page_size, perm_seed):
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
 @pytest.mark.parametrize("H,G,dk,dv,chunk,sink", [(4, 2, 24, 16, 37, 0.0), (8, 2, 48, 72, 100, 0.0), (3, 1, 10, 6, 64, 1.5), (6, 6, 16, 8, 1, 0.0),
                                                   (4, 2, 64, 64, 50, 0.0), (8, 2, 128, 128, 129, 0.0), (4, 1, 128, 128, None, 6.0),
-                                                  (16, 1, 64, 64, 96, 0.0), (2, 2, 64, 64, 16, 0.7), (24, 1, 64, 64, 70, 0.0)])
+                                                  (16, 1, 64, 64, 96, 0.0), (2, 2, 64, 64, 16, 0.7), (24, 1, 64, 64, 70, 0.0),
+                                                  (4, 2, 104, 64, 60, 0.0), (6, 2, 56, 120, 45, 0.0), (4, 4, 8, 8, 20, 0.0)])
 def test_attention_with_chunks_and_sink(H, G, dk, dv, chunk, sink, dtype):
     """Queries built so that one key would carry nearly all of a head's weight: the last key before the row's chunk (must
     not count), the chunk's first key from its last rows, keys at page borders, the row's own key; the other rows' scores are
@@ -363,25 +364,25 @@ def test_attention_with_chunks_and_sink(H, G, dk, dv, chunk, sink, dtype):
         ops.attn_flex(qd[n - last:], kc, vc, table, singles(), one, ps, 1, H, G, dk, dv, scale, sink=sd, chunk=cd, nsplit=nsplit,
                       scratch=scratch, max_rows=ratio)
         compare(one, want[n - last:], f"mma.sync, single rows in {nsplit} shares")
-    if dk == dv and ops.attn_portion_tc05_ok(H, G, dk, ps):
+    if ops.attn_portion_tc05_ok(H, G, dk, ps, dv):
         status = torch.zeros(1, dtype=torch.int32, device=DEV)
         per = ops.attn_portion_tc05_tokens(H, G)
         items = torch.tensor([(0, b, min(per, n - b), b) for b in range(0, n, per)], dtype=torch.int32, device=DEV)
         out.zero_()
-        ops.attn_portion_tc05(qd, kc, vc, table, items, out, ps, 1, H, G, dk, scale, status=status, chunk=cd, sink=sd)
+        ops.attn_portion_tc05(qd, kc, vc, table, items, out, ps, 1, H, G, dk, scale, status=status, chunk=cd, sink=sd, vs=dv)
         assert status.item() == 0
         compare(out, want, "tcgen05, prompt rows")
-        if ops.attn_decode_tma_ok(H, G, dk, ps):
+        if ops.attn_decode_tma_ok(H, G, dk, ps, dv):
             for nsplit in (1, 3):
                 one = torch.zeros(last, H * dv, dtype=dtype, device=DEV)
-                scratch = torch.zeros(max(1, ops.attn_decode_tma_scratch_floats(last, H, G, dk, nsplit)), dtype=torch.float32, device=DEV)
+                scratch = torch.zeros(max(1, ops.attn_decode_tma_scratch_floats(last, H, G, dv, nsplit)), dtype=torch.float32, device=DEV)
                 ops.attn_decode_tma(qd[n - last:], kc, vc, table, singles(), one, ps, 1, H, G, dk, scale, nsplit=nsplit, scratch=scratch,
-                                    status=status, max_rows=ratio, chunk=cd, sink=sd)
+                                    status=status, max_rows=ratio, chunk=cd, sink=sd, vs=dv)
                 compare(one, want[n - last:], f"TMA decode, single rows in {nsplit} shares")
             few = ops.attn_decode_tma_rows(H, G) // ratio          # items of several tokens, some over a chunk's edge
             items = torch.tensor([(0, b, min(few, last - b), n - last + b) for b in range(0, last, few)], dtype=torch.int32, device=DEV)
             one = torch.zeros(last, H * dv, dtype=dtype, device=DEV)
-            ops.attn_decode_tma(qd[n - last:], kc, vc, table, items, one, ps, 1, H, G, dk, scale, status=status, chunk=cd, sink=sd)
+            ops.attn_decode_tma(qd[n - last:], kc, vc, table, items, one, ps, 1, H, G, dk, scale, status=status, chunk=cd, sink=sd, vs=dv)
             compare(one, want[n - last:], "TMA decode, several rows an item")
             assert status.item() == 0
 
