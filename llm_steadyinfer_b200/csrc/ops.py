@@ -1789,7 +1789,7 @@ def qkv_conv(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, 
              k_weight=None, portions: int = 3, status=None) -> None:
     """Rows ``u`` = [q: NQ*dk | k: NK*dk | v: NV*dv | ...] of a stacked projection, plus ``bias`` (fp32 [C] or None), through a
     causal convolution over time per channel (``taps`` fp32 [K, C]; zeros before the sequence), then with ``norm`` every q and
-    k vector divided by its root mean square (times ``q_weight`` / ``k_weight``, fp32 [dk], where given); q into ``q_out``
+    k vector scaled to a root mean square of one (times ``q_weight`` / ``k_weight``, fp32 [dk], where given); q into ``q_out``
     [T, NQ*dk], k and v into their pages (``k_cache`` None: the queries alone are kept). ``state`` (fp32 [slots, >= (K-1)*C];
     None for K = 1) holds each request's last K - 1 values of every channel and is renewed. ``portions``: what the step
     holds beside sequences of one row: 1 portions of several rows from position 0, 2 such portions from a later position (a second

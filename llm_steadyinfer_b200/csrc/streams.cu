@@ -222,9 +222,10 @@ static int stream_launch(StreamArgs p, cudaStream_t stream) {
   const int pieces = p.width / 4, max_v = p.S > 4 ? 2 : 4, sms = si_sm_count();
   bool vec = p.S <= 8 && p.width % 4 == 0 && p.src_row % 4 == 0 && p.src_stream % 4 == 0 && al(p.src, 16) && al(p.dst, 16) &&
              al(p.y, 4 * sizeof(T)) && al(p.out, 4 * sizeof(T)) && al(p.weight, p.weight_bf16 ? 8 : 16);
-  // Blocks that share a row: while the rows alone leave most of the device idle and a part still fills a block of 128.
+  // Blocks that share a row of 2,048 columns or more, while the rows alone leave most of the device idle (measured: shorter
+  // rows are done sooner by one block than the cluster's two barriers take)
   int parts = 1;
-  while (parts < 8 && (long long)p.num_rows * parts * 2 <= sms && pieces / (parts * 2) >= 64) parts *= 2;
+  while (pieces >= 512 && parts < 8 && (long long)p.num_rows * parts * 2 <= sms && pieces / (parts * 2) >= 64) parts *= 2;
   int per = (pieces + parts - 1) / parts;
   while (parts < 8 && per > max_v * 512) { parts *= 2; per = (pieces + parts - 1) / parts; }
   if (per > max_v * 512) vec = false;

@@ -1,6 +1,6 @@
 """Risizen: a decoder whose residual stream has several copies ("streams") with learned connections between them and every
 sublayer. config.json lists the layers one by one: a grouped-query attention mixer without rotation (projections with
-biases, a short causal convolution on every channel of q, k and v, queries and keys divided by their root mean square,
+biases, a short causal convolution on every channel of q, k and v, queries and keys scaled to a root mean square of one,
 positions in chunks that see only themselves, a sink whose score is 0 in the softmax denominator), some layers of which read
 the keys and values of an earlier one, and a gated feed-forward with limits. The embedding's output is normalised and the
 logits are scaled.

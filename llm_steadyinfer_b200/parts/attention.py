@@ -29,7 +29,7 @@ Options beyond the reference's block, all parameters of the part:
 ``conv_taps``      K: every channel of q, k and v passes a causal convolution over time of K taps (tensor names: the matrix's +
                    ``conv_suffix``, [channels, K], the last tap the current token's); the last K - 1 projected values of a request
                    are its state.
-``qk_norm``        ``{"eps": e}``: every query and key head is divided by its root mean square (after the convolution).
+``qk_norm``        ``{"eps": e}``: every query and key head is scaled to a root mean square of one (after the convolution).
 ``sink_score``     a number s: exp(s) joins every row's softmax denominator once, without a value.
 ``chunk``          positions fall into runs of so many, counted from position 0; a query sees keys of its own run alone.
 ``own_keys``       False: the layer has no key and value projections and reads the cache of another one (its spec's

@@ -463,7 +463,7 @@ def test_convolution_norm_and_store(NQ, NK, NV, dk, dv, K, norm, bias, times, dt
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
 @pytest.mark.parametrize("T,S,d", [(1, 4, 4096), (3, 2, 256), (17, 3, 1000), (300, 4, 2048), (5, 1, 64), (9, 5, 96), (4, 8, 520), (6, 9, 70), (2, 2, 33),
-                                   (700, 2, 136), (2, 3, 20000)])
+                                   (700, 2, 136), (2, 3, 20000), (3, 2, 2052), (2, 7, 4100), (40, 4, 2048)])
 def test_streams_written_read_and_normalised(T, S, d, dtype):
     """x' = mix^T x + write y, u = read . x', the norm of u: in place, from one row that stands for all streams, without a
     result to write (the first sublayer), for chosen rows and the plain sum (the end of the model)."""
