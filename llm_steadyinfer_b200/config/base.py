@@ -101,6 +101,7 @@ class LayerSpec:
     # connections to a stream of several copies (arrangement "streams"): tensor prefixes below weight_prefix
     mixer_streams_prefix: Optional[str] = None
     feed_forward_streams_prefix: Optional[str] = None
+    token_side_prefix: Optional[str] = None      # tensor prefix of the layer's own input for each token (``ModelSpec.token_side``)
     residual_scale: float = 1.0                  # what a block adds to the stream is multiplied by it
 
 
@@ -114,6 +115,15 @@ class StreamAddSpec:
     embedding: bool = False
     vector_name: Optional[str] = None
     row: int = 0
+
+
+@dataclass(frozen=True)
+class TokenSideSpec:
+    """A second embedding table whose columns are shared out among the layers (``TokenSideInput``): layer i's input for a token is the part
+    [i * dim, (i + 1) * dim) of the token's row of ``table_name`` ([vocab, layers * dim])."""
+    dim: int
+    eps: float
+    table_name: str = "side.embed"
 
 
 @dataclass(frozen=True)
@@ -132,6 +142,7 @@ class ModelSpec:
     stream_adds: tuple = ()                      # StreamAddSpec entries, at most one a place
     stream_vector_shapes: Optional[Dict[str, tuple]] = None   # the tensors that ``stream_adds`` name: name -> shape
     streams: Optional[int] = None                # copies of the residual stream (arrangement "streams"); None: the one stream
+    token_side: Optional[TokenSideSpec] = None   # layers with a ``token_side_prefix`` have an input of their own for each token
     logit_scale: float = 1.0                     # logits are multiplied by it (before the soft cap)
     logit_softcap: float = 0.0                   # > 0: logits <- cap * tanh(logits / cap)
 

@@ -17,6 +17,10 @@
 // the warps do not wait for one another.
 // A request's state lies at the start of its slot, head by head, each head as [RPT][dv][NP] (see delta_shape); a
 // portion that begins at position 0 starts from zero whatever the slot held.
+//
+// With a decay per key channel (a factor for every row of S) the same recurrence runs in `channel_delta_scan`: S <- diag(g_t) S
+// first, then the sums over the decayed state, four packed operations for two rows as before. `channel_delta_prepare` makes
+// the decays, beta and q . k; q and k arrive as unit vectors.
 #include "common.cuh"
 #include <math.h>
 
@@ -271,14 +275,276 @@ SI_EXPORT int si_delta_scan(const float* xc, long long xc_stride, const float* b
   return si_last_error();
 }
 
+// ---- a decay per key channel -----------------------------------------------------------------------------------------
+// dec [T, H * dk] fp32 holds raw values x and receives g = exp(-exp(A_log_h) * softplus(x + dt_bias)) in place; ba: rows with H raw
+// values b at b_off in the compute dtype; bg fp32 [T, H + G]: beta = sigmoid(b), then q . k of the (unit) vectors per query/key
+// head, which lie in xc as [q: G * dk | k: G * dk | ...]. A warp takes a (row, head) or a (row, query/key head).
+template <typename T>
+__global__ void __launch_bounds__(256) channel_delta_prepare_kernel(const float* __restrict__ xc, long long xc_stride,
+    const T* __restrict__ ba, long long ba_stride, int b_off, float* __restrict__ dec, long long dec_stride,
+    const float* __restrict__ a_log, const float* __restrict__ dt_bias, float* __restrict__ bg, long long units, int G, int H, int dk,
+    int wide) {
+  pdl_prologue();
+  const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (unit >= units) return;
+  const int lane = threadIdx.x & 31;
+  const long long t = unit / (H + G);
+  const int h = (int)(unit - t * (H + G));
+  float* bgr = bg + t * (H + G);
+  if (h >= H) {
+    const float* q = xc + t * xc_stride + (size_t)(h - H) * dk;
+    const float* k = q + (size_t)G * dk;
+    float dot = 0.f;
+    if (wide) {
+      for (int i = lane * 4; i < dk; i += 128) {
+        const float4 a = *reinterpret_cast<const float4*>(q + i), b = *reinterpret_cast<const float4*>(k + i);
+        dot = fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, dot))));
+      }
+    } else {
+      for (int i = lane; i < dk; i += 32) dot = fmaf(q[i], k[i], dot);
+    }
+    dot = warp_sum(dot);
+    if (lane == 0) bgr[h] = dot;
+    return;
+  }
+  const float rate = expf(a_log[h]);
+  float* d = dec + t * dec_stride + (size_t)h * dk;
+  const float* bias = dt_bias + (size_t)h * dk;
+  auto decay = [&](float x, float b) { return expf(-rate * softplus_d(x + b)); };
+  if (wide) {
+    for (int i = lane * 4; i < dk; i += 128) {
+      const float4 x = *reinterpret_cast<const float4*>(d + i), b = *reinterpret_cast<const float4*>(bias + i);
+      *reinterpret_cast<float4*>(d + i) = make_float4(decay(x.x, b.x), decay(x.y, b.y), decay(x.z, b.z), decay(x.w, b.w));
+    }
+  } else {
+    for (int i = lane; i < dk; i += 32) d[i] = decay(d[i], bias[i]);
+  }
+  if (lane == 0) bgr[h] = 1.f / (1.f + expf(-to_f32<T>(ba[t * ba_stride + b_off + h])));
+}
+
+SI_EXPORT int si_channel_delta_prepare(const float* xc, long long xc_stride, const void* ba, int dtype, long long ba_stride, int b_off,
+                                       float* dec, long long dec_stride, const float* a_log, const float* dt_bias, float* bg,
+                                       int num_tokens, int G, int H, int dk, cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  if (G <= 0 || H <= 0 || dk <= 0) return -2;
+  const uintptr_t all = (uintptr_t)xc | (uintptr_t)dec | (uintptr_t)dt_bias;
+  const int wide = dk % 4 == 0 && xc_stride % 4 == 0 && dec_stride % 4 == 0 && (all & 15) == 0;
+  const long long units = (long long)num_tokens * (H + G);
+  const dim3 grid((unsigned)((units + 7) / 8)), block(256);
+  if (dtype == SI_BF16)
+    si_launch(channel_delta_prepare_kernel<__nv_bfloat16>, grid, block, 0, stream, xc, xc_stride, (const __nv_bfloat16*)ba, ba_stride,
+              b_off, dec, dec_stride, a_log, dt_bias, bg, units, G, H, dk, wide);
+  else
+    si_launch(channel_delta_prepare_kernel<float>, grid, block, 0, stream, xc, xc_stride, (const float*)ba, ba_stride, b_off, dec,
+              dec_stride, a_log, dt_bias, bg, units, G, H, dk, wide);
+  return si_last_error();
+}
+
+// The scan. Threads, shapes and the state's layout as in delta_scan_kernel. Shared memory: two buffers of `chunk` tokens of
+// [q: RPT * NP | k: RPT * NP | decay: RPT * NP | v: cols | beta, q . k, -, -] (rows beyond dk stay zero).
+#define CHANNEL_SLOTS 4
+template <int RPT, int NP>
+__global__ void __launch_bounds__(256, RPT <= 8 ? 2 : 1) channel_delta_scan_kernel(const float* __restrict__ xc, long long xc_stride,
+    const float* __restrict__ dec, long long dec_stride, const float* __restrict__ bg, float* __restrict__ state,
+    long long state_stride, float* __restrict__ y, long long y_stride, const int* __restrict__ q_start,
+    const int* __restrict__ ctx_len, const int* __restrict__ slots, int G, int H, int dk, int dv, int cols, int chunk) {
+  extern __shared__ __align__(16) float sm[];
+  pdl_prologue();
+  const int s = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * cols;
+  const int row0 = q_start[s], n = q_start[s + 1] - row0;
+  if (n <= 0) return;
+  const int pos0 = ctx_len[s] - n;
+  const int g = h / (H / G);
+  const int p = threadIdx.x % NP, jl = threadIdx.x / NP;
+  const int j = j0 + jl;
+  const bool col_ok = jl < cols && j < dv;
+  float* S = state + (size_t)slots[s] * state_stride + (size_t)h * RPT * NP * dv + (size_t)(col_ok ? j : 0) * NP + p;
+  const size_t s_step = (size_t)dv * NP;
+  float2 st[RPT / 2];
+#pragma unroll
+  for (int r = 0; r < RPT / 2; ++r) {
+    st[r].x = (col_ok && pos0 > 0) ? S[(size_t)(2 * r) * s_step] : 0.f;
+    st[r].y = (col_ok && pos0 > 0) ? S[(size_t)(2 * r + 1) * s_step] : 0.f;
+  }
+  const int dkp = RPT * NP;
+  const int per_tok = 3 * dkp + ((cols + 3) & ~3) + 4;
+  const int used = min(chunk, n) * per_tok;               // what of a buffer this launch's tokens reach
+  for (int idx = threadIdx.x; idx < 2 * used; idx += blockDim.x) sm[idx < used ? idx : chunk * per_tok + idx - used] = 0.f;
+  __syncthreads();
+  const size_t q_off = (size_t)g * dk, k_off = (size_t)(G + g) * dk, v_off = (size_t)2 * G * dk + (size_t)h * dv + j0, d_off = (size_t)h * dk;
+  const int bg_width = H + G;
+  const bool wide = dk % 4 == 0 && xc_stride % 4 == 0 && dec_stride % 4 == 0 && (((uintptr_t)xc | (uintptr_t)dec) & 15) == 0;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  // Where rows are aligned and a token is at most 32 * CHANNEL_SLOTS pieces of 16 bytes, every lane knows its pieces once and
+  // for all: where they lie in a row of xc or dec and where they go in a token's shared memory.
+  const int pr = dk / 4, pieces = 3 * pr + cols / 4;
+  const bool quick = wide && cols % 4 == 0 && j0 + cols <= dv && dv % 4 == 0 && pieces <= 32 * CHANNEL_SLOTS;
+  int src_off[CHANNEL_SLOTS], dst_off[CHANNEL_SLOTS];     // source of a decay piece: ~offset
+#pragma unroll
+  for (int q = 0; q < CHANNEL_SLOTS; ++q) {
+    const int idx = lane + 32 * q;
+    src_off[q] = 0;
+    dst_off[q] = -1;
+    if (quick && idx < 3 * pr) {
+      const int part = idx / pr, i = (idx - part * pr) * 4;
+      src_off[q] = part == 2 ? ~(int)(d_off + i) : (int)(part == 0 ? q_off : k_off) + i;
+      dst_off[q] = part * dkp + i;
+    } else if (quick && idx < pieces) {
+      const int e = (idx - 3 * pr) * 4;
+      src_off[q] = (int)v_off + e;
+      dst_off[q] = 3 * dkp + e;
+    }
+  }
+  auto fetch = [&](int c0, int buf) {                     // a token a warp
+    const int cn = min(chunk, n - c0);
+    for (int tt = warp; tt < cn; tt += nwarps) {
+      float* dst = sm + ((size_t)buf * chunk + tt) * per_tok;
+      const size_t t = (size_t)(row0 + c0 + tt);
+      const float* row = xc + t * xc_stride;
+      const float* drow = dec + t * dec_stride;
+      if (quick) {
+#pragma unroll
+        for (int q = 0; q < CHANNEL_SLOTS; ++q)
+          if (dst_off[q] >= 0) delta_cp16(dst + dst_off[q], src_off[q] < 0 ? drow + ~src_off[q] : row + src_off[q]);
+      } else {
+        const int unit = wide ? 4 : 1;
+#pragma unroll
+        for (int part = 0; part < 3; ++part) {
+          const float* src = part == 0 ? row + q_off : part == 1 ? row + k_off : drow + d_off;
+          for (int i = lane * unit; i < dk; i += 32 * unit) {
+            if (wide) delta_cp16(dst + part * dkp + i, src + i);
+            else delta_cp4(dst + part * dkp + i, src + i);
+          }
+        }
+        for (int e = lane; e < cols; e += 32)
+          if (j0 + e < dv) delta_cp4(dst + 3 * dkp + e, row + v_off + e);
+      }
+      if (lane < 2) delta_cp4(dst + per_tok - 4 + lane, bg + t * bg_width + (lane == 0 ? h : H + g));
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
+  };
+  fetch(0, 0);
+  int buf = 0;
+  for (int c0 = 0; c0 < n; c0 += chunk, buf ^= 1) {
+    const int cn = min(chunk, n - c0);
+    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    __syncthreads();                                      // this chunk has arrived, and everyone is done with the other buffer
+    if (c0 + chunk < n) fetch(c0 + chunk, buf ^ 1);
+    const float* tok = sm + (size_t)buf * chunk * per_tok;
+    float* yp = y + (size_t)(row0 + c0) * y_stride + (size_t)h * dv + j;
+#pragma unroll 2
+    for (int tt = 0; tt < cn; ++tt, tok += per_tok, yp += y_stride) {
+      const float4* q4 = reinterpret_cast<const float4*>(tok) + p;
+      const float4* k4 = reinterpret_cast<const float4*>(tok + dkp) + p;
+      const float4* g4 = reinterpret_cast<const float4*>(tok + 2 * dkp) + p;
+      float2 kk[RPT / 2];
+      float2 sk0 = make_float2(0.f, 0.f), sq0 = sk0;
+#pragma unroll
+      for (int c = 0; c < RPT / 4; ++c) {
+        const float4 kv = k4[c * NP], qv = q4[c * NP], gv = g4[c * NP];
+        kk[2 * c] = make_float2(kv.x, kv.y);
+        kk[2 * c + 1] = make_float2(kv.z, kv.w);
+        st[2 * c] = __fmul2_rn(make_float2(gv.x, gv.y), st[2 * c]);
+        st[2 * c + 1] = __fmul2_rn(make_float2(gv.z, gv.w), st[2 * c + 1]);
+        sk0 = __ffma2_rn(kk[2 * c], st[2 * c], sk0);
+        sq0 = __ffma2_rn(make_float2(qv.x, qv.y), st[2 * c], sq0);
+        sk0 = __ffma2_rn(kk[2 * c + 1], st[2 * c + 1], sk0);
+        sq0 = __ffma2_rn(make_float2(qv.z, qv.w), st[2 * c + 1], sq0);
+      }
+      float sk = sk0.x + sk0.y, sq = sq0.x + sq0.y;
+#pragma unroll
+      for (int o = 1; o < NP; o <<= 1) {
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      }
+      const float2 sc = *reinterpret_cast<const float2*>(tok + per_tok - 4);      // beta, q . k
+      const float vj = col_ok ? tok[3 * dkp + jl] : 0.f;
+      const float u = sc.x * (vj - sk);
+      const float2 u2 = make_float2(u, u);
+#pragma unroll
+      for (int r = 0; r < RPT / 2; ++r) st[r] = __ffma2_rn(kk[r], u2, st[r]);
+      if (p == 0 && col_ok) *yp = fmaf(sc.y, u, sq);
+    }
+  }
+  if (col_ok) {
+#pragma unroll
+    for (int r = 0; r < RPT / 2; ++r) {
+      S[(size_t)(2 * r) * s_step] = st[r].x;
+      S[(size_t)(2 * r + 1) * s_step] = st[r].y;
+    }
+  }
+}
+
+SI_EXPORT int si_channel_delta_scan(const float* xc, long long xc_stride, const float* dec, long long dec_stride, const float* bg,
+                                    float* state, long long state_stride, float* y, long long y_stride, const int* q_start,
+                                    const int* ctx_len, const int* slots, int num_seqs, int G, int H, int dk, int dv,
+                                    cudaStream_t stream) {
+  if (num_seqs <= 0) return 0;
+  if (G <= 0 || H % G || dk <= 0 || dv <= 0 || dk > 512 || H > 65535) return -2;
+  if (2LL * G * dk + (long long)H * dv >= (1LL << 30) || (long long)H * dk >= (1LL << 30)) return -2;
+  const DeltaShape sh = delta_shape(dk);
+  if (sh.rpt * sh.np < dk || state_stride < (long long)H * sh.rpt * sh.np * dv) return -2;
+  int cols = 256 / sh.np;                                 // columns a block: as in si_delta_scan
+  if (cols > dv) cols = dv;
+  if (cols < 1) cols = 1;
+  const long long per = (long long)num_seqs * H;
+  while (cols > 1 && (cols / 2) * sh.np >= 32 && per * ((dv + cols - 1) / cols) < si_sm_count()) cols /= 2;
+  const int zb = (dv + cols - 1) / cols;
+  if (zb > 65535) return -2;
+  const int threads = ((cols * sh.np + 31) / 32) * 32;
+  const size_t per_tok = (size_t)(3 * sh.np * sh.rpt + ((cols + 3) & ~3) + 4) * sizeof(float);
+  int chunk = DELTA_CHUNK;                                // fewer tokens a buffer where two of 32 would not fit
+  while (chunk > 1 && 2 * chunk * per_tok > (sh.rpt <= 8 ? 110 : 200) * 1024) chunk /= 2;
+  const size_t smem = 2 * chunk * per_tok;
+  if (smem > 200 * 1024) return -2;
+  const dim3 grid(num_seqs, H, zb), block(threads);
+#define CHANNEL_LAUNCH(R, P)                                                                                         \
+  {                                                                                                                  \
+    static size_t configured = 0;                                                                                    \
+    if (smem > 48 * 1024 && smem > configured) {                                                                     \
+      if (cudaFuncSetAttribute(channel_delta_scan_kernel<R, P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
+        return -2;                                                                                                   \
+      configured = smem;                                                                                             \
+    }                                                                                                                \
+    si_launch(channel_delta_scan_kernel<R, P>, grid, block, smem, stream, xc, xc_stride, dec, dec_stride, bg, state, state_stride, y, \
+              y_stride, q_start, ctx_len, slots, G, H, dk, dv, cols, chunk);                                         \
+  }
+  if (sh.np < 16) {
+    if (sh.rpt != 4) return -2;
+    switch (sh.np) {
+      case 1: CHANNEL_LAUNCH(4, 1) break;
+      case 2: CHANNEL_LAUNCH(4, 2) break;
+      case 4: CHANNEL_LAUNCH(4, 4) break;
+      case 8: CHANNEL_LAUNCH(4, 8) break;
+      default: return -2;
+    }
+  } else if (sh.np == 16) {
+    switch (sh.rpt) {
+      case 4: CHANNEL_LAUNCH(4, 16) break;
+      case 8: CHANNEL_LAUNCH(8, 16) break;
+      case 12: CHANNEL_LAUNCH(12, 16) break;
+      case 16: CHANNEL_LAUNCH(16, 16) break;
+      case 20: CHANNEL_LAUNCH(20, 16) break;
+      case 24: CHANNEL_LAUNCH(24, 16) break;
+      case 28: CHANNEL_LAUNCH(28, 16) break;
+      case 32: CHANNEL_LAUNCH(32, 16) break;
+      default: return -2;
+    }
+  } else {
+    return -2;
+  }
+#undef CHANNEL_LAUNCH
+  return si_last_error();
+}
+
 // ---- the read-out's norm and gate ------------------------------------------------------------------------------------
-//   out[t, h, :] = post * w_h * o[t, h, :] * rsqrt(mean(o[t, h, :]^2) + eps) * silu(z[t, h, :])
+//   out[t, h, :] = post * w_h * o[t, h, :] * rsqrt(mean(o[t, h, :]^2) + eps) * gate(z[t, h, :]),   gate silu or sigmoid
 // w [dv] shared by the heads (w_head_stride 0) or [H, dv] with one row a head (w_head_stride dv); post one number.
 // o fp32, z and out in the compute dtype (z and out views with a row stride). One warp a (row, head).
 template <typename T>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __restrict__ o, long long o_stride, const T* __restrict__ z,
     long long z_stride, const float* __restrict__ w, T* __restrict__ out, long long out_stride, long long pairs, int H, int dv,
-    float eps, long long w_head_stride, float post) {
+    float eps, long long w_head_stride, float post, int sigmoid) {
   pdl_prologue();
   const long long wi = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (wi >= pairs) return;
@@ -294,22 +560,22 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __rest
   T* dst = out + t * out_stride + (size_t)h * dv;
   for (int i = lane; i < dv; i += 32) {
     const float zz = to_f32<T>(zr[i]);
-    dst[i] = from_f32<T>(orow[i] * rs * w[i] * (zz / (1.f + expf(-zz))));
+    dst[i] = from_f32<T>(orow[i] * rs * w[i] * ((sigmoid ? 1.f : zz) / (1.f + expf(-zz))));
   }
 }
 
 SI_EXPORT int si_head_norm_gate(const float* o, long long o_stride, const void* z, int dtype, long long z_stride,
                                 const float* w, void* out, long long out_stride, int rows, int H, int dv, float eps,
-                                long long w_head_stride, float post, cudaStream_t stream) {
+                                long long w_head_stride, float post, int sigmoid, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (H <= 0 || dv <= 0) return -2;
   const long long pairs = (long long)rows * H;
   const dim3 grid((unsigned)((pairs + 7) / 8)), block(256);
   if (dtype == SI_BF16)
     si_launch(head_norm_gate_kernel<__nv_bfloat16>, grid, block, 0, stream, o, o_stride, (const __nv_bfloat16*)z, z_stride, w,
-              (__nv_bfloat16*)out, out_stride, pairs, H, dv, eps, w_head_stride, post);
+              (__nv_bfloat16*)out, out_stride, pairs, H, dv, eps, w_head_stride, post, sigmoid);
   else
     si_launch(head_norm_gate_kernel<float>, grid, block, 0, stream, o, o_stride, (const float*)z, z_stride, w, (float*)out,
-              out_stride, pairs, H, dv, eps, w_head_stride, post);
+              out_stride, pairs, H, dv, eps, w_head_stride, post, sigmoid);
   return si_last_error();
 }

@@ -117,3 +117,37 @@ SI_EXPORT int si_embedding_pair(const int* tokens, const int* positions, const i
               mul_prev, mul_cur, num_seqs, status);
   return si_last_error();
 }
+
+// ---- a layer's own input for a token ------------------------------------------------------------------------------------
+// out[t, j] = gelu_tanh(z[t, j]) * table[tokens[t] * stride + j] for j < dim, 0 for the columns from there to `width`; the table's
+// slice of the layer starts at `table`. z and out in the compute dtype, as the table.
+template <typename T>
+__global__ void __launch_bounds__(256) token_gate_kernel(const T* __restrict__ z, long long z_stride, const int* __restrict__ tokens,
+    const T* __restrict__ table, long long stride, T* __restrict__ out, long long out_stride, long long n, int width, int dim, int rows) {
+  pdl_prologue();
+  for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < n; idx += (long long)gridDim.x * blockDim.x) {
+    const long long t = idx / width;
+    const int j = (int)(idx - t * width), tok = tokens[t];
+    float g = 0.f;
+    if (j < dim && tok >= 0 && tok < rows) {
+      const float v = to_f32<T>(z[t * z_stride + j]);
+      g = 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v))) * to_f32<T>(table[(size_t)tok * stride + j]);
+    }
+    out[t * out_stride + j] = from_f32<T>(g);
+  }
+}
+
+SI_EXPORT int si_token_gate(const void* z, int dtype, long long z_stride, const int* tokens, const void* table, long long stride,
+                            void* out, long long out_stride, int num_tokens, int width, int dim, int rows, cudaStream_t stream) {
+  if (num_tokens <= 0 || width <= 0) return 0;
+  if (dim < 0 || dim > width) return -2;
+  const long long n = (long long)num_tokens * width, want = (n + 255) / 256;
+  const dim3 grid((unsigned)(want < 8LL * si_sm_count() ? want : 8LL * si_sm_count())), block(256);
+  if (dtype == SI_BF16)
+    si_launch(token_gate_kernel<__nv_bfloat16>, grid, block, 0, stream, (const __nv_bfloat16*)z, z_stride, tokens,
+              (const __nv_bfloat16*)table, stride, (__nv_bfloat16*)out, out_stride, n, width, dim, rows);
+  else
+    si_launch(token_gate_kernel<float>, grid, block, 0, stream, (const float*)z, z_stride, tokens, (const float*)table, stride,
+              (float*)out, out_stride, n, width, dim, rows);
+  return si_last_error();
+}

@@ -44,6 +44,9 @@ struct SkinnyRope {
   int glu;
   const float* glu_bias;
   float glu_limit, glu_alpha;
+  // act = 2: gelu_tanh of the sum (rounded to bf16 first) times entry n of a slice of the row's token in a table,
+  // side_table[tokens[m] * side_stride + n], columns beyond side_dim zero
+  const int* tokens; const bf16* side_table; long long side_stride; int side_dim, side_rows;
 };
 
 __device__ __forceinline__ void mma16816(float (&d)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3,
@@ -244,6 +247,12 @@ gemm_skinny_kernel(const bf16* __restrict__ x, long long ldx, const bf16* __rest
       if (rope.act == 1) {
         s = fmaxf(__bfloat162float(__float2bfloat16_rn(s)), 0.f);
         s *= s;
+      } else if (rope.act == 2 && m < M) {
+        const int tok = rope.tokens[m];
+        const bool have = n < rope.side_dim && tok >= 0 && tok < rope.side_rows;
+        const float z = __bfloat162float(__float2bfloat16_rn(s));
+        const float e = have ? __bfloat162float(rope.side_table[(size_t)tok * rope.side_stride + n]) : 0.f;
+        s = have ? 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))) * e : 0.f;
       }
       if (n < N && m < M) store_out<TO>(out + (size_t)m * ldo + n, s);
     }
@@ -318,6 +327,20 @@ SI_EXPORT int si_gemm_skinny_relu2(const void* x, long long ldx, const void* W, 
   if (((uintptr_t)x % 16) || ((uintptr_t)W % 16)) return -2;
   SkinnyRope r = SkinnyRope();
   r.act = 1;
+  skinny_dispatch<bf16, false, false>((unsigned)((N + 15) / 16), stream, (const bf16*)x, ldx, (const bf16*)W, ldw, (bf16*)out, ldo, M, N, K, r);
+  return si_last_error();
+}
+
+// out[M, N] (bf16) = gelu_tanh(x W^T) * e, e[m, n] = table[tokens[m], n] of the table's slice at `table` (rows `stride` apart, `rows` of
+// them, `dim` entries; columns of the product beyond them become zero): a layer's own input for the row's token.
+SI_EXPORT int si_gemm_skinny_token_gate(const void* x, long long ldx, const void* W, long long ldw, void* out, long long ldo, int M,
+                                        int N, int K, const int* tokens, const void* table, long long stride, int dim, int rows,
+                                        cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M > 16 || K <= 0 || (K % 8) || (ldx % 8) || (ldw % 8) || !tokens || !table || dim < 0 || dim > N) return -2;
+  if (((uintptr_t)x % 16) || ((uintptr_t)W % 16)) return -2;
+  SkinnyRope r = SkinnyRope();
+  r.act = 2; r.tokens = tokens; r.side_table = (const bf16*)table; r.side_stride = stride; r.side_dim = dim; r.side_rows = rows;
   skinny_dispatch<bf16, false, false>((unsigned)((N + 15) / 16), stream, (const bf16*)x, ldx, (const bf16*)W, ldw, (bf16*)out, ldo, M, N, K, r);
   return si_last_error();
 }

@@ -71,7 +71,7 @@ enum : int { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_ADD = 2, EPI_RELU2 = 3, EPI_GLU_
 
 // What EPI_GLU_LIMITED needs: the biases of the stacked gate/up columns (fp32, in the columns' order; may be null), the
 // limit and the sigmoid's factor.
-struct EpiArgs { const float* bias; float limit, alpha; };
+struct EpiArgs { const float* bias; float limit, alpha, shift = 1.f; };      // shift: what the pairs' form adds to its up
 
 // The square of relu of every sum, each rounded to bf16 first (what a stored product followed by the activation
 // kernel gives).
@@ -85,13 +85,13 @@ __device__ __forceinline__ void relu2_row32(float (&v)[32]) {
 
 // The gated activation with limits where gate and up columns come in turn (column 2i an entry's gate sum, column 2i + 1
 // its up sum; no biases): 16 outputs from 32 accumulator columns, gate and up rounded to bf16 first.
-__device__ __forceinline__ void store_glu_pairs16(bf16* dst, const float (&v)[32], float limit, float alpha, int valid, bool vec) {
+__device__ __forceinline__ void store_glu_pairs16(bf16* dst, const float (&v)[32], float limit, float alpha, float shift, int valid, bool vec) {
   float o[16];
 #pragma unroll
   for (int i = 0; i < 16; ++i) {
     const float gv = fminf(__bfloat162float(__float2bfloat16_rn(v[2 * i])), limit);
     const float uv = fminf(fmaxf(__bfloat162float(__float2bfloat16_rn(v[2 * i + 1])), -limit), limit);
-    o[i] = gv / (1.f + __expf(-alpha * gv)) * (uv + 1.f);
+    o[i] = gv / (1.f + __expf(-alpha * gv)) * (uv + shift);
   }
   if (vec && valid == 16) {
 #pragma unroll
@@ -679,7 +679,7 @@ gemm_tc05_grouped_kernel(const __grid_constant__ CUtensorMap amap, const __grid_
           const int n = n0 + h * 128 + c * 32;
           if (r < rows && n < N) {
             if (EPI == EPI_GLU_PAIRS) {              // out has N / 2 columns: an entry for every gate/up pair
-              store_glu_pairs16((bf16*)out + (size_t)(first + r) * ldo + n / 2, v[c], epi.limit, epi.alpha, min(16, (N - n) / 2), vec);
+              store_glu_pairs16((bf16*)out + (size_t)(first + r) * ldo + n / 2, v[c], epi.limit, epi.alpha, epi.shift, min(16, (N - n) / 2), vec);
             } else {
               if (EPI == EPI_RELU2) relu2_row32(v[c]);
               store_row32<TO>(out + (size_t)(first + r) * ldo + n, v[c], min(32, N - n), vec);
@@ -716,10 +716,10 @@ SI_EXPORT int si_gemm_tc05_grouped_ok(int P, int E) {
 // out[p, :] = act(x[p, :] W[e]^T) for the rows p of group e, offsets[e] <= p < offsets[e + 1] (int32 [E + 1] on the device,
 // offsets[E] <= P). x: [P, K] bf16 rows `ldx` apart; `wmap`: W [E, N, K] described as [E * N, K] with boxes of 256 rows;
 // out [P, N] bf16 or fp32; act 0: none, 1: the square of relu (of the sum rounded to bf16; bf16 out only), 2: the gated
-// activation with limits over gate/up columns in turn (out [P, N / 2] bf16; `limit`, `alpha`).
+// activation with limits over gate/up columns in turn (out [P, N / 2] bf16; `limit`, `alpha`, `shift`: g sigmoid(alpha g) (u + shift)).
 SI_EXPORT int si_gemm_tc05_grouped(const void* x, long long ldx, const void* wmap, void* out, long long ldo, int out_dtype,
                                    const int* offsets, int P, int E, int N, int K, int act, float limit, float alpha,
-                                   int* status, cudaStream_t stream) {
+                                   float shift, int* status, cudaStream_t stream) {
   if (P <= 0 || N <= 0) return 0;
   if (!si_gemm_tc05_grouped_ok(P, E) || act < 0 || act > 2 || (act >= 1 && out_dtype != SI_BF16)) return -2;
   if (act == 2 && (N % 2 || !(limit > 0.f))) return -2;
@@ -727,7 +727,7 @@ SI_EXPORT int si_gemm_tc05_grouped(const void* x, long long ldx, const void* wma
   const int rc = gemm_tc05_common(x, ldx, wmap, &am, P, K);
   if (rc) return rc;
   const CUtensorMap& bm = *(const CUtensorMap*)wmap;
-  if (act == 2) return launch_grouped<bf16, EPI_GLU_PAIRS>(am, bm, out, ldo, offsets, P, E, N, K, status, stream, EpiArgs{nullptr, limit, alpha});
+  if (act == 2) return launch_grouped<bf16, EPI_GLU_PAIRS>(am, bm, out, ldo, offsets, P, E, N, K, status, stream, EpiArgs{nullptr, limit, alpha, shift});
   if (act == 1) return launch_grouped<bf16, EPI_RELU2>(am, bm, out, ldo, offsets, P, E, N, K, status, stream);
   if (out_dtype == SI_BF16) return launch_grouped<bf16, EPI_STORE>(am, bm, out, ldo, offsets, P, E, N, K, status, stream);
   return launch_grouped<float, EPI_STORE>(am, bm, out, ldo, offsets, P, E, N, K, status, stream);

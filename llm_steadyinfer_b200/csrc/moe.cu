@@ -4,7 +4,9 @@
 //   moe_route    scores z = W_r x (fp32 sums over the row in fp32), s = sigmoid(z) (or softmax over the experts), the `top`
 //                largest (ties: the lower index), weights s * scale (optionally divided by their sum); rows of further
 //                gate matrices behind the router's give sigmoid(w . x) for the same row (a gate on a shared expert).
-//                With a choice bias the `top` largest of s + bias are chosen instead; the weights stay s.
+//                With a choice bias the `top` largest of s + bias are chosen instead; the weights stay s. With groups the experts
+//                fall into `groups` equal runs of neighbours; only those of the `keep` runs with the largest sum of their two best
+//                choice scores can be chosen.
 //   moe_plan     the (row, choice) pairs ordered by expert, rows in step order within an expert: offsets per expert, the
 //                row of every place, the place of every pair. Counting ranks within chunks of 1,024 pairs, so the order
 //                never depends on timing.
@@ -12,7 +14,8 @@
 //                found from the offsets by every block itself (blocks beyond the last tile leave). bf16 on mma.sync
 //                m16n8k16 with fp32 sums, tiles of 64 or 16 rows x 64 columns, three cp.async stages; fp32 on FFMA.
 //                act "glu_limited": W_e holds gate and up rows in turn (row 2i the gate of entry i, row 2i + 1 its up), and
-//                C[place, i] = g sigmoid(alpha g) (u + 1) with g = min(gate sum, limit), u = clamp(up sum, -limit, limit).
+//                C[place, i] = g sigmoid(alpha g) (u + shift) with g = min(gate sum, limit), u = clamp(up sum, -limit, limit)
+//                (no limit, alpha 1 and shift 0: silu(gate) * up).
 //                A row's sums run over k in the same order wherever the row lies in its tile. (Many rows in bf16
 //                go to the tcgen05 grouped product of gemm_tc05.cu instead, behind `moe_gather`.)
 //   moe_combine  out[t] = sum_c weight[t, c] * Y[place(t, c)] (+ gate[t] * shared[t]), the choices in their own order.
@@ -28,8 +31,8 @@ typedef __nv_bfloat16 bf16;
 // [T, top]; gates fp32 [T, extra]. mode 0: sigmoid scores; 1: softmax over the experts. One block a row.
 template <typename T>
 __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x, long long x_stride, const T* __restrict__ w,
-    int E, int extra, int d, int top, float scale, int mode, int renorm, const float* __restrict__ choice_bias,
-    int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ gates) {
+    int E, int extra, int d, int top, float scale, int mode, int renorm, float renorm_eps, int groups, int keep,
+    const float* __restrict__ choice_bias, int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ gates) {
   extern __shared__ float rsm[];                       // the row [d], scores [E + extra], used [E], choice keys [E]
   pdl_prologue();
   float* xr = rsm;
@@ -78,6 +81,26 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x,
     key[e] = kv;
   }
   __syncwarp();
+  if (groups > 1 && keep < groups) {                     // experts of the groups that are not kept cannot be chosen
+    float* gscore = key + E;
+    const int size = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float b1 = -INFINITY, b2 = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float kv = key[e];
+        if (kv > b1) { b2 = b1; b1 = kv; } else if (kv > b2) { b2 = kv; }
+      }
+      gscore[g] = size > 1 ? b1 + b2 : b1;
+    }
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      int better = 0;                                    // groups before this one in the order of scores (ties: the lower index)
+      for (int o = 0; o < groups; ++o) better += gscore[o] > gscore[g] || (gscore[o] == gscore[g] && o < g);
+      if (better >= keep)
+        for (int e = g * size; e < (g + 1) * size; ++e) used[e] = 1.f;
+    }
+    __syncwarp();
+  }
   float total = 0.f, mine = 0.f;
   int my_id = 0;
   for (int c = 0; c < top; ++c) {
@@ -101,16 +124,18 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x,
   }
   if (lane < top) {
     ids[t * top + lane] = my_id;
-    wts[t * top + lane] = (renorm ? mine / total : mine) * scale;
+    wts[t * top + lane] = (renorm ? mine / (total + renorm_eps) : mine) * scale;
   }
 }
 
 SI_EXPORT int si_moe_route(const void* x, int dtype, long long x_stride, const void* w, int E, int extra, int d, int top,
-                           float scale, int mode, int renorm, const float* choice_bias, int* ids, float* wts, float* gates,
-                           int rows, cudaStream_t stream) {
+                           float scale, int mode, int renorm, float renorm_eps, int groups, int keep, const float* choice_bias,
+                           int* ids, float* wts, float* gates, int rows, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || top > 32 || extra < 0 || d <= 0 || mode < 0 || mode > 1) return -2;
-  const size_t smem = (size_t)(d + 3 * E + extra) * sizeof(float);
+  if (groups > 1 && (E % groups || keep < 1 || keep > groups || !choice_bias)) return -2;      // groups go by choice scores
+  if (groups > 1 && (long long)keep * (E / groups) < top) return -2;
+  const size_t smem = (size_t)(d + 3 * E + extra + (groups > 1 ? groups : 0)) * sizeof(float);
   if (smem > 160 * 1024) return -2;
   const dim3 grid(rows), block(E + extra >= 8 ? 256 : 128);
 #define ROUTE_LAUNCH(T)                                                                                                \
@@ -121,7 +146,7 @@ SI_EXPORT int si_moe_route(const void* x, int dtype, long long x_stride, const v
       configured = smem;                                                                                             \
     }                                                                                                                \
     si_launch(moe_route_kernel<T>, grid, block, smem, stream, (const T*)x, x_stride, (const T*)w, E, extra, d, top, scale, \
-              mode, renorm, choice_bias, ids, wts, gates);                                                           \
+              mode, renorm, renorm_eps, groups, keep, choice_bias, ids, wts, gates);                                                           \
   }
   if (dtype == SI_BF16) ROUTE_LAUNCH(bf16) else ROUTE_LAUNCH(float)
 #undef ROUTE_LAUNCH
@@ -249,10 +274,10 @@ __device__ __forceinline__ float moe_act(float v, int act) {
   return v;
 }
 #define MOE_ACT_GLU_LIMITED 4
-// gate and up sums of one entry (neighbouring columns of the product): g sigmoid(alpha g) (u + 1) within the limit
-__device__ __forceinline__ float moe_glu_limited(float gate, float up, float limit, float alpha) {
+// gate and up sums of one entry (neighbouring columns of the product): g sigmoid(alpha g) (u + shift) within the limit
+__device__ __forceinline__ float moe_glu_limited(float gate, float up, float limit, float alpha, float shift) {
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
-  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+  return g / (1.f + expf(-alpha * g)) * (u + shift);
 }
 
 // The tile a block takes: expert, first place, places. Thread 0 walks the offsets; false: no tile is left for this block.
@@ -284,7 +309,7 @@ __device__ __forceinline__ void moe_cp16(void* dst, const void* src, int bytes) 
 template <int BM, int BN, int MOE_BK, int MOE_STAGES>
 __global__ void __launch_bounds__(128) moe_gemm_bf16_kernel(const bf16* __restrict__ A, long long a_stride,
     const int* __restrict__ a_rows, const bf16* __restrict__ W, void* __restrict__ C, long long c_stride, int c_f32,
-    const int* __restrict__ offsets, int E, int N, int K, int act, int wide, float limit, float alpha) {
+    const int* __restrict__ offsets, int E, int N, int K, int act, int wide, float limit, float alpha, float shift) {
   constexpr int MOE_PITCH = MOE_BK + 8, KC = MOE_BK / 8;
   __shared__ __align__(16) bf16 As[MOE_STAGES][BM][MOE_PITCH];
   __shared__ __align__(16) bf16 Ws[MOE_STAGES][BN][MOE_PITCH];
@@ -374,7 +399,7 @@ __global__ void __launch_bounds__(128) moe_gemm_bf16_kernel(const bf16* __restri
       if (act == MOE_ACT_GLU_LIMITED) {                 // the thread's two columns are an entry's gate and up
         const int n = n0 + wn0 + nt * 8 + 2 * tq;
         if (n + 1 >= N) continue;
-        const float v = moe_glu_limited(acc[nt][half * 2], acc[nt][half * 2 + 1], limit, alpha);
+        const float v = moe_glu_limited(acc[nt][half * 2], acc[nt][half * 2 + 1], limit, alpha, shift);
         if (c_f32) reinterpret_cast<float*>(C)[place * c_stride + (n >> 1)] = v;
         else reinterpret_cast<bf16*>(C)[place * c_stride + (n >> 1)] = __float2bfloat16_rn(v);
         continue;
@@ -394,7 +419,7 @@ __global__ void __launch_bounds__(128) moe_gemm_bf16_kernel(const bf16* __restri
 // True 32-bit: tiles of 32 places x 64 columns, 16 entries of k at a time, a thread 2 x 4 results.
 __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restrict__ A, long long a_stride,
     const int* __restrict__ a_rows, const float* __restrict__ W, float* __restrict__ C, long long c_stride,
-    const int* __restrict__ offsets, int E, int N, int K, int act, float limit, float alpha) {
+    const int* __restrict__ offsets, int E, int N, int K, int act, float limit, float alpha, float shift) {
   constexpr int BM = 32, BK = 16;
   __shared__ float As[BK][BM + 1];
   __shared__ float Ws[BK][MOE_BN + 1];
@@ -442,7 +467,7 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
 #pragma unroll
       for (int c = 0; c < 4; c += 2) {
         const int n = n0 + tx * 4 + c;
-        if (n + 1 < N) C[(size_t)(first + r) * c_stride + (n >> 1)] = moe_glu_limited(acc[rr][c], acc[rr][c + 1], limit, alpha);
+        if (n + 1 < N) C[(size_t)(first + r) * c_stride + (n >> 1)] = moe_glu_limited(acc[rr][c], acc[rr][c + 1], limit, alpha, shift);
       }
       continue;
     }
@@ -456,7 +481,7 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const float* __restri
 
 SI_EXPORT int si_moe_gemm(const void* A, int dtype, long long a_stride, const int* a_rows, const void* W, void* C, int c_dtype,
                           long long c_stride, const int* offsets, int P, int E, int N, int K, int act, float limit, float alpha,
-                          cudaStream_t stream) {
+                          float shift, cudaStream_t stream) {
   if (P <= 0) return 0;
   if (E <= 0 || N <= 0 || K <= 0 || act < 0 || act > MOE_ACT_GLU_LIMITED) return -2;
   if (act == MOE_ACT_GLU_LIMITED && (N % 2 || !(limit > 0.f))) return -2;
@@ -466,7 +491,7 @@ SI_EXPORT int si_moe_gemm(const void* A, int dtype, long long a_stride, const in
     if (c_dtype != SI_F32) return -2;
     const dim3 grid((P + 31) / 32 + E, ny), block(256);
     si_launch(moe_gemm_f32_kernel, grid, block, 0, stream, (const float*)A, a_stride, a_rows, (const float*)W, (float*)C, c_stride,
-              offsets, E, N, K, act, limit, alpha);
+              offsets, E, N, K, act, limit, alpha, shift);
     return si_last_error();
   }
   const int wide = (K % 8 == 0 && a_stride % 8 == 0 && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) ? 1 : 0;
@@ -474,11 +499,11 @@ SI_EXPORT int si_moe_gemm(const void* A, int dtype, long long a_stride, const in
     // (32 columns a block, twice the blocks, measured no faster: 0.61 against 0.58 ms for the 16 launches of a decode step)
     const dim3 grid((P + 15) / 16 + E, ny), block(128);
     si_launch(moe_gemm_bf16_kernel<16, 64, 64, 4>, grid, block, 0, stream, (const bf16*)A, a_stride, a_rows, (const bf16*)W, C, c_stride,
-              c_dtype == SI_F32 ? 1 : 0, offsets, E, N, K, act, wide, limit, alpha);
+              c_dtype == SI_F32 ? 1 : 0, offsets, E, N, K, act, wide, limit, alpha, shift);
   } else {
     const dim3 grid((P + 63) / 64 + E, ny), block(128);
     si_launch(moe_gemm_bf16_kernel<64, 64, 32, 3>, grid, block, 0, stream, (const bf16*)A, a_stride, a_rows, (const bf16*)W, C, c_stride,
-              c_dtype == SI_F32 ? 1 : 0, offsets, E, N, K, act, wide, limit, alpha);
+              c_dtype == SI_F32 ? 1 : 0, offsets, E, N, K, act, wide, limit, alpha, shift);
   }
   return si_last_error();
 }

@@ -237,6 +237,45 @@ def add_norm(resid, delta=None, weight=None, eps: float = 0.0, out=None, rows=No
              R, d, float(eps), _stream()), f"add_norm(hidden={d})")
 
 
+NORM_KINDS = {"copy": 0, "tanh": 1, "rms": 2}
+
+
+def stream_add(resid, delta=None, delta_norm=None, delta_bias=None, out=None, norm=None, rows=None) -> None:
+    """The residual add where the norms around it are of any kind, all sums and norms fp32:
+        d = delta (+ delta_bias);   resid (fp32, in place) += delta_norm(d);   out = norm(resid)     (each part may be absent)
+    A norm is ``None`` (the row as it is), ``("tanh", weight, bias, alpha)``: tanh(alpha x) * weight + bias, or
+    ``("rms", weight, eps)``: weight * x * rsqrt(mean(x^2) + eps); weights and biases fp32 [hidden]. ``out`` without ``norm`` is the
+    stream itself in out's dtype. With ``rows`` (int32 [R]) output row r comes from stream row rows[r] and resid stays as it is."""
+    _cuda(resid, delta, delta_bias, out, rows)
+    _i32(rows, "rows")
+    d = resid.shape[-1]
+    _need(resid.dtype == torch.float32 and resid.is_contiguous() and resid.dim() == 2, "stream_add: resid must be contiguous fp32 rows")
+    _need(out is not None or delta is not None, "stream_add: nothing to do")
+    _need(out is not None or rows is None, "stream_add: rows are for an output")
+    if out is not None:
+        _need(out.is_contiguous() and out.shape == (rows.numel() if rows is not None else resid.shape[0], d), "stream_add: out must be [rows, hidden]")
+    xd = out if out is not None else delta
+    _need(delta is None or (delta.is_contiguous() and delta.shape == resid.shape and delta.dtype == xd.dtype),
+          "stream_add: delta must match resid's shape and out's dtype")
+    _f32v(delta_bias, "delta_bias", d)
+
+    def parts(n):
+        if n is None:
+            return 0, None, None, 0.0
+        _need(n[0] in ("tanh", "rms"), f"stream_add: norm kind {n[0]!r}")
+        _cuda(*n[1:-1])
+        for t in n[1:-1]:
+            _f32v(t, "norm weight", d)
+        return NORM_KINDS[n[0]], n[1], (n[2] if n[0] == "tanh" else None), float(n[-1])
+
+    dk, dw, db, da = parts(delta_norm)
+    ok, ow, ob, oa = parts(norm)
+    f = _fn("stream_add", "si_stream_add",
+            [_c_p, _c_p, _c_p, _c_int, _c_p, _c_p, _c_f, _c_p, _c_p, _c_int, _c_p, _c_p, _c_f, _c_int, _c_int, _c_int, _c_p])
+    _check(f(_ptr(resid), _ptr(delta), _ptr(delta_bias), dk, _ptr(dw), _ptr(db), da, _ptr(rows), _ptr(out), ok, _ptr(ow), _ptr(ob), oa,
+             _dt(xd), out.shape[0] if out is not None else resid.shape[0], d, _stream()), f"stream_add(hidden={d})")
+
+
 def rope_kv_write(qkv, positions, row_seq, inv_freq, rot_dim: int, block_table, k_cache, v_cache,
                   page_size: int, num_seqs: int, H: int, KV: int, hs: int, status=None) -> None:
     """Rotate q (in place) and k, store k and v of every row into its page.
@@ -677,6 +716,36 @@ def gemm_skinny_relu2(a, w, out, checked: bool = False) -> None:
     f = _fn("gemm_skinny", "si_gemm_skinny_relu2", [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p])
     _check(f(_ptr(a), a.stride(0), _ptr(w), w.stride(0), _ptr(out), out.stride(0), M, N, K, _stream()),
            f"gemm_skinny_relu2(M={M}, N={N}, K={K})")
+
+
+def gemm_skinny_token_gate(a, w, out, tokens, table, dim: int, checked: bool = False) -> None:
+    """``token_gate`` in the epilogue of its product: out[m, n] (bf16) = gelu_tanh((a @ w^T)[m, n]) * table[tokens[m], n] for n < ``dim``,
+    0 behind it; M <= 16. ``table``: bf16 rows (a view of the layer's columns of the token table)."""
+    _cuda(a, w, out, tokens, table)
+    _i32(tokens, "tokens")
+    M, K = a.shape
+    N = w.shape[0]
+    _need(w.shape[1] == K and out.shape == (M, N) and out.dtype == torch.bfloat16 and tokens.numel() == M, "gemm_skinny_token_gate: shapes, bf16 output")
+    _need(table.dtype == torch.bfloat16 and table.dim() == 2 and table.stride(1) == 1 and table.shape[1] == dim <= N, "gemm_skinny_token_gate: table [vocab, dim]")
+    _need(checked or gemm_skinny_ok(a, w, out), "gemm_skinny_token_gate: bf16 inputs, at most 16 rows, K a multiple of 8, 16-byte aligned rows")
+    f = _fn("gemm_skinny", "si_gemm_skinny_token_gate",
+            [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_p])
+    _check(f(_ptr(a), a.stride(0), _ptr(w), w.stride(0), _ptr(out), out.stride(0), M, N, K, _ptr(tokens), _ptr(table), table.stride(0),
+             int(dim), table.shape[0], _stream()), f"gemm_skinny_token_gate(M={M}, N={N}, K={K})")
+
+
+def token_gate(z, tokens, table, out) -> None:
+    """out[t, j] = gelu_tanh(z[t, j]) * table[tokens[t], j] for the table's columns (a view [vocab, dim]), 0 for the columns behind them;
+    ``z`` and ``out`` [T, width], width >= dim, in the table's dtype."""
+    _cuda(z, tokens, table, out)
+    _i32(tokens, "tokens")
+    T, W = out.shape
+    _need(z.shape == (T, W) and z.stride(1) == 1 and out.stride(1) == 1 and z.dtype == out.dtype == table.dtype and tokens.numel() == T,
+          "token_gate: z and out must be [T, width] in the table's dtype")
+    _need(table.dim() == 2 and table.stride(1) == 1 and table.shape[1] <= W, "token_gate: table [vocab, dim]")
+    f = _fn("embedding", "si_token_gate", [_c_p, _c_int, _c_ll, _c_p, _c_p, _c_ll, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_int, _c_p])
+    _check(f(_ptr(z), _dt(z), z.stride(0), _ptr(tokens), _ptr(table), table.stride(0), _ptr(out), out.stride(0), T, W, table.shape[1],
+             table.shape[0], _stream()), f"token_gate(dim={table.shape[1]})")
 
 
 def gemm_skinny_swiglu(a, w, out, checked: bool = False) -> None:
@@ -1520,8 +1589,73 @@ def delta_scan(xc, bg, state, y, q_start, ctx_len, slots, num_seqs: int, G: int,
              _ptr(ctx_len), _ptr(slots), int(num_seqs), G, H, dk, dv, _stream()), f"delta_scan(heads={H}, dk={dk}, dv={dv})")
 
 
-def head_norm_gate(o, z, weight, out, H: int, dv: int, eps: float, post: float = 1.0) -> None:
-    """out[t, h, :] = post * weight * o[t, h, :] * rsqrt(mean(o[t, h, :]^2) + eps) * silu(z[t, h, :]); ``o`` fp32 [T, H*dv],
+def channel_delta_prepare(xc, ba, b_off: int, dec, a_log, dt_bias, bg, G: int, H: int, dk: int) -> None:
+    """What the delta rule with a decay per key channel reads beside q, k and v: ``dec`` fp32 [T, H*dk] holds raw values x and receives
+    exp(-exp(a_log[h]) * softplus(x + dt_bias)) in place; ``bg`` fp32 [T, H + G] receives beta = sigmoid(b) of the H raw values
+    at column ``b_off`` of ``ba`` and, per query/key head, q . k of the vectors in ``xc`` (fp32 rows [q: G*dk | k: G*dk | ...])."""
+    _cuda(xc, ba, dec, a_log, dt_bias, bg)
+    T = xc.shape[0]
+    _need(xc.dtype == torch.float32 and xc.stride(1) == 1 and xc.shape[1] >= 2 * G * dk, "channel_delta_prepare: xc must be fp32 rows")
+    _need(ba.shape[0] == T and ba.stride(1) == 1 and ba.shape[1] >= b_off + H, "channel_delta_prepare: ba rows")
+    _need(dec.dtype == torch.float32 and dec.shape == (T, H * dk) and dec.stride(1) == 1, "channel_delta_prepare: dec must be fp32 [T, H*dk]")
+    _need(bg.dtype == torch.float32 and bg.is_contiguous() and bg.shape == (T, H + G), "channel_delta_prepare: bg must be fp32 [T, H + G]")
+    _f32v(a_log, "a_log", H); _f32v(dt_bias, "dt_bias", H * dk)
+    f = _fn("delta_rule", "si_channel_delta_prepare",
+            [_c_p, _c_ll, _c_p, _c_int, _c_ll, _c_int, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_p])
+    _check(f(_ptr(xc), xc.stride(0), _ptr(ba), _dt(ba), ba.stride(0), int(b_off), _ptr(dec), dec.stride(0), _ptr(a_log), _ptr(dt_bias),
+             _ptr(bg), T, G, H, dk, _stream()), f"channel_delta_prepare(heads={H})")
+
+
+def channel_delta_scan(xc, dec, bg, state, y, q_start, ctx_len, slots, num_seqs: int, G: int, H: int, dk: int, dv: int) -> None:
+    """``delta_scan`` with a decay per key channel: per head S <- diag(dec) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q. ``xc`` fp32
+    rows [q | k | v] with unit vectors q and k, ``dec`` fp32 [T, H*dk] and ``bg`` fp32 [T, H + G] as ``channel_delta_prepare`` leaves them;
+    the state as in ``delta_scan``."""
+    _cuda(xc, dec, bg, state, y, q_start, ctx_len, slots)
+    for t, nm in ((q_start, "q_start"), (ctx_len, "ctx_len"), (slots, "slots")):
+        _i32(t, nm)
+    T = xc.shape[0]
+    _need(xc.dtype == torch.float32 and xc.stride(1) == 1 and xc.shape[1] >= 2 * G * dk + H * dv, "channel_delta_scan: xc must be fp32 [T, 2*G*dk + H*dv]")
+    _need(dec.dtype == torch.float32 and dec.shape == (T, H * dk) and dec.stride(1) == 1, "channel_delta_scan: dec must be fp32 [T, H*dk]")
+    _need(bg.dtype == torch.float32 and bg.is_contiguous() and bg.shape == (T, H + G), "channel_delta_scan: bg must be fp32 [T, H + G]")
+    _need(y.dtype == torch.float32 and y.shape == (T, H * dv) and y.stride(1) == 1, "channel_delta_scan: y must be fp32 [T, H*dv]")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
+          and state.shape[1] >= H * delta_state_floats(dk, dv),
+          "channel_delta_scan: state must be fp32 [slots, >= H * delta_state_floats(dk, dv)]")
+    f = _fn("delta_rule", "si_channel_delta_scan",
+            [_c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p])
+    _check(f(_ptr(xc), xc.stride(0), _ptr(dec), dec.stride(0), _ptr(bg), _ptr(state), state.stride(0), _ptr(y), y.stride(0), _ptr(q_start),
+             _ptr(ctx_len), _ptr(slots), int(num_seqs), G, H, dk, dv, _stream()), f"channel_delta_scan(heads={H}, dk={dk}, dv={dv})")
+
+
+def gated_linear(u, z, bias_r, bias_i, rate, y, y_bias, state, out, q_start, ctx_len, slots, num_seqs: int, scale: float = 1.0,
+                 kinds: int = 3) -> None:
+    """The real-gated linear recurrence per channel, all fp32: r = sigmoid(zr + bias_r), i = sigmoid(zi + bias_i), a = exp(-rate * r),
+    S <- a S + sqrt(1 - a^2) i u, out = scale * S * gelu_tanh(y + y_bias). ``u`` fp32 [T, W]; ``z`` fp32 [blocks, T, 2*W/blocks], a block's
+    raw gates [r | i]; ``bias_r``, ``bias_i``, ``rate``, ``y_bias`` fp32 [W] (the last may be None); ``y`` and ``out`` [T, W] views in the
+    compute dtype; ``state`` fp32 [slots, >= W], from zero for a portion that starts at position 0. ``kinds``: what the step holds, 1
+    sequences of one row, 2 longer portions, 3 both."""
+    _cuda(u, z, bias_r, bias_i, rate, y, y_bias, state, out, q_start, ctx_len, slots)
+    for t, nm in ((q_start, "q_start"), (ctx_len, "ctx_len"), (slots, "slots")):
+        _i32(t, nm)
+    T, W = u.shape
+    B = z.shape[0]
+    _need(u.dtype == torch.float32 and u.stride(1) == 1 and W % B == 0, "gated_linear: u must be fp32 [T, W]")
+    _need(z.dtype == torch.float32 and z.is_contiguous() and z.shape == (B, T, 2 * (W // B)), "gated_linear: z must be fp32 [blocks, T, 2*W/blocks]")
+    _need(y.shape == (T, W) and out.shape == (T, W) and y.stride(1) == 1 and out.stride(1) == 1 and y.dtype == out.dtype, "gated_linear: y and out must be [T, W]")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and state.shape[1] >= W, "gated_linear: state must be fp32 [slots, >= W]")
+    _f32v(bias_r, "bias_r", W); _f32v(bias_i, "bias_i", W); _f32v(rate, "rate", W); _f32v(y_bias, "y_bias", W)
+    f = _fn("gated_linear", "si_gated_linear",
+            [_c_p, _c_ll, _c_p, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_int, _c_ll, _c_p, _c_p, _c_ll, _c_p, _c_ll, _c_f, _c_p, _c_p,
+             _c_p, _c_int, _c_int, _c_int, _c_p, _c_p])
+    launches = ctypes.c_int(0)
+    _check(f(_ptr(u), u.stride(0), _ptr(z), W // B, z.stride(0), _ptr(bias_r), _ptr(bias_i), _ptr(rate), _ptr(y), _dt(y), y.stride(0),
+             _ptr(y_bias), _ptr(state), state.stride(0), _ptr(out), out.stride(0), float(scale), _ptr(q_start), _ptr(ctx_len),
+             _ptr(slots), int(num_seqs), W, int(kinds), ctypes.addressof(launches), _stream()), f"gated_linear(width={W})",
+           kernels=launches.value)
+
+
+def head_norm_gate(o, z, weight, out, H: int, dv: int, eps: float, post: float = 1.0, gate: str = "silu") -> None:
+    """out[t, h, :] = post * weight * o[t, h, :] * rsqrt(mean(o[t, h, :]^2) + eps) * gate(z[t, h, :]), gate "silu" or "sigmoid"; ``o`` fp32 [T, H*dv],
     ``z`` and ``out`` [T, H*dv] in the compute dtype (views with a row stride are fine), ``weight`` fp32 [dv] (shared by
     the heads) or [H*dv] (a row a head)."""
     _cuda(o, z, weight, out)
@@ -1532,9 +1666,10 @@ def head_norm_gate(o, z, weight, out, H: int, dv: int, eps: float, post: float =
     per_head = weight.numel() == H * dv and H > 1
     _f32v(weight, "weight", H * dv if per_head else dv)
     f = _fn("delta_rule", "si_head_norm_gate", [_c_p, _c_ll, _c_p, _c_int, _c_ll, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_int, _c_f,
-                                                 _c_ll, _c_f, _c_p])
+                                                 _c_ll, _c_f, _c_int, _c_p])
+    _need(gate in ("silu", "sigmoid"), f"head_norm_gate: gate {gate!r}")
     _check(f(_ptr(o), o.stride(0), _ptr(z), _dt(z), z.stride(0), _ptr(weight), _ptr(out), out.stride(0), T, H, dv, float(eps),
-             dv if per_head else 0, float(post), _stream()), f"head_norm_gate(heads={H}, dv={dv})")
+             dv if per_head else 0, float(post), 1 if gate == "sigmoid" else 0, _stream()), f"head_norm_gate(heads={H}, dv={dv})")
 
 
 # ---- small elementwise steps -----------------------------------------------------------------------------------------
@@ -1576,12 +1711,14 @@ MOE_SCORES = {"sigmoid": 0, "softmax": 1}
 
 
 def moe_route(x, w, E: int, top: int, scale: float, ids, wts, gates=None, scores: str = "sigmoid", renorm: bool = False,
-              choice_bias=None) -> None:
+              choice_bias=None, renorm_eps: float = 0.0, groups=None) -> None:
     """Scores of ``E`` experts for every row and the ``top`` largest: ``w`` [E + extra, d] holds the router's rows and
     behind them ``extra`` gate rows; ``ids`` int32 [T, top], ``wts`` fp32 [T, top] = score * scale (``renorm``: divided by
     the chosen scores' sum first), ``gates`` fp32 [T, extra] = sigmoid(w_gate . x). Scores are sigmoid(z) or softmax(z) of
     z = w x, summed in fp32 whatever the storage. ``choice_bias`` (fp32 [E]): the ``top`` largest of score + bias are chosen;
-    the weights are still made of the scores alone."""
+    the weights are still made of the scores alone. ``groups`` ``(count, keep)``: the experts fall into ``count`` equal runs of neighbours and
+    only those of the ``keep`` runs with the largest sum of their two best choice scores can be chosen. ``renorm_eps`` joins the sum
+    that the weights are divided by."""
     _cuda(x, w, ids, wts, gates, choice_bias)
     _f32v(choice_bias, "choice_bias", E)
     T, d = x.shape
@@ -1593,10 +1730,11 @@ def moe_route(x, w, E: int, top: int, scale: float, ids, wts, gates=None, scores
     if extra:
         _need(gates is not None and gates.dtype == torch.float32 and gates.is_contiguous() and gates.shape == (T, extra),
               "moe_route: gates must be fp32 [T, extra]")
-    f = _fn("moe", "si_moe_route", [_c_p, _c_int, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_int, _c_p, _c_p,
-                                    _c_p, _c_p, _c_int, _c_p])
+    f = _fn("moe", "si_moe_route", [_c_p, _c_int, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_int, _c_f, _c_int, _c_int, _c_f, _c_int, _c_int,
+                                    _c_p, _c_p, _c_p, _c_p, _c_int, _c_p])
+    count, keep = groups if groups is not None else (1, 1)
     _check(f(_ptr(x), _dt(x), x.stride(0), _ptr(w), E, extra, d, top, float(scale), MOE_SCORES[scores], 1 if renorm else 0,
-             _ptr(choice_bias), _ptr(ids), _ptr(wts), _ptr(gates), T, _stream()), f"moe_route(experts={E}, top={top})")
+             float(renorm_eps), int(count), int(keep), _ptr(choice_bias), _ptr(ids), _ptr(wts), _ptr(gates), T, _stream()), f"moe_route(experts={E}, top={top})")
 
 
 MOE_PLAN_CHUNK = 1024
@@ -1648,7 +1786,8 @@ def moe_gather(a, rows, out) -> None:
     _check(f(_ptr(a), _dt(a), a.stride(0), _ptr(rows), _ptr(out), out.stride(0), P, a.shape[0], K, _stream()), f"moe_gather(K={K})")
 
 
-def moe_gemm_tc05(a, w, out, offsets, act: str = "none", status=None, limit: float = 0.0, alpha: float = 1.702) -> None:
+def moe_gemm_tc05(a, w, out, offsets, act: str = "none", status=None, limit: float = 0.0, alpha: float = 1.702,
+                  shift: float = 1.0) -> None:
     """The grouped product on the tcgen05 tensor cores: out[p, :] = act(a[p, :] @ w[e]^T) for the places p of expert e
     (``a`` [P, K] already in the order of the places; ``moe_gemm_grouped_ok`` says when it may be called)."""
     _cuda(a, w, out, offsets, status)
@@ -1659,12 +1798,13 @@ def moe_gemm_tc05(a, w, out, offsets, act: str = "none", status=None, limit: flo
           and offsets.numel() >= E + 1, "moe_gemm_tc05: a [P, K], w [E, N, K], out [P, N] (glu_limited: [P, N / 2])")
     _need(moe_gemm_grouped_ok(a, w, out, P, act), "moe_gemm_tc05: bf16, at least 128 places, K a multiple of 8, aligned rows")
     f = _fn("gemm_tc05", "si_gemm_tc05_grouped", [_c_p, _c_ll, _c_p, _c_p, _c_ll, _c_int, _c_p, _c_int, _c_int, _c_int, _c_int,
-                                                  _c_int, _c_f, _c_f, _c_p, _c_p])
+                                                  _c_int, _c_f, _c_f, _c_f, _c_p, _c_p])
     _check(f(_ptr(a), a.stride(0), _weight_map(w.view(E * N, K)), _ptr(out), out.stride(0), _dt(out), _ptr(offsets), P, E, N, K,
-             _GROUPED_TC05_ACTS[act], float(limit), float(alpha), _ptr(status), _stream()), f"moe_gemm_tc05(experts={E}, N={N}, K={K})")
+             _GROUPED_TC05_ACTS[act], float(limit), float(alpha), float(shift), _ptr(status), _stream()), f"moe_gemm_tc05(experts={E}, N={N}, K={K})")
 
 
-def moe_gemm_tiles(a, a_rows, w, out, offsets, act: str = "none", limit: float = 0.0, alpha: float = 1.702) -> None:
+def moe_gemm_tiles(a, a_rows, w, out, offsets, act: str = "none", limit: float = 0.0, alpha: float = 1.702,
+                  shift: float = 1.0) -> None:
     """``moe_gemm`` on the mma.sync tiles (bf16) or in true 32-bit, whatever the number of places."""
     _cuda(a, a_rows, w, out, offsets)
     _i32(a_rows, "a_rows"); _i32(offsets, "offsets")
@@ -1678,27 +1818,28 @@ def moe_gemm_tiles(a, a_rows, w, out, offsets, act: str = "none", limit: float =
           "moe_gemm: out must be [P, N] (glu_limited: [P, N / 2])")
     _need(offsets.numel() >= E + 1 and (a_rows is None or a_rows.numel() == P) and (a_rows is not None or a.shape[0] >= P), "moe_gemm: sizes")
     f = _fn("moe", "si_moe_gemm", [_c_p, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_ll, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                   _c_f, _c_f, _c_p])
+                                   _c_f, _c_f, _c_f, _c_p])
     _check(f(_ptr(a), _dt(a), a.stride(0), _ptr(a_rows), _ptr(w), _ptr(out), _dt(out), out.stride(0), _ptr(offsets), P, E, N, K,
-             MOE_ACTS[act], float(limit), float(alpha), _stream()), f"moe_gemm(experts={E}, N={N}, K={K})")
+             MOE_ACTS[act], float(limit), float(alpha), float(shift), _stream()), f"moe_gemm(experts={E}, N={N}, K={K})")
 
 
 def moe_gemm(a, a_rows, w, out, offsets, act: str = "none", gathered=None, status=None, limit: float = 0.0,
-             alpha: float = 1.702) -> None:
+             alpha: float = 1.702, shift: float = 1.0) -> None:
     """out[p, :] = act(a[row(p), :] @ w[e]^T) for every place p of expert e (``offsets`` int32 [E + 1] as ``moe_plan``
     leaves them); row(p) = a_rows[p] (int32 [P]) or p itself (None). ``a`` [*, K] and ``w`` [E, N, K] of one dtype;
     ``out`` [P, N] in that dtype or fp32. bf16 on the tensor cores with fp32 sums (tcgen05 where ``moe_gemm_grouped_ok``;
     a product that gathers then copies its rows into ``gathered`` [P, K] first), fp32 in true 32-bit. ``offsets`` may hold
     more entries than E + 1 (experts behind the E that have weights, which get no product); places behind offsets[E] are
-    left alone. act "glu_limited": ``w`` holds gate and up rows in turn and ``out`` is [P, N / 2] (``limit``, ``alpha``)."""
+    left alone. act "glu_limited": ``w`` holds gate and up rows in turn and ``out`` is [P, N / 2]
+    (``limit``, ``alpha``, ``shift``: g sigmoid(alpha g) (u + shift) of the limited sums)."""
     P = out.shape[0]
     if moe_gemm_grouped_ok(a, w, out, P, act) and (a_rows is None or gathered is not None):
         if a_rows is not None:
             moe_gather(a, a_rows, gathered)
             a = gathered
-        moe_gemm_tc05(a[:P], w, out, offsets, act, status, limit, alpha)
+        moe_gemm_tc05(a[:P], w, out, offsets, act, status, limit, alpha, shift)
     else:
-        moe_gemm_tiles(a, a_rows, w, out, offsets, act, limit, alpha)
+        moe_gemm_tiles(a, a_rows, w, out, offsets, act, limit, alpha, shift)
 
 
 def moe_combine(y, place_of, wts, out, shared=None, gate=None, ids=None, real: int = 0, x=None) -> None:
@@ -1786,14 +1927,17 @@ def stream_norm(src, weight, eps: float, out, streams: int, dst=None, y=None, mi
 
 def qkv_conv(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, block_table, k_cache, v_cache, page_size: int,
              num_seqs: int, NQ: int, NK: int, NV: int, dk: int, dv: int, q_out, norm: bool, eps: float, q_weight=None,
-             k_weight=None, portions: int = 3, status=None) -> None:
+             k_weight=None, portions: int = 3, status=None, inv_freq=None, rot_dims: int = 0) -> None:
     """Rows ``u`` = [q: NQ*dk | k: NK*dk | v: NV*dv | ...] of a stacked projection, plus ``bias`` (fp32 [C] or None), through a
     causal convolution over time per channel (``taps`` fp32 [K, C]; zeros before the sequence), then with ``norm`` every q and
     k vector scaled to a root mean square of one (times ``q_weight`` / ``k_weight``, fp32 [dk], where given); q into ``q_out``
     [T, NQ*dk], k and v into their pages (``k_cache`` None: the queries alone are kept). ``state`` (fp32 [slots, >= (K-1)*C];
     None for K = 1) holds each request's last K - 1 values of every channel and is renewed. ``portions``: what the step
     holds beside sequences of one row: 1 portions of several rows from position 0, 2 such portions from a later position (a second
-    launch), 3 both, 0 neither."""
+    launch), 3 both, 0 neither. ``inv_freq`` (fp32 [rot_dims / 2]): before the norm the neighbouring pairs (2i, 2i + 1) of the first ``rot_dims``
+    entries of every q and k vector are turned by position * inv_freq[i]."""
+    _need(inv_freq is None or (inv_freq.is_cuda and rot_dims % 2 == 0 and 0 <= rot_dims <= dk), "qkv_conv: rot_dims must be even and at most dk")
+    _f32v(inv_freq, "inv_freq", rot_dims // 2)
     _cuda(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, block_table, k_cache, v_cache, q_out, q_weight, k_weight, status)
     for t, nm in ((positions, "positions"), (row_seq, "row_seq"), (q_start, "q_start"), (ctx_len, "ctx_len"), (slots, "slots"),
                   (block_table, "block_table")):
@@ -1813,11 +1957,43 @@ def qkv_conv(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, 
               and tuple(v_cache.shape) == (k_cache.shape[0], NV, page_size, dv), "qkv_conv: values must be [pages, NV, page_size, dv]")
     f = _fn("qkv_conv", "si_qkv_conv",
             [_c_p, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_p, _c_p, _c_int, _c_int,
-             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_f, _c_int, _c_p, _c_p, _c_p])
+             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p, _c_ll, _c_int, _c_p, _c_p, _c_f, _c_p, _c_int, _c_int,
+             _c_p, _c_p, _c_p])
     launches = ctypes.c_int(1)
     _check(f(_ptr(u), _dt(u), u.stride(0), _ptr(bias), _ptr(taps), _ptr(state), state.stride(0) if state is not None else 0,
              _ptr(positions), _ptr(row_seq), _ptr(q_start), _ptr(ctx_len), _ptr(slots), _ptr(block_table),
              block_table.shape[1] if block_table is not None else 0, _ptr(k_cache), _ptr(v_cache),
              k_cache.shape[0] if k_cache is not None else 0, page_size, T, num_seqs, NQ, NK, NV, dk, dv, K, _ptr(q_out),
-             q_out.stride(0), 1 if norm else 0, _ptr(q_weight), _ptr(k_weight), float(eps), int(portions), ctypes.addressof(launches),
+             q_out.stride(0), 1 if norm else 0, _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(inv_freq), int(rot_dims), int(portions), ctypes.addressof(launches),
              _ptr(status), _stream()), f"qkv_conv(dk={dk}, dv={dv}, taps={K})", kernels=launches.value)
+
+
+def conv_rows(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, num_seqs: int, NQ: int, NK: int, NV: int, dk: int, dv: int,
+              out, unit: bool = False, eps: float = 1e-6, q_scale: float = 1.0, silu: bool = False, out_bias=None, copy=None,
+              portions: int = 3, status=None) -> None:
+    """The convolution of ``qkv_conv`` in front of a recurrence: the same rows ``u`` (+ ``bias``), ``taps`` and ``state``, then (+ ``out_bias``,
+    fp32 [C]), silu where asked, and with ``unit`` every q and k vector made a unit vector (x * rsqrt(sum(x^2) + eps), q times ``q_scale``).
+    Everything goes into ``out`` fp32 [T, C]. ``copy`` [NQ + NK + NV, T, size] in u's dtype (contiguous, size at least a vector's): a
+    second copy vector by vector, for products of a matrix per vector."""
+    _cuda(u, bias, taps, state, positions, row_seq, q_start, ctx_len, slots, out, out_bias, copy, status)
+    for t, nm in ((positions, "positions"), (row_seq, "row_seq"), (q_start, "q_start"), (ctx_len, "ctx_len"), (slots, "slots")):
+        _i32(t, nm)
+    T = u.shape[0]
+    C = (NQ + NK) * dk + NV * dv
+    K = taps.shape[0]
+    _need(u.stride(1) == 1 and u.shape[1] >= C and tuple(taps.shape) == (K, C), "conv_rows: u must hold C channels, taps [K, C]")
+    _f32v(taps, "taps"); _f32v(bias, "bias", C); _f32v(out_bias, "out_bias", C)
+    _need(out.dtype == torch.float32 and out.stride(1) == 1 and tuple(out.shape) == (T, C), "conv_rows: out must be fp32 [T, C]")
+    _need(K == 1 or (state is not None and state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
+                     and state.shape[1] >= (K - 1) * C), "conv_rows: state must be fp32 [slots, >= (K-1)*C]")
+    _need(copy is None or (copy.dtype == u.dtype and copy.is_contiguous() and tuple(copy.shape[:2]) == (NQ + NK + NV, T)
+                           and copy.shape[2] >= max(dk if NQ + NK else 0, dv if NV else 0)), "conv_rows: copy must be [vectors, T, size] in u's dtype")
+    f = _fn("qkv_conv", "si_conv_rows",
+            [_c_p, _c_int, _c_ll, _c_p, _c_p, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+             _c_int, _c_int, _c_p, _c_ll, _c_int, _c_f, _c_f, _c_int, _c_p, _c_p, _c_ll, _c_int, _c_int, _c_p, _c_p, _c_p])
+    launches = ctypes.c_int(1)
+    _check(f(_ptr(u), _dt(u), u.stride(0), _ptr(bias), _ptr(taps), _ptr(state), state.stride(0) if state is not None else 0,
+             _ptr(positions), _ptr(row_seq), _ptr(q_start), _ptr(ctx_len), _ptr(slots), T, num_seqs, NQ, NK, NV, dk, dv, K, _ptr(out),
+             out.stride(0), 1 if unit else 0, float(eps), float(q_scale), 1 if silu else 0, _ptr(out_bias), _ptr(copy),
+             copy.stride(0) if copy is not None else 0, copy.shape[2] if copy is not None else 0, int(portions),
+             ctypes.addressof(launches), _ptr(status), _stream()), f"conv_rows(channels={C}, taps={K})", kernels=launches.value)

@@ -10,7 +10,15 @@
 // portion starts from them (from zeros at position 0) and leaves its own behind, so a sequence may be cut anywhere. The slot
 // of a sequence that brings one row (decode) is renewed by the threads that read it, that of a sequence from its start by the
 // threads of its last row (nobody reads the old values); the other portions' by a second small launch, since other blocks
-// read the old values. All arithmetic is fp32.
+// read the old values.// All arithmetic is fp32.
+//
+// Two further forms:
+//   rotation  q and k are turned by their row's position between the convolution and the norm: the neighbouring pairs (2i, 2i + 1) of
+//             a vector's first `rot_dims` entries by position * inv_freq[i]. A block makes the sines of the rows at hand once, in
+//             shared memory, for all of its vectors.
+//   rows      (what stands before a recurrence) y <- silu(y + out_bias) where asked, q and k unit vectors, y * rsqrt(sum(y^2) + eps)
+//             (q times `q_scale`), and everything goes into fp32 rows [T, C] instead of `q_out` and pages; a second copy in
+//             the compute dtype, vector by vector [vector][T][copy_size], feeds a product per vector.
 //
 // The fast kernel: a thread holds eight neighbouring channels (16 bytes of bfloat16) with their taps, their last K - 1
 // inputs and their bias in registers and walks a few dozen rows (prompts; one row in decode steps), so that every input and
@@ -28,6 +36,10 @@ struct ConvArgs {
   int num_pages, page_size, num_tokens, num_seqs, NQ, NK, NV, dk, dv, C, K;
   void* q_out; long long q_out_stride;
   int norm; const float* q_w; const float* k_w; float eps;
+  const float* inv_freq; int rot_dims;                   // rotation: fp32 [rot_dims / 2] or null
+  float* rows_out; long long rows_stride;                // rows: fp32 [T, C] or null
+  int silu; const float* out_bias; float q_scale;        // rows only
+  void* copy; long long copy_vec; int copy_size;         // rows only: entries between vectors and between rows of the copy, or null
   int lanes_qk, rows_per_block, trigger;                 // fast kernel: lanes a q or k vector, rows a block walks
   int state_from_start;                                  // second launch: portions from position 0 as well (plain kernel)
   int* status;
@@ -80,17 +92,22 @@ struct ConvRow {
 #define CONV_FROM_START 1
 #define CONV_CONTINUED 2
 #define CONV_ROWS 128                                    // most rows a block walks
+#define CONV_PLAIN 0                                     // forms of the fast kernel
+#define CONV_ROTATE 1
+#define CONV_TO_ROWS 2
+#define CONV_MAX_PAIRS 128                               // rotation in the fast kernel: pairs of a vector (of 256 entries at most)
 
 // R: 1 (a block has one row) or 4 (it walks rows_per_block rows, the loads of four of them in flight together). The last
 // values of the thread's channels stand in a ring of four, the row's place in it being a compile-time number, in pairs for
 // the packed fp32 instructions.
-template <typename T, int K, int R>
+template <typename T, int K, int R, int FORM>
 __global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) {
   static_assert(K >= 1 && K <= 4 && (R == 1 || R == 4), "");
   constexpr int PACK = (int)sizeof(T) / 2;               // 16-byte pieces that hold eight channels
   constexpr bool STAGED = R > 1 && PACK == 1;            // rows come through shared memory, four rows ahead of the sums
   __shared__ ConvRow rows[R == 1 ? 1 : CONV_ROWS];
   __shared__ uint4 stage[STAGED ? 2 * R * 256 : 1];      // [half][row][thread]: every thread reads what it fetched itself
+  __shared__ float2 turn[FORM == CONV_ROTATE ? 2 * R * CONV_MAX_PAIRS : 1];      // [half][row][pair]: cosine and sine
   const int lane = threadIdx.x & 31;
   const int id = blockIdx.y * blockDim.x + threadIdx.x;
   // threads of the q and k vectors first (lanes_qk each, those beyond dk / 8 idle), then one for every 8 channels of v
@@ -157,6 +174,10 @@ __global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) 
 #pragma unroll
     for (int e = 0; e < 4; ++e) v[e] = make_float2(f[2 * e], f[2 * e + 1]);
   };
+  float2 ob[4];                                          // what is added behind the convolution
+#pragma unroll
+  for (int e = 0; e < 4; ++e) ob[e] = make_float2(0.f, 0.f);
+  if (FORM == CONV_TO_ROWS && p.out_bias && on) load_pairs(p.out_bias + c, ob);
   // row r of the four at hand: its values join the ring, y = the convolution; returns the sum of y^2
   auto sums = [&](int r, int half, const uint4* raw, float2 (&y)[4]) {
     float2 (&x)[4] = ring[r & 3];
@@ -173,13 +194,32 @@ __global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) 
       y[e] = __fmul2_rn(w[0][e], ring[(r - K + 1) & 3][e]);
 #pragma unroll
       for (int j = 1; j < K; ++j) y[e] = __ffma2_rn(w[j][e], ring[(r - K + 1 + j) & 3][e], y[e]);
+      if (FORM == CONV_TO_ROWS) {
+        y[e] = __fadd2_rn(y[e], ob[e]);
+        if (p.silu) y[e] = make_float2(y[e].x / (1.f + expf(-y[e].x)), y[e].y / (1.f + expf(-y[e].y)));
+      }
       s2 = __ffma2_rn(y[e], y[e], s2);
     }
     return s2.x + s2.y;
   };
-  const float inv_dk = 1.f / (float)p.dk;
+  // rows take the sum of the squares, the other forms their mean
+  const float inv_dk = FORM == CONV_TO_ROWS ? 1.f : 1.f / (float)p.dk;
+  const float after = FORM == CONV_TO_ROWS && is_q ? p.q_scale : 1.f;
+  const int pairs = FORM == CONV_ROTATE ? p.rot_dims / 2 : 0;
+  auto turn_row = [&](int half, int r, float2 (&y)[4]) {       // row r of the four at hand
+    if constexpr (FORM == CONV_ROTATE) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int i = off / 2 + e;
+        if (!is_v && i < pairs) {
+          const float2 cs = turn[(half * R + r) * CONV_MAX_PAIRS + i];
+          y[e] = make_float2(y[e].x * cs.x - y[e].y * cs.y, y[e].y * cs.x + y[e].x * cs.y);
+        }
+      }
+    }
+  };
   auto normalise = [&](float ss, float2 (&y)[4]) {       // ss: over the whole vector
-    const float inv = rsqrtf(fmaf(ss, inv_dk, p.eps));
+    const float inv = rsqrtf(fmaf(ss, inv_dk, p.eps)) * after;
 #pragma unroll
     for (int e = 0; e < 4; ++e) y[e] = __fmul2_rn(y[e], make_float2(inv, inv));
     if (gw && on) {
@@ -196,6 +236,12 @@ __global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) 
   if (kv) kv += (long long)head * p.page_size * size + off;
   auto put = [&](int i, const float2 (&y)[4]) {
     T* dst;
+    if (FORM == CONV_TO_ROWS) {
+      const float v[8] = {y[0].x, y[0].y, y[1].x, y[1].y, y[2].x, y[2].y, y[3].x, y[3].y};
+      store8<float>(p.rows_out + (size_t)(t0 + i) * p.rows_stride + c, v);
+      if (p.copy) store8<T>((T*)p.copy + ((is_v ? p.NQ + p.NK : 0) + vec) * p.copy_vec + (size_t)(t0 + i) * p.copy_size + off, v);
+      return;
+    }
     if (is_q) {
       dst = qo + (size_t)i * p.q_out_stride;
     } else {
@@ -218,6 +264,17 @@ __global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) 
   for (int i0 = 0; i0 < nrows; i0 += R) {
     uint4 raw[STAGED ? 1 : R * PACK];                    // the thread's channels of R rows
     const int half = (i0 / R) & 1;
+    if constexpr (FORM == CONV_ROTATE) {                 // the rows' sines; the other half is still being read by slower warps
+      for (int idx = threadIdx.x; idx < R * pairs; idx += blockDim.x) {
+        const int r = idx / pairs, i = idx - r * pairs;
+        if (i0 + r < nrows) {
+          float sn, cs;
+          sincosf((float)rows[i0 + r].pos * p.inv_freq[i], &sn, &cs);
+          turn[(half * R + r) * CONV_MAX_PAIRS + i] = make_float2(cs, sn);
+        }
+      }
+      __syncthreads();
+    }
     if (STAGED) {
       fetch(i0 + R, half ^ 1);
       asm volatile("cp.async.wait_group 1;\n" ::: "memory");      // the rows at i0 have arrived
@@ -241,6 +298,8 @@ __global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) 
           if (on) {
             s0 = sums(r, half, raw, y0);
             s1 = sums(r + 1, half, raw, y1);
+            turn_row(half, r, y0);
+            turn_row(half, r + 1, y1);
           }
           if (norm) {
             for (int o = 1; o < p.lanes_qk; o <<= 1) {
@@ -290,6 +349,7 @@ __global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) 
       float ss = 0.f;
       if (on) {
         ss = sums(r, half, raw, y);
+        turn_row(half, r, y);
         if (K > 1 && rows[i].leaves) {                   // nobody else reads or writes its slot in this launch
 #pragma unroll
           for (int d = 0; d < K - 1; ++d) {
@@ -309,7 +369,7 @@ __global__ void __launch_bounds__(256, 2) qkv_conv_vec_kernel(const ConvArgs p) 
   }
 }
 
-template <typename T, int R>
+template <typename T, int R, int FORM>
 static void conv_launch_vec(ConvArgs& p, int yb, int threads, cudaStream_t stream) {
   p.rows_per_block = 1;
   if (R > 1) {                                           // as many rows as let all blocks run at once (two a multiprocessor)
@@ -320,10 +380,10 @@ static void conv_launch_vec(ConvArgs& p, int yb, int threads, cudaStream_t strea
   const dim3 grid((p.num_tokens + p.rows_per_block - 1) / p.rows_per_block, yb);
   p.trigger = si_pdl_trigger_mode((long long)grid.x * grid.y, 2LL * si_sm_count()) == 1;
   switch (p.K) {
-    case 1: si_launch(qkv_conv_vec_kernel<T, 1, R>, grid, dim3(threads), 0, stream, p); break;
-    case 2: si_launch(qkv_conv_vec_kernel<T, 2, R>, grid, dim3(threads), 0, stream, p); break;
-    case 3: si_launch(qkv_conv_vec_kernel<T, 3, R>, grid, dim3(threads), 0, stream, p); break;
-    default: si_launch(qkv_conv_vec_kernel<T, 4, R>, grid, dim3(threads), 0, stream, p); break;
+    case 1: si_launch(qkv_conv_vec_kernel<T, 1, R, FORM>, grid, dim3(threads), 0, stream, p); break;
+    case 2: si_launch(qkv_conv_vec_kernel<T, 2, R, FORM>, grid, dim3(threads), 0, stream, p); break;
+    case 3: si_launch(qkv_conv_vec_kernel<T, 3, R, FORM>, grid, dim3(threads), 0, stream, p); break;
+    default: si_launch(qkv_conv_vec_kernel<T, 4, R, FORM>, grid, dim3(threads), 0, stream, p); break;
   }
 }
 
@@ -353,16 +413,28 @@ __global__ void __launch_bounds__(128) qkv_conv_kernel(const ConvArgs p) {
       const float x = d <= back ? to_f32<T>(u[(size_t)(t - d) * p.u_stride + c]) + b : st[(size_t)(K - 1 - (d - back)) * p.C + c];
       y = fmaf(p.w[(size_t)j * p.C + c], x, y);
     }
-    return y;
+    if (p.out_bias) y += p.out_bias[c];
+    return p.silu ? y / (1.f + expf(-y)) : y;
+  };
+  // entry i of this warp's vector, turned where the vector is a query or key and the entry lies among those that are
+  auto entry = [&](int i) {
+    const float y = value(c0 + i);
+    if (is_v || !p.inv_freq || i >= p.rot_dims) return y;
+    const float other = value(c0 + (i ^ 1));
+    float sn, cs;
+    sincosf((float)pos * p.inv_freq[i / 2], &sn, &cs);
+    return (i & 1) ? y * cs + other * sn : y * cs - other * sn;
   };
   float inv = 1.f;
   if (!is_v && p.norm) {
     float ss = 0.f;
     for (int i = lane; i < size; i += 32) { const float y = value(c0 + i); ss = fmaf(y, y, ss); }
-    inv = rsqrtf(warp_sum(ss) / (float)size + p.eps);
+    inv = p.rows_out ? rsqrtf(warp_sum(ss) + p.eps) * (vec < p.NQ ? p.q_scale : 1.f) : rsqrtf(warp_sum(ss) / (float)size + p.eps);
   }
   T* dst = nullptr;
-  if (!is_v && vec < p.NQ) {
+  if (p.rows_out) {
+    // nothing but the rows
+  } else if (!is_v && vec < p.NQ) {
     dst = (T*)p.q_out + (size_t)t * p.q_out_stride + c0;
   } else if (p.k_cache) {
     const long long page = conv_page(p, seq, pos, lane == 0);
@@ -372,14 +444,27 @@ __global__ void __launch_bounds__(128) qkv_conv_kernel(const ConvArgs p) {
   }
   const float* gw = (is_v || !p.norm) ? nullptr : (vec < p.NQ ? p.q_w : p.k_w);
   const bool alone = p.q_start[seq + 1] - start == 1;
+  // a turned entry reads its neighbour's past, so the slot moves on only when all of them have been formed
+  const bool two = alone && K > 1 && p.inv_freq && !is_v;
   for (int i = lane; i < size; i += 32) {
-    const float y = value(c0 + i) * inv;
+    const float y = entry(i) * inv;
+    if (p.rows_out) {
+      p.rows_out[(size_t)t * p.rows_stride + c0 + i] = y;
+      if (p.copy) ((T*)p.copy)[vec * p.copy_vec + (size_t)t * p.copy_size + i] = from_f32<T>(y);
+    }
     if (dst) dst[i] = from_f32<T>(gw ? y * gw[i] : y);
-    if (alone && K > 1) {                                // the slot moves on by one row (this lane alone reads this channel)
+    if (alone && K > 1 && !two) {                        // the slot moves on by one row (this lane alone reads this channel)
       float* sc = st + c0 + i;
       for (int j = 0; j + 1 < K - 1; ++j) sc[(size_t)j * p.C] = pos > 0 ? sc[(size_t)(j + 1) * p.C] : 0.f;
       sc[(size_t)(K - 2) * p.C] = to_f32<T>(u[(size_t)t * p.u_stride + c0 + i]) + (p.bias ? p.bias[c0 + i] : 0.f);
     }
+  }
+  if (!two) return;
+  __syncwarp();
+  for (int i = lane; i < size; i += 32) {
+    float* sc = st + c0 + i;
+    for (int j = 0; j + 1 < K - 1; ++j) sc[(size_t)j * p.C] = pos > 0 ? sc[(size_t)(j + 1) * p.C] : 0.f;
+    sc[(size_t)(K - 2) * p.C] = to_f32<T>(u[(size_t)t * p.u_stride + c0 + i]) + (p.bias ? p.bias[c0 + i] : 0.f);
   }
 }
 
@@ -421,6 +506,8 @@ static int conv_launch(ConvArgs p, int portions, int* launches, cudaStream_t str
   bool vec = p.K <= 4 && p.dk % 8 == 0 && p.dk <= 256 && (p.NV == 0 || p.dv % 8 == 0) && p.u_stride % elem == 0 &&
              p.q_out_stride % elem == 0 && p.state_stride % 4 == 0 && al(p.u) && al(p.bias) && al(p.w) && al(p.state) && al(p.k_cache) &&
              al(p.v_cache) && al(p.q_out) && al(p.q_w) && al(p.k_w);
+  const int form = p.rows_out ? CONV_TO_ROWS : p.inv_freq ? CONV_ROTATE : CONV_PLAIN;
+  if (form == CONV_TO_ROWS) vec = vec && al(p.rows_out) && p.rows_stride % 4 == 0 && al(p.out_bias) && al(p.copy) && p.copy_vec % elem == 0 && p.copy_size % elem == 0;
   if (vec) {
     p.lanes_qk = 1;
     while (p.lanes_qk * 8 < p.dk) p.lanes_qk *= 2;
@@ -428,8 +515,17 @@ static int conv_launch(ConvArgs p, int portions, int* launches, cudaStream_t str
     const int threads = want <= 128 ? 128 : 256;
     const int yb = (int)((want + threads - 1) / threads);
     // a row a block while all of them run at once, else several rows whose loads overlap
-    if ((long long)p.num_tokens * yb <= 2LL * si_sm_count()) conv_launch_vec<T, 1>(p, yb, threads, stream);
-    else conv_launch_vec<T, 4>(p, yb, threads, stream);
+    const bool few = (long long)p.num_tokens * yb <= 2LL * si_sm_count();
+    if (form == CONV_TO_ROWS) {
+      if (few) conv_launch_vec<T, 1, CONV_TO_ROWS>(p, yb, threads, stream);
+      else conv_launch_vec<T, 4, CONV_TO_ROWS>(p, yb, threads, stream);
+    } else if (form == CONV_ROTATE) {
+      if (few) conv_launch_vec<T, 1, CONV_ROTATE>(p, yb, threads, stream);
+      else conv_launch_vec<T, 4, CONV_ROTATE>(p, yb, threads, stream);
+    } else {
+      if (few) conv_launch_vec<T, 1, CONV_PLAIN>(p, yb, threads, stream);
+      else conv_launch_vec<T, 4, CONV_PLAIN>(p, yb, threads, stream);
+    }
   } else {
     const dim3 grid(p.num_tokens, (p.NQ + p.NK + p.NV + 3) / 4);
     si_launch(qkv_conv_kernel<T>, grid, dim3(128), 0, stream, p);
@@ -443,22 +539,58 @@ static int conv_launch(ConvArgs p, int portions, int* launches, cudaStream_t str
   return si_last_error();
 }
 
+static bool conv_sizes_ok(const ConvArgs& p, long long C) {
+  return p.NQ >= 0 && p.NK >= 0 && p.NV >= 0 && p.dk > 0 && p.dv >= 0 && p.K >= 1 && p.num_seqs <= 65535 && !(p.K > 1 && !p.state) &&
+         C <= (1LL << 30) && !(p.K > 1 && p.state_stride < (long long)(p.K - 1) * C);
+}
+
 // `portions`: what the step holds beside sequences of one row: 1 portions of several rows that begin at position 0, 2 such
 // portions that begin later, 3 both (or not known); 0 neither (a decode step). `launches` (may be null): kernels launched.
+// `inv_freq` (fp32 [rot_dims / 2], may be null): q and k are turned in neighbouring pairs before the norm.
 // Returns 0, a CUDA error code, or -2 (size refused).
 SI_EXPORT int si_qkv_conv(const void* u, int dtype, long long u_stride, const float* bias, const float* w, float* state,
                           long long state_stride, const int* positions, const int* row_seq, const int* q_start,
                           const int* ctx_len, const int* slots, const int* block_table, int table_width, void* k_cache,
                           void* v_cache, int num_pages, int page_size, int num_tokens, int num_seqs, int NQ, int NK, int NV,
                           int dk, int dv, int K, void* q_out, long long q_out_stride, int norm, const float* q_w,
-                          const float* k_w, float eps, int portions, int* launches, int* status, cudaStream_t stream) {
+                          const float* k_w, float eps, const float* inv_freq, int rot_dims, int portions, int* launches, int* status,
+                          cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
-  if (NQ < 0 || NK < 0 || NV < 0 || dk <= 0 || dv < 0 || K < 1 || num_seqs > 65535 || (K > 1 && !state)) return -2;
-  if ((NK > 0 || NV > 0) && k_cache && (!block_table || page_size <= 0 || (NV > 0 && !v_cache))) return -2;
   const long long C = (long long)(NQ + NK) * dk + (long long)NV * dv;
-  if (C > (1LL << 30) || state_stride < (long long)(K - 1) * C) return -2;
-  ConvArgs p{u, u_stride, bias, w, state, state_stride, positions, row_seq, q_start, ctx_len, slots, block_table, table_width,
-             k_cache, v_cache, num_pages, page_size, num_tokens, num_seqs, NQ, NK, NV, dk, dv, (int)C, K, q_out, q_out_stride,
-             norm, q_w, k_w, eps, 1, 1, 0, 0, status};
+  if ((NK > 0 || NV > 0) && k_cache && (!block_table || page_size <= 0 || (NV > 0 && !v_cache))) return -2;
+  if (inv_freq && (rot_dims < 0 || rot_dims % 2 || rot_dims > dk)) return -2;
+  ConvArgs p = {};
+  p.u = u; p.u_stride = u_stride; p.bias = bias; p.w = w; p.state = state; p.state_stride = state_stride;
+  p.positions = positions; p.row_seq = row_seq; p.q_start = q_start; p.ctx_len = ctx_len; p.slots = slots;
+  p.block_table = block_table; p.table_width = table_width; p.k_cache = k_cache; p.v_cache = v_cache;
+  p.num_pages = num_pages; p.page_size = page_size; p.num_tokens = num_tokens; p.num_seqs = num_seqs;
+  p.NQ = NQ; p.NK = NK; p.NV = NV; p.dk = dk; p.dv = dv; p.C = (int)C; p.K = K; p.q_out = q_out; p.q_out_stride = q_out_stride;
+  p.norm = norm; p.q_w = q_w; p.k_w = k_w; p.eps = eps; p.inv_freq = rot_dims > 0 ? inv_freq : nullptr; p.rot_dims = rot_dims;
+  p.q_scale = 1.f; p.lanes_qk = 1; p.rows_per_block = 1; p.status = status;
+  if (!conv_sizes_ok(p, C)) return -2;
+  return dtype == SI_BF16 ? conv_launch<__nv_bfloat16>(p, portions, launches, stream) : conv_launch<float>(p, portions, launches, stream);
+}
+
+// The form that leaves fp32 rows (see the head of this file): rows_out [T, C]; `unit`: q and k become unit vectors
+// (x * rsqrt(sum(x^2) + eps), q times q_scale); `silu` and `out_bias` (fp32 [C], may be null) behind the convolution; `copy`
+// (may be null): vector v of row t at copy + v * copy_vec + t * copy_size, in the compute dtype.
+SI_EXPORT int si_conv_rows(const void* u, int dtype, long long u_stride, const float* bias, const float* w, float* state,
+                           long long state_stride, const int* positions, const int* row_seq, const int* q_start,
+                           const int* ctx_len, const int* slots, int num_tokens, int num_seqs, int NQ, int NK, int NV, int dk, int dv,
+                           int K, float* rows_out, long long rows_stride, int unit, float eps, float q_scale, int silu,
+                           const float* out_bias, void* copy, long long copy_vec, int copy_size, int portions, int* launches,
+                           int* status, cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  const long long C = (long long)(NQ + NK) * dk + (long long)NV * dv;
+  if (!rows_out || rows_stride < C) return -2;
+  ConvArgs p = {};
+  p.u = u; p.u_stride = u_stride; p.bias = bias; p.w = w; p.state = state; p.state_stride = state_stride;
+  p.positions = positions; p.row_seq = row_seq; p.q_start = q_start; p.ctx_len = ctx_len; p.slots = slots;
+  p.page_size = 1; p.num_tokens = num_tokens; p.num_seqs = num_seqs;
+  p.NQ = NQ; p.NK = NK; p.NV = NV; p.dk = dk; p.dv = dv; p.C = (int)C; p.K = K;
+  p.norm = unit; p.eps = eps; p.rows_out = rows_out; p.rows_stride = rows_stride; p.silu = silu; p.out_bias = out_bias;
+  p.q_scale = q_scale; p.copy = copy; p.copy_vec = copy_vec; p.copy_size = copy_size;
+  p.lanes_qk = 1; p.rows_per_block = 1; p.status = status;
+  if (!conv_sizes_ok(p, C)) return -2;
   return dtype == SI_BF16 ? conv_launch<__nv_bfloat16>(p, portions, launches, stream) : conv_launch<float>(p, portions, launches, stream);
 }

@@ -1,2 +1,2 @@
-from . import fevosun, llama, mivorax, nufasun, risizen, vibunex  # noqa: F401  (register "Fevosun", "LlamaForCausalLM", "Mivorax", "Nufasun", "Risizen", "Vibunex")
+from . import fevosun, llama, mivorax, nufasun, risizen, samulorn, vibunex  # noqa: F401  (register "Fevosun", "LlamaForCausalLM", "Mivorax", "Nufasun", "Risizen", "Samulorn", "Vibunex")
 from .model import Model

@@ -14,8 +14,9 @@ import torch
 
 from ..config.base import EmbedderSpec, ModelConfig, ModelSpec
 from ..csrc import ops
-from ..parts import Block, NormedDelta, StreamConnections, StreamDelta, SublayerGate, SummedDelta, embedder_class, feed_forward_class, mixer_class, norm_class, position_class
+from ..parts import Block, NormedDelta, StreamConnections, StreamDelta, SublayerGate, SummedDelta, TokenSideInput, embedder_class, feed_forward_class, mixer_class, norm_class, position_class
 from ..parts.linear import configure_library_gemm, linear
+from ..parts.norm import RMSNorm, add_to_stream
 from ..engine import tracing
 
 
@@ -57,7 +58,14 @@ class Model:
                 c1 = StreamConnections({"streams": self.spec.streams}, dtype, self.device)
                 if ffn is not None:
                     c2 = StreamConnections({"streams": self.spec.streams}, dtype, self.device)
-            self.blocks.append(Block(mixer, ffn, n1, n2, ls.arrangement, n1b, n2b, g1, g2, ls.residual_scale, c1, c2))
+            side = None                               # an input of the layer's own for each token
+            if ls.token_side_prefix is not None:
+                ts = self.spec.token_side
+                if ts is None or self.spec.streams is not None:
+                    raise ValueError("a layer's own token input needs the model's table of them and a single residual stream")
+                side = TokenSideInput({"hidden_size": self.spec.hidden_size, "dim": ts.dim, "index": len(self.blocks), "eps": ts.eps},
+                                      dtype, self.device)
+            self.blocks.append(Block(mixer, ffn, n1, n2, ls.arrangement, n1b, n2b, g1, g2, ls.residual_scale, c1, c2, side))
         if self.spec.streams is not None and self.spec.stream_adds:
             raise ValueError("additions between layers go with a single residual stream")
         # a scale on the logits is a gain of the final norm, so that it costs nothing and rounds nothing twice
@@ -100,6 +108,8 @@ class Model:
                 yield p + ls.feed_forward_gate_name, b.feed_forward_gate
             if b.mixer_streams is not None:
                 yield p + ls.mixer_streams_prefix, b.mixer_streams
+            if b.token_side is not None:
+                yield p + ls.token_side_prefix, b.token_side
             if b.feed_forward_streams is not None:
                 yield p + ls.feed_forward_streams_prefix, b.feed_forward_streams
             if b.feed_forward is not None:
@@ -121,6 +131,8 @@ class Model:
                 shapes[prefix + n] = tuple(s)
         for n, s in (self.spec.stream_vector_shapes or {}).items():
             shapes[n] = tuple(s)
+        if self.spec.token_side is not None:
+            shapes[self.spec.token_side.table_name] = (self.spec.vocab_size, len(self.blocks) * self.spec.token_side.dim)
         return shapes
 
     def optional_weights(self) -> List[str]:
@@ -156,6 +168,11 @@ class Model:
         for prefix, part in self._named_parts():
             part.load_weights({n: tensors[prefix + n] for n in part.weight_shapes()})
         self.stream_vectors = {n: tensors[n].float().contiguous() for n in (self.spec.stream_vector_shapes or {})}
+        if self.spec.token_side is not None:
+            table = tensors[self.spec.token_side.table_name].contiguous()
+            for b in self.blocks:
+                if b.token_side is not None:
+                    b.token_side.set_table(table)
         self.embed = self.embedder.table
         self.lm_head = self.embed if self.spec.tie_word_embeddings else tensors[self.spec.lm_head_name].contiguous()
 
@@ -238,6 +255,9 @@ class Model:
     @staticmethod
     def _stream_add(resid, delta, extra, vec) -> None:
         """``resid += delta (+ extra) (+ vec)`` in one launch; ``delta`` may be None, a tensor or a ``NormedDelta``."""
+        if isinstance(delta, NormedDelta) and not isinstance(delta.norm, RMSNorm):
+            add_to_stream(resid, delta)
+            delta = None
         if isinstance(delta, SummedDelta):
             ops.add_norm(resid, delta.a)
             ops.add_norm(resid, delta.b, extra=extra, vec=vec)

@@ -30,6 +30,9 @@ Options beyond the reference's block, all parameters of the part:
                    ``conv_suffix``, [channels, K], the last tap the current token's); the last K - 1 projected values of a request
                    are its state.
 ``qk_norm``        ``{"eps": e}``: every query and key head is scaled to a root mean square of one (after the convolution).
+``rot_interleaved`` the layer's rotary position encoding turns neighbouring pairs (2i, 2i + 1) of its first entries (in the launch behind the
+                   projection, between convolution and norm).
+``head_scale``     the heads' results are multiplied by it (their values are, in fp32, before they are stored).
 ``sink_score``     a number s: exp(s) joins every row's softmax denominator once, without a value.
 ``chunk``          positions fall into runs of so many, counted from position 0; a query sees keys of its own run alone.
 ``own_keys``       False: the layer has no key and value projections and reads the cache of another one (its spec's
@@ -67,6 +70,7 @@ MIN_TILES_PER_SPLIT = 2      # a split covers at least this many 64-key tiles
 
 class Attention(Mixer):
     adds_into_residual = True
+    folds_head_scale = True          # a pair of mixers passes this side's scale as a parameter
 
     def __init__(self, params, dtype, device, position=None):
         super().__init__(params, dtype, device, position)
@@ -112,7 +116,11 @@ class Attention(Mixer):
         self.qk_norm = qkn is not None
         self.qk_eps = float(qkn["eps"]) if self.qk_norm else 0.0
         self.own_keys = bool(params.get("own_keys", True))
-        self.prepared = self.biases or self.has_conv or self.qk_norm or not self.own_keys     # a launch behind the projection
+        self.rot_interleaved = bool(params.get("rot_interleaved", False))
+        self.head_scale = float(params.get("head_scale", 1.0))
+        # a launch behind the projection
+        self.prepared = self.biases or self.has_conv or self.qk_norm or not self.own_keys or self.rot_interleaved or self.head_scale != 1.0
+        self.head_width = self.H * self.vs
         # scores that the fast kernels know: q . k times the scale, a window or chunks, a sink
         self.plain_scores = (self.bias_spec is None and self.own_v and self.slopes is None and self.q_temp is None
                              and self.gate_name is None)
@@ -124,9 +132,14 @@ class Attention(Mixer):
         if self.prepared and (not self.own_v or self.gate_name is not None):
             raise ValueError("attention: values that are the keys and an output gate go without biases, convolution, query/key "
                              "norm and another layer's keys")
-        if self.general and position is not None:
+        self.rot = None                  # (inverse frequencies, entries turned), neighbouring pairs
+        if self.prepared and position is not None and self.rot_interleaved:
+            self.rot = position.rotary()
+            if self.rot is None or self.rot[1] > self.hs or getattr(position, "magnitude", 1.0) != 1.0:
+                raise ValueError("attention: rot_interleaved goes with a rotary position encoding of at most head_dim entries and magnitude 1")
+        elif self.general and position is not None:
             raise ValueError("attention: the general form (a distance bias, slopes, a value size of its own, values that are "
-                             "the keys, a query temperature, an output gate) goes without a position encoding")
+                             "the keys, a query temperature, an output gate) goes without a position encoding, or with rot_interleaved")
         # columns of the stacked projection: q, k, v (if the layer has values of its own), the gate (if it has one)
         self.kv_cols = self.KV * (self.hs + (self.vs if self.own_v else 0)) if self.own_keys else 0
         self.channels = self.H * self.hs + self.kv_cols
@@ -136,6 +149,7 @@ class Attention(Mixer):
         self.qkv = None
         self.qkv_bias = self.qkv_taps = None        # fp32 [channels], fp32 [taps, channels]
         self.o = None
+        self.stacked = False             # True: a pair of mixers makes this layer's projections with the other side's
 
     def _projections(self):
         """(name, rows) of the matrices in the stacked projection that biases and convolutions belong to."""
@@ -181,6 +195,8 @@ class Attention(Mixer):
             self.qkv_taps = stacked(self.conv_suffix).t().contiguous()
         elif self.prepared:                                  # one tap of one: the value itself
             self.qkv_taps = torch.ones(1, self.channels, dtype=torch.float32, device=parts[0].device)
+        if self.head_scale != 1.0:                           # linear in the values: the taps that make them carry the scale
+            self.qkv_taps[:, self.channels - self.KV * self.vs:] *= self.head_scale
         rows = sum(p.shape[0] for p in parts)
         if self.general and rows < self.proj_cols:           # rows of the product's result stay 16-byte aligned
             parts.append(torch.zeros(self.proj_cols - rows, self.hidden, dtype=parts[0].dtype, device=parts[0].device))
@@ -188,6 +204,23 @@ class Attention(Mixer):
         self.o = tensors[n["o"]].contiguous()
         if self.bias_spec is not None:
             self.dist_bias = spread_by_distance(tensors[self.bias_name].float(), self.bias_max)
+
+    # what a pair of mixers stacks: the input projection's rows, the output projection
+    @property
+    def input_weight(self):
+        return self.qkv if self.general else None
+
+    @input_weight.setter
+    def input_weight(self, w):
+        self.qkv = w
+
+    @property
+    def output_weight(self):
+        return self.o
+
+    @output_weight.setter
+    def output_weight(self, w):
+        self.o = w
 
     def cache_need(self):
         if not self.own_v:
@@ -299,13 +332,27 @@ class Attention(Mixer):
         return out
 
     def forward_general(self, x, ctx, cache):
-        """No rotation; keys (and values of their own size, where the layer has them) into the pages as they are, or behind
+        """Keys (and values of their own size, where the layer has them) into the pages as they are, or behind
         biases, convolution and norm; scores with the bias, the slopes and the query temperature, the sink in the denominator;
         the gate on the heads' results."""
         T = x.shape[0]
+        attn = ctx.buf("attn_out", (T, self.H * self.vs), self.dtype)
+        self.forward_heads(x, ctx, cache, attn)
+        out = ctx.buf("delta", (T, self.hidden), self.dtype)
+        linear(attn, self.o, out, ctx.status)
+        return out
+
+    def forward_heads(self, x, ctx, cache, attn, scale: float = 1.0, proj=None):
+        """The heads' results into ``attn`` [T, heads * value_dim] (a view with a row stride): everything but the output projection.
+        ``proj``: the input projection's result where the caller has made it."""
+        if not self.general or scale != 1.0:
+            raise ValueError("attention: heads before the output projection are the general form's; their scale is the parameter head_scale")
+        T = x.shape[0]
         H, KV, hs, vs = self.H, self.KV, self.hs, self.vs
-        qkv = ctx.buf("attn_qkv", (T, self.proj_cols), self.dtype)
-        linear(x, self.qkv, qkv, ctx.status)
+        qkv = proj
+        if qkv is None:
+            qkv = ctx.buf("attn_qkv", (T, self.proj_cols), self.dtype)
+            linear(x, self.qkv, qkv, ctx.status)
         v_cache = cache.v if self.own_v else None
         q = qkv[:, :H * hs]
         if self.prepared:
@@ -314,11 +361,11 @@ class Attention(Mixer):
             kv = KV if self.own_keys else 0
             ops.qkv_conv(qkv, self.qkv_bias, self.qkv_taps, cache.state, ctx.positions, ctx.row_seq, ctx.q_start, ctx.ctx_len,
                          ctx.slots, cache.block_table, cache.k if stores else None, cache.v if stores else None, cache.page_size,
-                         ctx.seq_slots, H, kv, kv, hs, vs, q, self.qk_norm, self.qk_eps, portions=_portions(ctx), status=ctx.status)
+                         ctx.seq_slots, H, kv, kv, hs, vs, q, self.qk_norm, self.qk_eps, portions=portions(ctx), status=ctx.status,
+                         inv_freq=None if self.rot is None else self.rot[0], rot_dims=0 if self.rot is None else self.rot[1])
         elif cache.writes:
             ops.kv_store(qkv, ctx.positions, ctx.row_seq, cache.block_table, cache.k, v_cache, cache.page_size,
                          ctx.seq_slots, H, KV, hs, vs if self.own_v else 0, status=ctx.status)
-        attn = ctx.buf("attn_out", (T, H * vs), self.dtype)
         gate = qkv[:, self.gate_off:self.gate_off + H * vs] if self.gate_name else None      # applied in the attention's epilogue
         if self.uses_fast(cache.page_size):
             self.attend(q, cache, ctx, attn)
@@ -339,9 +386,6 @@ class Attention(Mixer):
                                   cache.page_size, ctx.seq_slots, H, KV, hs, vs, self.scale, self.window or 0,
                                   dist_bias=self.dist_bias, sink=self.sink, status=ctx.status, slopes=self.slopes,
                                   q_temp=self.q_temp, gate=gate, chunk=self.chunk or 0)
-        out = ctx.buf("delta", (T, self.hidden), self.dtype)
-        linear(attn, self.o, out, ctx.status)
-        return out
 
     # ---- kernels ---------------------------------------------------------------------
     def target_blocks(self) -> int:
@@ -473,9 +517,9 @@ class Attention(Mixer):
             portion(q, cache.k, cache.v, cache.block_table, plan["por"], out, *args, status=ctx.status, **extra)
 
 
-def _portions(ctx) -> int:
-    """What the step holds beside sequences of one row, as ``ops.qkv_conv`` takes it: 1 portions from position 0, 2 portions
-    that go on, 3 both, 0 neither."""
+def portions(ctx) -> int:
+    """What the step holds beside sequences of one row, as ``ops.qkv_conv`` and ``ops.conv_rows`` take it: 1 portions from position 0,
+    2 portions that go on, 3 both, 0 neither."""
     if ctx.seq_cap is not None:                          # fixed shapes hold single rows
         return 0
     got = ctx.plans.get("portions")

@@ -98,9 +98,7 @@ class NormedDelta:
     bias: Optional[torch.Tensor] = None
 
     def value(self) -> torch.Tensor:
-        d = self.x.float() if self.bias is None else self.x.float() + self.bias
-        w = self.norm.weight.float()
-        return d * torch.rsqrt((d * d).mean(-1, keepdim=True) + self.norm.eps) * w
+        return self.norm.plain(self.x.float() if self.bias is None else self.x.float() + self.bias)
 
 
 @dataclass
@@ -194,6 +192,14 @@ class Norm(Part):
         """The norm on a residual stream of several copies (``resid`` [T, S, d]): do what ``delta`` leaves to be done,
         read the row that ``connections`` make of the streams (None: their sum) and normalise it into ``out``. With
         ``rows`` the streams stay as they are. Kinds that have no such form leave this unimplemented."""
+        raise NotImplementedError
+
+    def plain(self, x: torch.Tensor) -> torch.Tensor:
+        """The norm of fp32 rows in plain tensor operations (hooks and tests; no step runs through it)."""
+        raise NotImplementedError
+
+    def stream_norm(self):
+        """The norm as ``ops.stream_add`` takes it, for launches that combine norms of different kinds."""
         raise NotImplementedError
 
     def normalize(self, x: torch.Tensor, out: Optional[torch.Tensor] = None) -> None:

@@ -27,6 +27,8 @@ all of them and writes its result back into all of them through numbers of its o
     u = sum_s in1[s] x_s;  y = mixer(norm1(u));  x_t <- sum_s mix1[s, t] x_s + out1[t] y;  likewise the feed-forward
 ``resid`` is [T, S, d] then, and what a sublayer hands on is a ``StreamDelta``: the next norm's launch writes the streams,
 reads for its own sublayer and normalises.
+A block may also have an input of its own for each token (``TokenSideInput``), whatever the arrangement of a single stream: it
+adds the pending delta, reads the stream itself and hands its own result on as a ``NormedDelta``.
 Another arrangement (post-norm, ...) is added with ``register_arrangement`` and needs no change here.
 """
 from __future__ import annotations
@@ -39,6 +41,7 @@ from ..csrc import ops
 from .base import FeedForward, Mixer, Norm, NormedDelta, Part, StreamDelta, SummedDelta
 from .linear import linear
 from .streams import StreamConnections
+from .token_side import TokenSideInput
 
 _ARRANGEMENTS: Dict[str, Callable] = {}
 _CAPTURABLE: Dict[str, bool] = {}
@@ -99,7 +102,7 @@ class Block:
                  mixer_post_norm: Optional[Norm] = None, feed_forward_post_norm: Optional[Norm] = None,
                  mixer_gate: Optional[SublayerGate] = None, feed_forward_gate: Optional[SublayerGate] = None,
                  residual_scale: float = 1.0, mixer_streams: Optional[StreamConnections] = None,
-                 feed_forward_streams: Optional[StreamConnections] = None):
+                 feed_forward_streams: Optional[StreamConnections] = None, token_side: Optional[TokenSideInput] = None):
         self.mixer = mixer
         self.feed_forward = feed_forward
         self.mixer_norm = mixer_norm
@@ -111,12 +114,14 @@ class Block:
         self.residual_scale = float(residual_scale)
         self.mixer_streams = mixer_streams
         self.feed_forward_streams = feed_forward_streams
+        self.token_side = token_side
         self.arrangement = arrangement_name
         self._run = arrangement(arrangement_name)
         self.capturable = _CAPTURABLE[arrangement_name]
 
     def forward(self, resid: torch.Tensor, delta: Optional[torch.Tensor], ctx, cache) -> torch.Tensor:
-        return self._run(self, resid, delta, ctx, cache)
+        delta = self._run(self, resid, delta, ctx, cache)
+        return delta if self.token_side is None else self.token_side.forward(resid, delta, ctx)
 
     @staticmethod
     def norm(norm: Norm, resid, delta, out, ahead=None) -> None:

@@ -13,6 +13,10 @@ Further parameters:
                                g = min(W_gate,e x, limit), u = clamp(W_up,e x, -limit, limit), expert_e(x) = W_down,e (g sigmoid(alpha g) (u + 1));
                                gate and up rows are stacked in turn, and the first grouped product applies the activation to
                                each pair of neighbouring columns in its epilogue.
+``activation`` "silu_glu"      experts with a gate matrix: expert_e(x) = W_down,e (silu(W_gate,e x) * (W_up,e x)), laid out and run in the same way.
+``groups`` {"count", "keep"}   the experts fall into ``count`` equal runs of neighbours; only experts of the ``keep`` runs with the largest sum of
+                               their two best choice scores (s + bias) can be chosen.
+``renorm_eps``                 joins the chosen scores' sum that ``renorm`` divides by.
 ``choice_bias``                name of a vector [experts + identity]: the ``top`` largest of s + bias are chosen, the weights stay s.
 ``identity`` I                 the router has I more rows behind the experts'; a choice among them stands for an expert that returns
                                x itself (no tensors, no product: the combining kernel reads the row).
@@ -54,12 +58,24 @@ class RoutedMLP(FeedForward):
         self.choice_bias_name = p.get("choice_bias") or None
         self.limit = float(p.get("limit", 0.0) or 0.0)
         self.alpha = float(p.get("alpha", 1.702))
-        self.gated = self.activation == "glu_limited"
+        self.gated = self.activation in ("glu_limited", "silu_glu")
+        self.act, self.shift = self.activation, 1.0       # what the first grouped product's epilogue applies
+        if self.activation == "silu_glu":                 # the limited form without a limit: g sigmoid(g) (u + 0)
+            self.act, self.limit, self.alpha, self.shift = "glu_limited", float("inf"), 1.0, 0.0
+        gr = p.get("groups") or None
+        self.groups = None if gr is None else (int(gr["count"]), int(gr["keep"]))
+        self.renorm_eps = float(p.get("renorm_eps", 0.0) or 0.0)
+        if self.groups is not None:
+            count, keep = self.groups
+            if self.choice_bias_name is None or self.identity or count < 1 or self.E % count or not 1 <= keep <= count \
+                    or keep * (self.E // count) < self.top:
+                raise ValueError(f"routed_mlp: {count} groups of which {keep} are kept do not go with {self.E} experts and top {self.top}, or "
+                                 "without a choice bias, or with identity experts")
         if not 1 <= self.top <= min(self.routes, 32) or self.identity < 0:
             raise ValueError(f"routed_mlp: top {self.top} must be between 1 and min(experts + identity, 32)")
         if self.gated and not self.limit > 0:
             raise ValueError("routed_mlp: activation 'glu_limited' needs a positive limit")
-        if self.activation not in ops.MOE_ACTS or self.scores not in ops.MOE_SCORES:
+        if self.act not in ops.MOE_ACTS or self.scores not in ops.MOE_SCORES:
             raise ValueError(f"routed_mlp: activation {self.activation!r} or scores {self.scores!r} is not supported")
         sh = p.get("shared") or None
         self.shared = None
@@ -120,7 +136,7 @@ class RoutedMLP(FeedForward):
         gates = ctx.buf("moe_gates", (T, 1), torch.float32) if self.shared_gate else None
         R = self.routes                                           # experts with weights, then the identity experts
         ops.moe_route(x, self.w_route, R, top, self.scale, ids, wts, gates, scores=self.scores, renorm=self.renorm,
-                      choice_bias=self.choice_bias)
+                      choice_bias=self.choice_bias, renorm_eps=self.renorm_eps, groups=self.groups)
         scratch = ctx.buf("moe_plan", (ops.moe_plan_ints(P, R),), torch.int32)
         offsets = ctx.buf("moe_offsets", (R + 1,), torch.int32)
         row_of = ctx.buf("moe_row_of", (P,), torch.int32)
@@ -128,9 +144,9 @@ class RoutedMLP(FeedForward):
         ops.moe_plan(ids, R, scratch, offsets, row_of, place_of)
         # the places of the identity experts lie behind offsets[E]: the grouped products never reach them
         act = ctx.buf("moe_act", (P, self.inter), self.dtype)
-        gathered = ctx.buf("moe_x", (P, self.hidden), self.dtype) if ops.moe_gemm_grouped_ok(x, self.w_up, act, P, self.activation) else None
-        ops.moe_gemm(x, row_of, self.w_up, act, offsets, act=self.activation, gathered=gathered, status=ctx.status,
-                     limit=self.limit, alpha=self.alpha)
+        gathered = ctx.buf("moe_x", (P, self.hidden), self.dtype) if ops.moe_gemm_grouped_ok(x, self.w_up, act, P, self.act) else None
+        ops.moe_gemm(x, row_of, self.w_up, act, offsets, act=self.act, gathered=gathered, status=ctx.status,
+                     limit=self.limit, alpha=self.alpha, shift=self.shift)
         y = ctx.buf("moe_y", (P, self.hidden), torch.float32)
         ops.moe_gemm(act, None, self.w_down, y, offsets, status=ctx.status)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
