@@ -329,6 +329,27 @@ def _risizen_config(size="base"):
             "layers": layers}, {"attention": own, "feed_forward": mlp, "streams": 4}
 
 
+# ---- the Samulorn design beside the closest existing models ---------------------------------------------------
+# Sizes as the Vibunex section's (--design-size): three of four layers a delta rule with a decay per key channel (the Nufasun section's
+# heads at width 2,048: 16 of 128 x 128 over 8 query/key heads, four taps, rank 128), every fourth a pair of attention (the Llama twin's heads) and a
+# linear recurrence of the stream's width in parts of 128; feed-forwards dense and routed in turn, the routed ones with as many active
+# entries a token as the dense ones (4 experts, of groups of which half are kept); an input of 128 entries a layer and token.
+def _samulorn_config(size="base"):
+    width, ff, heads, kv, _, experts, eff, _ = _VIBUNEX_SIZES[size]
+    delta = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4, "rank": 128}
+    left = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "conv": 4, "scale": 128 ** 0.5,
+            "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    right = {"width": width, "blocks": width // 128, "conv": 4}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": experts, "top": 4, "scale": 2.0, "groups": {"count": 4, "keep": 2}}}
+    pair = {"left": left, "right": right, "left_scale": 1.0, "right_scale": 0.8}
+    one = [{"type": "channel_delta", "mixer": delta, "mlp": dense}, {"type": "channel_delta", "mixer": delta, "mlp": moe},
+           {"type": "parallel", "mixer": pair, "mlp": dense}, {"type": "channel_delta", "mixer": delta, "mlp": moe}]
+    return {"architecture": "Samulorn", "vocab": MIVORAX_VOCAB, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+            "token_side": {"dim": 128}, "loop": {"start": 0, "stop": 8, "times": 1}, "layers": one + one}, \
+        {"delta": delta, "pair": pair, "feed_forward": moe, "token_side": 128}
+
+
 def mivorax_section(args, section="mivorax") -> int:
     """Prefill of 2,048 tokens and decode (batch 8, context 4,096) of an 8-layer Mivorax model (2 latent attention,
     4 attention with distance bias, 2 state-space layers; width 2,048) and of a Llama model of the same width, depth,
@@ -349,7 +370,15 @@ def mivorax_section(args, section="mivorax") -> int:
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda:0")        # larger than L2: written between timed steps
     results = {}
     width, ff = MIVORAX_WIDTH, MIVORAX_FF
-    if section == "risizen":
+    if section == "samulorn":
+        # 8 layers (6 delta rule with a decay per channel, 2 pairs of attention and a linear recurrence; 4 dense and 4 routed
+        # feed-forwards) beside the Nufasun model (its closest in the delta rule), the Vibunex model (its closest in the routed
+        # feed-forward) and the Llama model of the same width, depth, heads and vocabulary (its closest in the attention)
+        width, ff, heads, kv = _VIBUNEX_SIZES[args.design_size][:4]
+        sam, mixers = _samulorn_config(args.design_size)
+        designs = (("samulorn", sam),) + ((("nufasun", _nufasun_config()),) if args.design_size == "base" else ()) \
+            + (("vibunex", _vibunex_config(args.design_size)), ("llama", _llama_twin(width, ff, heads, kv)))
+    elif section == "risizen":
         # 8 layers (6 with keys of their own, 2 that read them; four streams) beside the Llama model of the same width, depth, heads,
         # feed-forward size and vocabulary, its closest in the attention, and the Nufasun model, its closest in the feed-forward
         width, ff, heads, kv = _VIBUNEX_SIZES[args.design_size][:4]
@@ -500,17 +529,17 @@ def main() -> int:
     ap.add_argument("--profiler-range", action="store_true",
                     help="bracket the timed region of --section with cudaProfilerStart/Stop "
                          "(for ncu --profile-from-start off)")
-    ap.add_argument("--section", default="all", choices=["all", "decode", "prefill", "mivorax", "nufasun", "vibunex", "fevosun", "risizen"],
+    ap.add_argument("--section", default="all", choices=["all", "decode", "prefill", "mivorax", "nufasun", "vibunex", "fevosun", "risizen", "samulorn"],
                     help="run only the device-timed decode steps or only the prefill (for profiling); 'mivorax': prefill "
                          "and decode of a Mivorax model at layer sizes of a real model beside a Llama model of equal "
                          "width, with time per kind of kernel (its own JSON line; the default workload is not run); "
                          "'nufasun': the same for a Nufasun model beside the Mivorax and Llama models; 'vibunex': the same for a "
                          "Vibunex model beside the Nufasun and Llama models; 'fevosun': the same for a Fevosun model beside the "
                          "Mivorax, Vibunex and Llama models; 'risizen': the same for a Risizen model beside the Nufasun and Llama "
-                         "models")
+                         "models; 'samulorn': the same for a Samulorn model beside the Nufasun, Vibunex and Llama models")
     ap.add_argument("--design-size", default="base", choices=["narrow", "base", "wide"],
-                    help="--section vibunex / fevosun / risizen: width 1,024 / 2,048 / 4,096 with heads, experts and feed-forward to match")
-    ap.add_argument("--only-design", default=None, help="--section mivorax / nufasun / vibunex / fevosun / risizen: run this model alone (for profiling)")
+                    help="--section vibunex / fevosun / risizen / samulorn: width 1,024 / 2,048 / 4,096 with heads, experts and feed-forward to match")
+    ap.add_argument("--only-design", default=None, help="--section mivorax / nufasun / vibunex / fevosun / risizen / samulorn: run this model alone (for profiling)")
     args = ap.parse_args()
 
     if args.gpus != 1:
@@ -519,7 +548,7 @@ def main() -> int:
     if args.impl == "reference":
         return reference_arm(args)
     K, W = args.steps, max(3, args.warmup)
-    if args.section in ("mivorax", "nufasun", "vibunex", "fevosun", "risizen"):
+    if args.section in ("mivorax", "nufasun", "vibunex", "fevosun", "risizen", "samulorn"):
         return mivorax_section(args, args.section)
 
     import torch

@@ -1,0 +1,731 @@
+"""Samulorn on the GPU against the plain implementation (tests/plain_samulorn.py): every mechanism alone, prompts against
+token-by-token decoding, portions down to two tokens, unequal batches with pages and slots used again, keys far away and at page
+borders, tokens far back that only a state remembers, the first tokens, long decoding, other sizes, and greedy generation through
+the entry point. Weights come from tests/samulorn_configs.py, which makes them so that a lost key, state, tap, bias, norm or
+group shows in the logits."""
+import json
+import math
+import os
+import random
+import subprocess
+import sys
+
+import pytest
+import torch
+
+import plain_samulorn as ps
+import replay_util as ru
+import samulorn_configs as sc
+
+pytestmark = pytest.mark.gpu
+
+# A row's error: root mean square of the difference of the logits (mean taken off) over that of the plain logits. In 32-bit every
+# row is held to the limit. In bfloat16 rounding alone gives a median well below it with single rows above: the limit holds for the
+# median and for all but one row in twenty, and no row may pass four times the limit; rows whose router choice is closer than
+# MARGIN (in some layer run) may choose otherwise and are left out there.
+LIMIT = {torch.float32: 2e-4, torch.bfloat16: 8e-2}
+MARGIN = {torch.float32: 1e-5, torch.bfloat16: 0.02}
+DTYPES = [torch.float32, torch.bfloat16]
+IDS = ["fp32", "bf16"]
+DEV = "cuda:0"
+
+
+class Plain(ru.PlainLogits):
+    """The plain logits, and per position how close the closest router choice was up to there (a choice made otherwise
+    stays in the states behind it)."""
+
+    def __init__(self, folder):
+        super().__init__(folder, ps)
+        self.margins = {}
+
+    def of(self, tokens):
+        key = tuple(tokens)
+        if key not in self._cache:
+            m = []
+            self._cache[key] = ps.forward(self.cfg, self.w, tokens, margins=m)
+            T = len(tokens)
+            self.margins[key] = torch.tensor(m, dtype=torch.float64).view(-1, T).min(0).values if m else torch.full((T,), math.inf)
+        return self._cache[key]
+
+    def margin(self, tokens, p):
+        self.of(tokens)
+        return self.margins[tuple(tokens)][p].item()
+
+
+@pytest.fixture(scope="module")
+def folders(tmp_path_factory):
+    root = tmp_path_factory.mktemp("samulorn")
+    return {n: sc.write_folder(os.path.join(str(root), n), cfg, seed=31 + i, change=sc.CHANGES.get(n))
+            for i, (n, cfg) in enumerate(sc.CONFIGS.items())}
+
+
+@pytest.fixture(scope="module")
+def plains(folders):
+    return {n: Plain(d) for n, d in folders.items()}
+
+
+def replayer(folder, page_size, dtype, max_tokens, max_requests=4):
+    from llm_steadyinfer_b200.engine.replay import Replayer
+    return Replayer(folder, dtype, max_tokens, page_size=page_size, max_requests=max_requests)
+
+
+def row_error(row, ref):
+    d = row.to(torch.float64) - ref
+    d = d - d.mean()
+    return (d.pow(2).mean().sqrt() / ref.sub(ref.mean()).pow(2).mean().sqrt()).item()
+
+
+def check(rp, steps, reqs, plain, dtype, what):
+    worst, errors, seen = 0.0, [], 0
+    hard = LIMIT[dtype] * (4 if dtype == torch.bfloat16 else 1)
+    for rid, p, row in ru.replay_in_process(rp, steps):
+        e = row_error(row, plain.of(reqs[rid])[p])
+        seen += 1
+        assert e == e, f"{what}: request {rid!r} position {p}: not a number"
+        if plain.margin(reqs[rid], p) < MARGIN[dtype]:
+            continue
+        assert e <= hard, f"{what}: request {rid!r} position {p}: error {e:.3e} (allowed {hard:.0e})"
+        worst = max(worst, e)
+        errors.append(e)
+    n = len(errors)
+    assert seen > 0 and n >= seen // 3
+    if dtype == torch.bfloat16 and n:
+        errors.sort()
+        over = sum(e > LIMIT[dtype] for e in errors)
+        assert over <= max(1, n // 20), f"{what}: {over} of {n} rows above {LIMIT[dtype]:.0e}"
+        assert errors[n // 2] <= LIMIT[dtype] / 2 or n < 4, f"{what}: median error {errors[n // 2]:.3e}"
+    mgr = rp.runner.manager
+    mgr.check_invariant()
+    assert not mgr.requests
+    assert all(mgr.free_pages(g) == mgr.groups[g].pool.num_pages for g in range(len(mgr.groups)))
+    return worst
+
+
+def requests_of(name, lengths, seed=0):
+    vocab = sc.CONFIGS[name]["vocab"]
+    return {f"q{i}": ru.random_tokens(vocab, n, 1000 * seed + i) for i, n in enumerate(lengths)}
+
+
+# ---- each mechanism alone, and the layers of a whole model one by one ------------------------------------
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("name", ["delta", "pair", "moe", "dense", "side", "loop"])
+def test_each_mechanism_alone(folders, plains, name, dtype):
+    reqs = requests_of(name, [1, 2, 37, 90])
+    for mode, steps in (("whole", ru.trace_whole(reqs)), ("tail", ru.trace_tail(reqs, tail=30))):
+        rp = replayer(folders[name], sc.PAGE_SIZE[name], dtype, 128)
+        check(rp, steps, reqs, plains[name], dtype, f"{name}/{mode}")
+
+
+@pytest.mark.parametrize("name", ["mixed_a", "mixed_b", "odd"])
+def test_layers_one_by_one_in_32_bit(folders, name):
+    """The residual stream after every layer run against the plain one (a looped layer counted each time)."""
+    toks = ru.random_tokens(sc.CONFIGS[name]["vocab"], 45, 5)
+    cfg, w = ps.read_model_folder(folders[name])
+    want = []
+    ps.forward(cfg, w, toks, want)
+    rp = replayer(folders[name], sc.PAGE_SIZE[name], torch.float32, 64)
+    got = {}
+    rp.runner.model.hook_layers(lambda run, resid: got.__setitem__(run, resid.double().cpu()))
+    rp.run_step([{"id": "a", "tokens": toks, "want": [len(toks) - 1]}], end=["a"])
+    order = ps.run_order(cfg)
+    assert sorted(got) == list(range(len(order))) and len(want) == len(order)
+    for run, i in enumerate(order):
+        scale = want[run].abs().max().item()
+        diff = (got[run] - want[run]).abs().max().item()
+        assert diff <= 1e-4 * scale, f"{name}: run {run} (layer {i}, {cfg['layers'][i]['type']}) differs by {diff:.2e} of {scale:.1f}"
+
+
+# ---- schedules ------------------------------------------------------------------------------------------
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("name", ["mixed_a", "mixed_b", "odd"])
+@pytest.mark.parametrize("mode", ["whole", "tail", "portions", "mixed"])
+def test_schedules(folders, plains, name, dtype, mode):
+    reqs = requests_of(name, [1, 3, 19, 64, 65, 130, 201], seed=1)
+    longest = ru.round64(max(len(t) for t in reqs.values()))
+    if mode == "whole":
+        steps, max_tokens = ru.trace_whole(reqs), longest
+    elif mode == "tail":
+        steps, max_tokens = ru.trace_tail(reqs, tail=40), longest
+    elif mode == "portions":
+        steps, max_tokens = ru.trace_portions(reqs, sizes=(2, 17, 3, 2, 31, 5, 64, 2, 9, 1, 40)), longest
+    else:
+        max_tokens = longest + 128                       # two or three live at a time: pages and slots come again
+        steps = ru.trace_mixed(reqs, max_tokens, seed=3, max_live=3)
+    rp = replayer(folders[name], sc.PAGE_SIZE[name], dtype, max_tokens, max_requests=3)
+    worst = check(rp, steps, reqs, plains[name], dtype, f"{name}/{mode}")
+    print(f"{name} {mode} {dtype}: worst row error {worst:.2e}")
+
+
+@pytest.mark.parametrize("seed", range(10))
+def test_configurations_drawn_at_random(tmp_path, seed):
+    """Sizes, layer orders, loops and constants over wide ranges, each through portions and a mixed schedule in both precisions."""
+    rng = random.Random(4000 + seed)
+    cfg = sc.random_config(rng, aligned=seed % 2 == 0)
+    folder = sc.write_folder(str(tmp_path / "m"), cfg, seed)
+    plain = Plain(folder)
+    reqs = {f"q{i}": ru.random_tokens(cfg["vocab"], n, 10 * seed + i) for i, n in enumerate([70, 5, 33, 101])}
+    for dtype in DTYPES:
+        rp = replayer(folder, rng.choice([4, 8, 16]), dtype, 256, max_requests=3)
+        check(rp, ru.trace_portions(reqs, sizes=(17, 2, 1, 40, 3)), reqs, plain, dtype, f"{cfg}: portions")
+        check(rp, ru.trace_mixed(reqs, 256, seed=seed, max_live=3), reqs, plain, dtype, f"{cfg}: mixed")
+
+
+def test_batch_equals_alone_and_slots_come_again(folders, plains):
+    """Unequal requests in one batch against each alone, with two state slots for five requests: every slot and page is used again,
+    and what the request before left there (recurrent states, convolution inputs, keys) must not show."""
+    name, dtype = "mixed_a", torch.float32
+    reqs = requests_of(name, [70, 9, 33, 2, 51], seed=2)
+    rp = replayer(folders[name], sc.PAGE_SIZE[name], dtype, 192, max_requests=2)
+    check(rp, ru.trace_mixed(reqs, 192, seed=9, max_live=2, prompt_frac=0.5), reqs, plains[name], dtype, "two slots")
+    again = dict(reversed(list(reqs.items())))
+    check(rp, ru.trace_mixed(again, 192, seed=10, max_live=2, prompt_frac=0.3), again, plains[name], dtype, "two slots again")
+
+
+def test_large_batches(folders, plains):
+    """Twenty requests decoding beside one another (more rows than the weight-streaming products take), prompts beside them."""
+    name = "mixed_b"
+    reqs = requests_of(name, [20 + 3 * (i % 7) for i in range(24)], seed=6)
+    for dtype in DTYPES:
+        rp = replayer(folders[name], sc.PAGE_SIZE[name], dtype, 24 * 64, max_requests=24)
+        check(rp, ru.trace_mixed(reqs, 24 * 64, seed=4, max_live=24, prompt_frac=0.3), reqs, plains[name], dtype, "large batch")
+
+
+def test_long_decoding(folders, plains):
+    """A short prompt, then 300 tokens one by one, across many page borders; the states are carried 300 times."""
+    name = "mixed_a"
+    reqs = requests_of(name, [310], seed=3)
+    for dtype in DTYPES:
+        rp = replayer(folders[name], sc.PAGE_SIZE[name], dtype, 320)
+        check(rp, ru.trace_tail(reqs, tail=300), reqs, plains[name], dtype, "long decoding")
+
+
+def test_first_tokens(folders, plains):
+    """Positions 0 to 4 alone and as the start of portions: zeros before the sequence in every convolution, states that start at zero,
+    a softmax over one key, a rotation by angle zero."""
+    name = "mixed_b"
+    reqs = requests_of(name, [1, 2, 3, 5], seed=4)
+    for dtype in DTYPES:
+        for sizes in ((1,), (2, 1), (1, 2)):
+            rp = replayer(folders[name], sc.PAGE_SIZE[name], dtype, 64)
+            check(rp, ru.trace_portions(reqs, sizes=sizes), reqs, plains[name], dtype, f"first tokens {sizes}")
+
+
+def slow_delta(t):
+    t["l0.mix.dt_bias"][:] = -9.0                        # decay about exp(-1e-4) a token
+    t["l0.mix.a2"][:] = 0.0
+    t["l0.mix.b"][:] = 0.0                               # beta 1/2
+
+
+def slow_recurrence(t):
+    t["l0.mix.right.lam"][:] = -9.0                      # decay about exp(-1e-3) a token at most
+    t["l0.mix.left.o"][:] = 0.0
+
+
+@pytest.mark.parametrize("mixer,change", [(sc.delta(4, 2, 64, 16, 2), slow_delta),
+                                          (sc.pair((2, 1, 16, 16, 2, None), (64, 4, 3)), slow_recurrence)], ids=["delta", "recurrence"])
+def test_a_token_far_back_reaches_through_the_state(tmp_path, mixer, change):
+    """A state whose decay is almost one: what token 3 wrote is read 400 tokens later, in portions cut anywhere."""
+    cfg = sc.model(120, 64, [sc.layer(mixer, sc.dense(48))])
+    folder = sc.write_folder(str(tmp_path / "far"), cfg, 5, change=change)
+    plain = Plain(folder)
+    a = ru.random_tokens(120, 420, 77)
+    b = list(a)
+    b[3] = (a[3] + 17) % 120
+    assert row_error(plain.of(a)[-1], plain.of(b)[-1]) > 10 * LIMIT[torch.float32], "the test's weights do not carry the far token"
+    for dtype in DTYPES:
+        rp = replayer(folder, 8, dtype, 448)
+        check(rp, ru.trace_portions({"a": a, "b": b}, sizes=(64, 2, 100, 31, 1)), {"a": a, "b": b}, plain, dtype, "far token")
+
+
+@pytest.mark.parametrize("dim", [64, 20])
+def test_a_key_that_stands_out_far_back_and_at_page_borders(tmp_path, dim):
+    """Attention whose scores are so steep that one key decides: a query's own token type is found wherever it lies, among hundreds of
+    others (no rotation, so that the query's own key and the far one share the weight). A marker token appears twice; the logits at its second place must depend on what stands beside the first."""
+    cfg = sc.model(60, 64, [sc.layer(sc.pair((2, 1, dim, dim, 2, None), (16, 2, 2)))])
+    cfg["layers"][0]["mixer"]["left"]["scale"] = 60.0 / dim          # scores of at most 60: the best key outweighs a few hundred others
+
+    def steep(t):
+        t["l0.mix.right.o"][:] = 0.0
+        for n in ("q", "k"):                                         # the current token's query and key; queries and keys of one matrix
+            t[f"l0.mix.left.{n}.conv"][:] = [0.0, 1.0]
+            t[f"l0.mix.left.{n}.b"][:] = 0.0
+        t["l0.mix.left.q"][:dim] = t["l0.mix.left.k"]
+        t["l0.mix.left.q"][dim:] = t["l0.mix.left.k"]
+        t["l0.mix.left.v.conv"][:] = [1.0, 0.3]                      # the value speaks of the token before as well
+
+    folder = sc.write_folder(str(tmp_path / "far"), cfg, 8, change=steep)
+    plain = Plain(folder)
+    base = [1 + t % 58 for t in ru.random_tokens(58, 330, 3)]        # token 59 is the marker
+    for place in (0, 15, 16, 17, 63, 64, 200, 311):                  # at page borders, far back, just before
+        a = list(base)
+        a[place] = a[-1] = 59
+        if place:
+            b = list(a)
+            b[place - 1] = 1 + (b[place - 1] + 5) % 58
+            assert row_error(plain.of(a)[-1], plain.of(b)[-1]) > 50 * LIMIT[torch.float32], "the far key does not decide"
+        for dtype in DTYPES:
+            rp = replayer(folder, 16, dtype, 384)
+            check(rp, ru.trace_portions({"a": a}, sizes=(100, 2, 200, 25, 1)), {"a": a}, plain, dtype, f"marker at {place}")
+
+
+# ---- kernels ----------------------------------------------------------------------------------------------------
+
+i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device=DEV)
+
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("T,width", [(11, 70), (1, 64), (3, 1000), (5, 4096), (1100, 256), (2, 20000)])
+def test_norms_of_every_kind_around_the_stream(T, width, dtype):
+    from llm_steadyinfer_b200.csrc import ops
+    torch.manual_seed(width)
+    resid, delta, bias = torch.randn(T, width) * 2, torch.randn(T, width).to(dtype), torch.randn(width)
+    vec = lambda: 1 + 0.3 * torch.randn(width)
+    norms = {"copy": None, "tanh": ("tanh", vec(), vec() - 1, 0.7), "rms": ("rms", vec(), 1e-5)}
+
+    def plain(n, x):
+        if n is None:
+            return x
+        if n[0] == "tanh":
+            return ps.tanh_norm(x, {"n": n[1].double(), "n.b": n[2].double(), "n.alpha": n[3]}, "n")
+        return ps.over_rms(x, n[2]) * n[1].double()
+
+    dev = lambda n: None if n is None else tuple(v.to(DEV) if torch.is_tensor(v) else v for v in n)
+    tol = 2e-5 if dtype == torch.float32 else 1e-2
+    for dn in norms.values():
+        for with_bias in (False, True):
+            d = delta.double() + (bias.double() if with_bias else 0.0)
+            h = resid.double() + plain(dn, d)
+            for on in norms.values():
+                r, out = resid.to(DEV).clone(), torch.zeros(T, width, dtype=dtype, device=DEV)
+                ops.stream_add(r, delta.to(DEV), dev(dn), bias.to(DEV) if with_bias else None, out, dev(on))
+                assert (r.double().cpu() - h).abs().max() <= 2e-5 * h.abs().max()
+                want = plain(on, h)
+                assert (out.double().cpu() - want).abs().max() <= tol * want.abs().max()
+        r2 = resid.to(DEV).clone()
+        ops.stream_add(r2, delta.to(DEV), dev(dn), bias.to(DEV))                    # without an output the same sums
+        assert torch.equal(r2, r)
+    rows = i32(T - 1, 0, T // 2)
+    for on in norms.values():
+        keep, out = resid.to(DEV).clone(), torch.zeros(3, width, dtype=dtype, device=DEV)
+        ops.stream_add(keep, delta.to(DEV), dev(norms["rms"]), None, out, dev(on), rows)
+        want = plain(on, resid.double() + plain(norms["rms"], delta.double()))[rows.cpu().long()]
+        assert torch.equal(keep.cpu(), resid) and (out.double().cpu() - want).abs().max() <= tol * want.abs().max()
+        out = torch.zeros(T, width, dtype=dtype, device=DEV)
+        ops.stream_add(keep, None, None, None, out, dev(on))                        # nothing to add
+        assert torch.equal(keep.cpu(), resid) and (out.double().cpu() - plain(on, resid.double())).abs().max() <= tol * 10
+
+
+def portions_of(lens, sizes):
+    """Steps of [(sequence, first row, rows)] that walk all sequences to their ends."""
+    at = [0] * len(lens)
+    for step in sizes:
+        live = [(s, at[s], min(m, lens[s] - at[s])) for s, m in enumerate(step) if min(m, lens[s] - at[s]) > 0]
+        if live:
+            yield live
+        for s, a, m in live:
+            at[s] = a + m
+    assert at == lens
+
+
+def step_ints(live, slots, pad=1):
+    """positions, row_seq, q_start, ctx_len, slots of a step with padding rows behind it, and what the launch is told of it."""
+    pos = [p for _, a, m in live for p in range(a, a + m)] + [0] * pad
+    seq = [i for i, (_, _, m) in enumerate(live) for _ in range(m)] + [-1] * pad
+    starts = [0]
+    for _, _, m in live:
+        starts.append(starts[-1] + m)
+    portions = (1 if any(m > 1 and a == 0 for _, a, m in live) else 0) | (2 if any(m > 1 and a > 0 for _, a, m in live) else 0)
+    kinds = (1 if any(m == 1 for _, _, m in live) else 0) | (2 if any(m > 1 for _, _, m in live) else 0)
+    return i32(*pos), i32(*seq), i32(*starts), i32(*[a + m for _, a, m in live]), i32(*[slots[s] for s, _, _ in live]), portions, kinds
+
+
+STEPS = [(1, 2, 17), (1, 1, 1), (2, 3, 1), (1, 5, 2), (20, 0, 9), (3, 1, 30), (0, 11, 0), (13, 0, 0)]
+LENS = [41, 23, 60]
+SLOTS = [3, 0, 2]
+
+
+def scaled(times):
+    return [n * times for n in LENS], [tuple(m * times if m > 1 else m for m in s) for s in STEPS] + [(times, times, times)] * 3
+
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("NQ,NK,NV,dk,dv,K,unit,silu,bias,copy", [
+    (2, 2, 4, 24, 16, 4, True, True, False, False), (3, 3, 3, 64, 128, 2, True, True, False, False), (2, 2, 2, 10, 6, 3, True, True, False, False),
+    (0, 0, 3, 16, 24, 4, False, False, True, True), (0, 0, 5, 7, 7, 3, False, False, True, True), (2, 2, 4, 128, 64, 6, True, True, False, True),
+    (1, 1, 1, 8, 8, 1, True, False, True, False), (0, 0, 2, 128, 128, 1, False, True, True, True)])
+@pytest.mark.parametrize("times", [1, 24], ids=["few_rows", "many_rows"])
+def test_convolution_in_front_of_a_recurrence(NQ, NK, NV, dk, dv, K, unit, silu, bias, copy, times, dtype):
+    """Biases before and behind the convolution, silu, unit vectors and the copy by vectors, over three sequences in unequal portions whose
+    states lie in slots that held something else."""
+    from llm_steadyinfer_b200.csrc import ops
+    torch.manual_seed(K * 100 + dk + dv)
+    C = (NQ + NK) * dk + NV * dv
+    lens, sizes = scaled(times)
+    width = -(-C // 8) * 8 + 8
+    u = [torch.randn(n, width).to(dtype) for n in lens]
+    taps = torch.randn(K, C) * 0.6
+    b, ob = (torch.randn(C) * 0.4, torch.randn(C) * 0.4) if bias else (None, None)
+    q_scale, want = 0.37, []
+    for x in u:
+        y = ps.causal_conv(x[:, :C].double() + (b.double() if bias else 0.0), taps.double().T) + (ob.double() if bias else 0.0)
+        if silu:
+            y = ps.silu(y)
+        if unit:
+            y[:, :NQ * dk] = (ps.unit(y[:, :NQ * dk].view(-1, NQ, dk)) * q_scale).reshape(-1, NQ * dk)
+            y[:, NQ * dk:(NQ + NK) * dk] = ps.unit(y[:, NQ * dk:(NQ + NK) * dk].view(-1, NK, dk)).reshape(-1, NK * dk)
+        want.append(y)
+    state = torch.full((4, -(-(K - 1) * C // 4) * 4), 7.0, device=DEV) if K > 1 else None
+    got = [torch.zeros(n, C) for n in lens]
+    size = -(-max(dk if NQ + NK else 0, dv) // 8) * 8
+    status = i32(0)
+    dev = lambda t: None if t is None else t.to(DEV)
+    for live in portions_of(lens, sizes):
+        pos, seq, starts, ctx, slots, portions, _ = step_ints(live, SLOTS)
+        rows = torch.cat([u[s][a:a + m] for s, a, m in live] + [torch.full((1, width), 9.0).to(dtype)]).to(DEV)
+        R = rows.shape[0]
+        out = torch.zeros(R, C, device=DEV)
+        cp = torch.zeros(NQ + NK + NV, R, size, dtype=dtype, device=DEV) if copy else None
+        ops.conv_rows(rows, dev(b), taps.to(DEV), state, pos, seq, starts, ctx, slots, len(live), NQ, NK, NV, dk, dv, out, unit=unit,
+                      q_scale=q_scale, silu=silu, out_bias=dev(ob), copy=cp, portions=portions, status=status)
+        r = 0
+        for s, a, m in live:
+            got[s][a:a + m] = out[r:r + m].cpu()
+            r += m
+        if copy:
+            whole = [out[:R - 1, i * dk:(i + 1) * dk] for i in range(NQ + NK)] + [out[:R - 1, (NQ + NK) * dk + i * dv:(NQ + NK) * dk + (i + 1) * dv] for i in range(NV)]
+            for i, part in enumerate(whole):
+                assert torch.equal(cp[i, :R - 1, :part.shape[1]], part.to(dtype)) and not cp[i, :, part.shape[1]:].any()
+    assert status.item() == 0
+    for s, n in enumerate(lens):
+        assert (got[s].double() - want[s]).abs().max() < 2e-5 * max(1.0, want[s].abs().max().item()), f"sequence {s}"
+        if K > 1:
+            kept = state[SLOTS[s], :(K - 1) * C].cpu().double().view(K - 1, C)
+            assert (kept - (u[s][n - K + 1:, :C].double() + (b.double() if bias else 0.0))).abs().max() < 1e-6
+    if K > 1:
+        assert (state[1] == 7.0).all()
+
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("NQ,NK,NV,dk,dv,K,dims", [(6, 2, 2, 16, 24, 4, 16), (4, 4, 4, 64, 64, 3, 32), (8, 2, 2, 128, 40, 2, 128), (3, 1, 1, 10, 6, 3, 6),
+                                                   (2, 1, 1, 8, 8, 1, 2), (2, 2, 2, 32, 16, 7, 28), (2, 1, 1, 256, 128, 4, 256)])
+@pytest.mark.parametrize("times", [1, 24], ids=["few_rows", "many_rows"])
+def test_rotation_between_convolution_and_norm(NQ, NK, NV, dk, dv, K, dims, times, dtype):
+    """The launch behind the stacked projection with a rotation: queries in their rows, keys and values in their pages."""
+    from llm_steadyinfer_b200.csrc import ops
+    torch.manual_seed(K + dk)
+    C = (NQ + NK) * dk + NV * dv
+    lens, sizes = scaled(times)
+    ps_, eps = 8, 1e-5
+    rot = {"base": 300.0, "dims": dims, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 200}}
+    inv = ps.frequencies(rot).float()
+    width = -(-C // 8) * 8
+    u = [torch.randn(n, width).to(dtype) for n in lens]
+    taps, b = torch.randn(K, C) * 0.6, torch.randn(C) * 0.4
+    want = []
+    for x in u:
+        y = ps.causal_conv(x[:, :C].double() + b.double(), taps.double().T)
+        q, k = y[:, :NQ * dk].view(-1, NQ, dk), y[:, NQ * dk:(NQ + NK) * dk].view(-1, NK, dk)
+        want.append((ps.over_rms(ps.rotate(q, rot), eps), ps.over_rms(ps.rotate(k, rot), eps), y[:, (NQ + NK) * dk:].view(-1, NV, dv)))
+    state = torch.full((4, -(-(K - 1) * C // 4) * 4), 7.0, device=DEV) if K > 1 else None
+    blocks = -(-max(lens) // ps_)
+    pages = torch.randperm(3 * blocks + 2, generator=torch.Generator().manual_seed(1))[:3 * blocks].view(3, blocks)
+    table = pages.to(torch.int32).to(DEV)
+    kc = torch.zeros(3 * blocks + 2, NK, ps_, dk, dtype=dtype, device=DEV)
+    vc = torch.zeros(3 * blocks + 2, NV, ps_, dv, dtype=dtype, device=DEV)
+    got = [torch.zeros(n, NQ * dk, dtype=dtype) for n in lens]
+    status = i32(0)
+    for live in portions_of(lens, sizes):
+        pos, seq, starts, ctx, slots, portions, _ = step_ints(live, SLOTS)
+        rows = torch.cat([u[s][a:a + m] for s, a, m in live] + [torch.full((1, width), 9.0).to(dtype)]).to(DEV)
+        q = torch.zeros(rows.shape[0], NQ * dk, dtype=dtype, device=DEV)
+        ops.qkv_conv(rows, b.to(DEV), taps.to(DEV), state, pos, seq, starts, ctx, slots, table[[s for s, _, _ in live]].contiguous(), kc, vc, ps_,
+                     len(live), NQ, NK, NV, dk, dv, q, True, eps, portions=portions, status=status, inv_freq=inv.to(DEV), rot_dims=dims)
+        r = 0
+        for s, a, m in live:
+            got[s][a:a + m] = q[r:r + m].cpu()
+            r += m
+    assert status.item() == 0
+    # an angle of a position up to 1,500 in 32-bit is off by up to 1.2e-4, and so is a turned pair
+    tol = (3e-5 if times == 1 else 4e-4) if dtype == torch.float32 else 6e-3
+    off = lambda a, ref: ((a.double() - ref).abs() / (1.0 + ref.abs())).max().item()
+    for s, n in enumerate(lens):
+        assert off(got[s].view(n, NQ, dk), want[s][0]) < tol, f"queries of sequence {s}"
+        at_page, place = pages[s, torch.arange(n) // ps_], torch.arange(n) % ps_
+        assert off(kc.cpu()[at_page, :, place], want[s][1]) < tol, f"keys of sequence {s}"
+        assert off(vc.cpu()[at_page, :, place], want[s][2]) < tol, f"values of sequence {s}"
+
+
+@pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 24, 16), (3, 3, 64, 128), (2, 1, 5, 9), (8, 2, 128, 64), (2, 2, 160, 24), (16, 8, 128, 128), (1, 1, 512, 40),
+                                       (2, 2, 4, 4), (2, 1, 200, 36)])
+def test_channel_delta_kernels_in_portions(H, G, dk, dv):
+    """Preparation, recurrence and the read-out's norm with its sigmoid gate over three sequences in unequal portions."""
+    from llm_steadyinfer_b200.csrc import ops
+    torch.manual_seed(H * 100 + dk)
+    C = 2 * G * dk + H * dv
+    raw = [torch.randn(n, H * dk) for n in LENS]
+    ba = [torch.randn(n, H + 5) for n in LENS]
+    z = [torch.randn(n, H * dv) for n in LENS]
+    x, want = [], []
+    a_log, dt_bias, norm_w = torch.empty(H).uniform_(-1, 1), torch.empty(H * dk).uniform_(-4, -1), 1 + 0.1 * torch.randn(dv)
+    for s, n in enumerate(LENS):
+        q, k = ps.unit(torch.randn(n, G, dk)), ps.unit(torch.randn(n, G, dk))
+        v = torch.randn(n, H, dv)
+        x.append(torch.cat([q.reshape(n, -1), k.reshape(n, -1), v.reshape(n, -1)], 1))
+        beta = torch.sigmoid(ba[s][:, 3:3 + H].double())
+        decay = torch.exp(-torch.exp(a_log.double())[:, None] * torch.nn.functional.softplus(raw[s].double() + dt_bias.double()).view(n, H, dk))
+        o = torch.stack([ps.delta_head(q[:, h // (H // G)].double(), k[:, h // (H // G)].double(), v[:, h].double(), beta[:, h], decay[:, h])
+                         for h in range(H)], 1)
+        want.append(ps.over_rms(o, 1e-5) * norm_w.double() * torch.sigmoid(z[s].double().view(n, H, dv)))
+    state = torch.randn(4, H * ops.delta_state_floats(dk, dv) + 4, device=DEV)         # stale contents
+    got = [torch.zeros(n, H * dv) for n in LENS]
+    for live in portions_of(LENS, scaled(1)[1]):
+        _, _, starts, ctx, slots, _, _ = step_ints(live, SLOTS, pad=0)
+        cat = lambda t: torch.cat([t[s][a:a + m] for s, a, m in live]).to(DEV)
+        xc, dec, rows = cat(x), cat(raw), cat(ba)
+        R = xc.shape[0]
+        bg, y = torch.zeros(R, H + G, device=DEV), torch.zeros(R, H * dv, device=DEV)
+        ops.channel_delta_prepare(xc, rows, 3, dec, a_log.to(DEV), dt_bias.to(DEV), bg, G, H, dk)
+        ops.channel_delta_scan(xc, dec, bg, state, y, starts, ctx, slots, len(live), G, H, dk, dv)
+        out = torch.zeros(R, H * dv, device=DEV)
+        ops.head_norm_gate(y, cat(z), norm_w.to(DEV), out, H, dv, 1e-5, gate="sigmoid")
+        r = 0
+        for s, a, m in live:
+            got[s][a:a + m] = out[r:r + m].cpu()
+            r += m
+    for s, n in enumerate(LENS):
+        diff = (got[s].double().view(n, H, dv) - want[s]).abs().max().item()
+        assert diff <= 2e-4 * max(1.0, want[s].abs().max().item()), f"sequence {s} differs by {diff:.2e}"
+
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("W,blocks,times", [(48, 3, 1), (21, 1, 1), (30, 6, 24), (256, 2, 24)])
+def test_linear_recurrence_in_portions(W, blocks, times, dtype):
+    """Single rows and portions (some longer than a round of 256 rows) of three sequences side by side; the two launches keep
+    to their own sequences and slots."""
+    from llm_steadyinfer_b200.csrc import ops
+    torch.manual_seed(W + times)
+    lens, sizes = scaled(times)
+    bs, scale = W // blocks, 1.3
+    u = [torch.randn(n, W) for n in lens]
+    zr, zi, y = ([torch.randn(n, W) * 2 for n in lens] for _ in range(3))
+    y = [t.to(dtype) for t in y]
+    br, bi, by, lam = torch.randn(W), torch.randn(W), torch.randn(W), torch.empty(W).uniform_(-7, -1)
+    rate = (8.0 * torch.nn.functional.softplus(lam.double())).float()
+    want = []
+    for s, n in enumerate(lens):
+        la = -torch.sigmoid(zr[s].double() + br.double()) * rate.double()
+        b = torch.sqrt(1 - torch.exp(2 * la)) * torch.sigmoid(zi[s].double() + bi.double()) * u[s].double()
+        S, out = torch.zeros(W, dtype=torch.float64), []
+        for t in range(n):
+            S = torch.exp(la[t]) * S + b[t]
+            out.append(S)
+        want.append(scale * torch.stack(out) * ps.gelu_tanh(y[s].double() + by.double()))
+    state = torch.randn(4, W + 8, device=DEV)
+    untouched = state[1].clone()
+    got = [torch.zeros(n, W, dtype=dtype) for n in lens]
+    for live in portions_of(lens, sizes):
+        _, _, starts, ctx, slots, _, kinds = step_ints(live, SLOTS, pad=0)
+        cat = lambda t: torch.cat([t[s][a:a + m] for s, a, m in live])
+        R = sum(m for _, _, m in live)
+        z = torch.stack([cat(zr).view(R, blocks, bs), cat(zi).view(R, blocks, bs)], 2).permute(1, 0, 2, 3).reshape(blocks, R, 2 * bs).contiguous()
+        out = torch.zeros(R, W + 3, dtype=dtype, device=DEV)
+        ops.gated_linear(cat(u).to(DEV), z.to(DEV), br.to(DEV), bi.to(DEV), rate.to(DEV), cat(y).to(DEV), by.to(DEV), state, out[:, 1:1 + W],
+                         starts, ctx, slots, len(live), scale, kinds)
+        assert not out[:, 0].any() and not out[:, 1 + W:].any()
+        r = 0
+        for s, a, m in live:
+            got[s][a:a + m] = out[r:r + m, 1:1 + W].cpu()
+            r += m
+    assert torch.equal(state[1], untouched) and torch.isfinite(state).all()
+    for s in range(3):
+        diff = (got[s].double() - want[s]).abs().max().item()
+        assert diff <= (2e-5 if dtype == torch.float32 else 1e-2) * max(1.0, want[s].abs().max().item()), f"sequence {s} differs by {diff:.2e}"
+
+
+@pytest.mark.parametrize("E,top,count,keep", [(12, 3, 4, 2), (64, 8, 8, 4), (15, 5, 5, 2), (9, 2, 9, 3), (8, 4, 2, 2), (200, 6, 40, 3)])
+def test_router_with_groups(E, top, count, keep):
+    """Choices and weights against the plain rule, with choice scores of both signs, exact ties among them."""
+    from llm_steadyinfer_b200.csrc import ops
+    torch.manual_seed(E)
+    T, d, scale = 57, 40, 1.7
+    x, w = torch.randn(T, d), torch.randn(E, d) / math.sqrt(d)
+    corr = torch.randn(E) * 0.4 - 0.6
+    w[1], corr[1] = w[0], corr[0]                        # two experts alike: the lower index goes first
+    ids = torch.zeros(T, top, dtype=torch.int32, device=DEV)
+    wts = torch.zeros(T, top, device=DEV)
+    ops.moe_route(x.to(DEV), w.to(DEV), E, top, scale, ids, wts, renorm=True, choice_bias=corr.to(DEV), renorm_eps=1e-20, groups=(count, keep))
+    s = torch.sigmoid(x.double() @ w.double().T)
+    router = {"top": top, "groups": {"count": count, "keep": keep}}
+    for t in range(T):
+        best = ps.choose(s[t], corr.double(), router)
+        distinct = s[t].clone()
+        distinct[1] = 0.0                                # the planted tie aside
+        if ps.choice_margin(distinct, corr.double(), router) > 1e-5:
+            assert sorted(ids[t].tolist()) == sorted(best), f"row {t}"
+            want = scale * s[t, ids[t].long().cpu()] / (s[t, best].sum() + 1e-20)
+            assert (wts[t].double().cpu() - want).abs().max() < 1e-5
+    tiny = torch.zeros(1, d)                             # scores so small that only the added constant keeps the weights finite
+    deep = torch.zeros(E, d)
+    tiny[0, 0], deep[:, 0] = 1.0, -95.0
+    ops.moe_route(tiny.to(DEV), deep.to(DEV), E, top, scale, ids[:1], wts[:1], renorm=True, choice_bias=corr.to(DEV), renorm_eps=1e-20, groups=(count, keep))
+    assert torch.isfinite(wts[:1]).all()
+
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("T,d,F,E", [(5, 64, 24, 4), (300, 128, 96, 6), (70, 50, 18, 5)])
+def test_gated_experts(T, d, F, E, dtype):
+    """silu(gate) * up in the epilogue of the grouped product, for few places, many places (the tcgen05 kernel) and odd sizes."""
+    from llm_steadyinfer_b200.parts.moe import RoutedMLP
+    from llm_steadyinfer_b200.csrc import ops
+    torch.manual_seed(T)
+    top, scale = 2, 1.5
+    part = RoutedMLP({"hidden_size": d, "intermediate_size": F, "experts": E, "top": top, "scale": scale, "renorm": True, "renorm_eps": 1e-20,
+                      "choice_bias": "correction", "activation": "silu_glu"}, dtype, torch.device(DEV))
+    w = {n: (torch.randn(s) * (1.5 / math.sqrt(s[-1]) if len(s) > 1 else 0.3)).to(dtype) for n, s in part.weight_shapes().items()}
+    part.load_weights({n: t.to(DEV) for n, t in w.items()})
+    x = torch.randn(T, d).to(dtype)
+
+    class Ctx:
+        status = i32(0)
+        buf = staticmethod(lambda key, shape, dt: torch.zeros(shape, dtype=dt, device=DEV))
+
+    got = part.forward(x.to(DEV), Ctx()).double().cpu()
+    margins = []
+    want = ps.routed_feed_forward(x.double(), {n: t.double() for n, t in w.items()}, "", {"router": {"top": top, "scale": scale}}, margins)
+    sure = torch.tensor(margins) > (1e-5 if dtype == torch.float32 else 1e-4)
+    assert sure.sum() > T // 2
+    diff = (got - want)[sure].abs().max().item()
+    assert diff <= (1e-5 if dtype == torch.float32 else 2e-2) * max(1.0, want.abs().max().item()), f"differs by {diff:.2e}"
+    assert Ctx.status.item() == 0 and ops.launch_count() > 0
+
+
+@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("T,d,dim", [(1, 64, 16), (7, 256, 20), (16, 70, 5), (150, 128, 40)])
+def test_token_side_input(T, d, dim, dtype):
+    """The layer's own columns of the table, gated by the stream as a tanh-normed result leaves it; the norm and the add behind it."""
+    from llm_steadyinfer_b200.parts import NormedDelta, TokenSideInput
+    from llm_steadyinfer_b200.parts.norm import DynamicTanh, add_to_stream
+    torch.manual_seed(d)
+    dev = torch.device(DEV)
+    part = TokenSideInput({"hidden_size": d, "dim": dim, "index": 2, "eps": 1e-5}, dtype, dev)
+    w = {n: (torch.randn(s) / math.sqrt(s[-1]) if len(s) > 1 else 1 + 0.2 * torch.randn(s)).to(dtype) for n, s in part.weight_shapes().items()}
+    part.load_weights({n: t.to(DEV) for n, t in w.items()})
+    table = torch.randn(30, 4 * dim).to(dtype)
+    part.set_table(table.to(DEV))
+    norm = DynamicTanh({"size": d, "weight_name": ""}, dtype, dev)
+    nw = {"": torch.randn(d), ".b": torch.randn(d), ".alpha": torch.tensor(0.8)}
+    norm.load_weights({n: t.to(DEV) for n, t in nw.items()})
+    toks = torch.randint(0, 30, (T,))
+
+    class Ctx:
+        status = i32(0)
+        tokens = toks.to(torch.int32).to(DEV)
+        buf = staticmethod(lambda key, shape, dt: torch.zeros(shape, dtype=dt, device=DEV))
+
+    resid, f = torch.randn(T, d), torch.randn(T, d).to(dtype)
+    r = resid.to(DEV).clone()
+    pending = part.forward(r, NormedDelta(f.to(DEV), norm), Ctx())
+    x = resid.double() + ps.tanh_norm(f.double(), {n: t.double() for n, t in (("n", nw[""]), ("n.b", nw[".b"]), ("n.alpha", nw[".alpha"]))}, "n")
+    assert (r.double().cpu() - x).abs().max() < 1e-5
+    add_to_stream(r, pending)
+    want = x + ps.token_side_input(x, table[toks].double()[:, 2 * dim:3 * dim], {n: t.double() for n, t in w.items()}, "", 1e-5)
+    assert (r.double().cpu() - want).abs().max() <= (2e-5 if dtype == torch.float32 else 5e-2) * want.abs().max()
+
+
+# ---- the entry point ----------------------------------------------------------------------------------------
+
+def greedy(cfg, w, prompt, new):
+    """``new`` greedy tokens of the plain implementation, and the smallest gap between the two best logits on the way."""
+    toks, gap = list(prompt), math.inf
+    for _ in range(new):
+        logits = ps.forward(cfg, w, toks)[-1]
+        top2 = torch.topk(logits, 2).values
+        gap = min(gap, (top2[0] - top2[1]).item())
+        toks.append(int(logits.argmax()))
+    return toks[len(prompt):], gap
+
+
+@pytest.mark.parametrize("name", ["mixed_a", "mixed_b"])
+def test_greedy_generation_through_the_entry_point(folders, name):
+    """Greedy tokens through LLM (scheduler, sampler, graphs and steps launched ahead) equal the plain implementation's in 32-bit;
+    bfloat16 runs and mostly agrees."""
+    from llm_steadyinfer_b200 import LLM, SamplingParams
+    cfg, w = ps.read_model_folder(folders[name])
+    prompts = [ru.random_tokens(cfg["vocab"], n, 50 + n) for n in (5, 23, 1, 40)]
+    both = [greedy(cfg, w, p, 12) for p in prompts]
+    want = [b[0] for b in both]
+    assert min(b[1] for b in both) > 1e-3, "the test's prompts meet a close call between two tokens"
+    for dtype in ("float32", "bfloat16"):
+        for graphs in (True, False):
+            llm = LLM(folders[name], dtype=dtype, max_batch=3, max_seq_len=64, max_gen_len=12, block_size=sc.PAGE_SIZE[name],
+                      max_num_batched_tokens=32, use_cuda_graph=graphs, async_decode=graphs)
+            got = [g.token_ids for g in llm.generate(prompts, SamplingParams(ignore_eos=True))]
+            if dtype == "float32":
+                assert got == want, f"{name} graphs={graphs}: {got} != {want}"
+            else:
+                same = sum(a == b for g, x in zip(got, want) for a, b in zip(g, x))
+                assert same >= 24, f"{name} bf16: only {same} of 48 tokens agree"
+            if graphs:
+                assert llm.runner.graphs_available() and llm.stats["graph_steps"] > 0
+
+
+def test_preemption_recomputes_from_the_start(folders):
+    """A pool too small for all requests: some are cut back and computed again, and the tokens still equal the plain
+    implementation's."""
+    from llm_steadyinfer_b200 import LLM, SamplingParams
+    name = "mixed_a"
+    cfg, w = ps.read_model_folder(folders[name])
+    prompts = [ru.random_tokens(cfg["vocab"], n, 90 + n) for n in (30, 28, 26)]
+    want = [greedy(cfg, w, p, 20)[0] for p in prompts]
+    llm = LLM(folders[name], dtype="float32", max_batch=3, max_seq_len=64, max_gen_len=20, block_size=8, num_blocks=14,
+              max_num_batched_tokens=64)
+    assert [r.token_ids for r in llm.generate(prompts, SamplingParams(ignore_eos=True))] == want
+
+
+def test_trace_program_replays_a_mixed_trace(folders, plains, tmp_path):
+    """``bin/trace_run`` as a program: a mixed trace in 32-bit, its files and its "done" lines."""
+    name = "mixed_a"
+    reqs = requests_of(name, [40, 3, 90, 17, 66], seed=7)
+    steps = ru.trace_mixed(reqs, 256, seed=1, max_live=3)
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    out = tmp_path / "out"
+    proc = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", folders[name], "--dtype", "float32",
+                           "--out", str(out), "--max-tokens", "256", "--page-size", str(sc.PAGE_SIZE[name])],
+                          input="\n".join(json.dumps(s) for s in steps) + "\n", capture_output=True, text=True, timeout=900)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    assert [l for l in proc.stdout.splitlines() if l.startswith("done ")] == [f"done {s['step']}" for s in steps]
+    pos, vocab = {}, sc.CONFIGS[name]["vocab"]
+    for rec in steps:
+        wanted = sum(len(e["want"]) for e in rec["entries"])
+        rows = None
+        if wanted:
+            rows = torch.from_file(str(out / f"{rec['step']}.f32"), size=wanted * vocab, dtype=torch.float32).view(wanted, vocab)
+        r = 0
+        for e in rec["entries"]:
+            base = pos.get(e["id"], 0)
+            for wpos in e["want"]:
+                if plains[name].margin(reqs[e["id"]], base + wpos) > MARGIN[torch.float32]:
+                    assert row_error(rows[r], plains[name].of(reqs[e["id"]])[base + wpos]) <= LIMIT[torch.float32]
+                r += 1
+            pos[e["id"]] = base + len(e["tokens"])
+
+
+def test_command_line_serves_the_design(folders, tmp_path):
+    """The serving program on a Samulorn folder: requests of random lengths arriving over time, sampling, a pool that is used again; and
+    once more on random weights drawn from a configuration file."""
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    out = tmp_path / "m.json"
+    common = ["--num-requests", "12", "--max-batch", "4", "--max-gen", "10", "--prompt-len-dist", "lognormal:30,0.7,2,90",
+              "--output-len-dist", "lognormal:6,0.5,1,10", "--request-rate", "300", "--temperature", "0.8", "--top-p", "0.9",
+              "--ignore-eos", "--kv-block-size", "8", "--num-kv-blocks", "60", "--max-num-batched-tokens", "40",
+              "--max-model-len", "128", "--output-json", str(out)]
+    cfg_file = tmp_path / "config.json"
+    cfg_file.write_text(json.dumps(sc.MIXED_A))
+    for source in (["--checkpoint", folders["mixed_a"]], ["--model-config", str(cfg_file)]):
+        proc = subprocess.run([sys.executable, os.path.join(root, "bin", "offline_batch_benchmark"), *source, *common],
+                              capture_output=True, text=True, timeout=600)
+        assert proc.returncode == 0, proc.stderr[-3000:]
+        m = json.loads(out.read_text())[0]
+        assert m["completed"] == 12 and m["rejected"] == 0 and m["output_tokens"] > 12 and m["output_tps"] > 0
