@@ -28,19 +28,22 @@ struct LruArgs {
 };
 
 struct LruRow { float a, b; };
-__device__ __forceinline__ float lru_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float lru_gelu(float v) { return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v))); }
+__device__ __forceinline__ float lru_sigmoid(float x) { return __fdividef(1.f, 1.f + expf(-x)); }      // (1 + e^-x beyond 2^126: 0)
+// gelu_tanh: 0.5 v (1 + tanh(w)) = v sigmoid(2 w)
+__device__ __forceinline__ float lru_gelu(float v) { return v * lru_sigmoid(1.5957691216057308f * (v + 0.044715f * v * v * v)); }
 
 __device__ __forceinline__ LruRow lru_row(float zr, float zi, float u, float sp) {
-  const float la = -sp * lru_sigmoid(zr);
+  const float e = expm1f(-sp * lru_sigmoid(zr));          // a - 1, so that 1 - a^2 = -e (2 + e) keeps its digits near a = 1
+  float root;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(root) : "f"(-e * (2.f + e)));
   LruRow o;
-  o.a = expf(la);
-  o.b = sqrtf(-expm1f(2.f * la)) * lru_sigmoid(zi) * u;
+  o.a = 1.f + e;
+  o.b = root * lru_sigmoid(zi) * u;
   return o;
 }
 
 template <typename T>
-__global__ void __launch_bounds__(LRU_CH * LRU_SEG) lru_portion_kernel(const LruArgs p) {
+__global__ void __launch_bounds__(LRU_CH * LRU_SEG, 1) lru_portion_kernel(const LruArgs p) {
   __shared__ float2 fold[LRU_SEG][LRU_CH];
   __shared__ float last[LRU_CH];
   pdl_prologue();
@@ -54,11 +57,13 @@ __global__ void __launch_bounds__(LRU_CH * LRU_SEG) lru_portion_kernel(const Lru
   float S0 = on && pos0 > 0 ? *slot : 0.f;               // the state before the round
   const float br = p.br[cc], bi = p.bi[cc], sp = p.sp[cc], by = p.by ? p.by[cc] : 0.f;
   const float* z = p.z + blk * p.z_block + j;
-  for (int c0 = 0; c0 < n; c0 += LRU_SEG * LRU_RP) {
-    float a[LRU_RP], b[LRU_RP], y[LRU_RP], zr[LRU_RP], zi[LRU_RP], u[LRU_RP];
+  const int mine = seg * LRU_RP;                         // the segment's first row in a round
+  float zr[LRU_RP], zi[LRU_RP], u[LRU_RP], y[LRU_RP];
+  auto load = [&](int c0) {
 #pragma unroll
     for (int r = 0; r < LRU_RP; ++r) {
-      const int t = c0 + seg * LRU_RP + r;
+      const int t = c0 + mine + r;
+      zr[r] = zi[r] = u[r] = y[r] = 0.f;
       if (t < n) {
         const size_t row = (size_t)(row0 + t);
         zr[r] = z[row * 2 * p.bs];
@@ -67,26 +72,32 @@ __global__ void __launch_bounds__(LRU_CH * LRU_SEG) lru_portion_kernel(const Lru
         y[r] = to_f32<T>(((const T*)p.y)[row * p.y_stride + cc]);
       }
     }
+  };
+  load(0);
+  for (int c0 = 0; c0 < n; c0 += LRU_SEG * LRU_RP) {
+    float a[LRU_RP], b[LRU_RP], yg[LRU_RP];
     float A = 1.f, B = 0.f;
 #pragma unroll
     for (int r = 0; r < LRU_RP; ++r) {
-      a[r] = 1.f; b[r] = 0.f;                            // rows behind the portion leave the state as it is
-      if (c0 + seg * LRU_RP + r < n) {
-        const LruRow o = lru_row(zr[r] + br, zi[r] + bi, u[r], sp);
-        a[r] = o.a; b[r] = o.b;
-        A *= o.a;
-        B = fmaf(o.a, B, o.b);
-      }
+      const LruRow o = lru_row(zr[r] + br, zi[r] + bi, u[r], sp);
+      const bool have = c0 + mine + r < n;               // rows behind the portion leave the state as it is
+      a[r] = have ? o.a : 1.f;
+      b[r] = have ? o.b : 0.f;
+      A *= a[r];
+      B = fmaf(a[r], B, b[r]);
+      yg[r] = y[r];
     }
+    if (c0 + LRU_SEG * LRU_RP < n) load(c0 + LRU_SEG * LRU_RP);      // the next round's rows are on their way meanwhile
     fold[seg][ch] = make_float2(A, B);
     __syncthreads();
     float S = S0;
+#pragma unroll 4
     for (int k = 0; k < seg; ++k) { const float2 f = fold[k][ch]; S = fmaf(f.x, S, f.y); }
 #pragma unroll
     for (int r = 0; r < LRU_RP; ++r) {
-      const int t = c0 + seg * LRU_RP + r;
+      const int t = c0 + mine + r;
       S = fmaf(a[r], S, b[r]);
-      if (on && t < n) ((T*)p.out)[(size_t)(row0 + t) * p.out_stride + c] = from_f32<T>(p.scale * S * lru_gelu(y[r] + by));
+      if (on && t < n) ((T*)p.out)[(size_t)(row0 + t) * p.out_stride + c] = from_f32<T>(p.scale * S * lru_gelu(yg[r] + by));
     }
     if (seg == LRU_SEG - 1) last[ch] = S;
     __syncthreads();                                     // everyone has read the pairs, and the round's last state is there

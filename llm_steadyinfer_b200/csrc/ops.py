@@ -1627,6 +1627,62 @@ def channel_delta_scan(xc, dec, bg, state, y, q_start, ctx_len, slots, num_seqs:
              _ptr(ctx_len), _ptr(slots), int(num_seqs), G, H, dk, dv, _stream()), f"channel_delta_scan(heads={H}, dk={dk}, dv={dv})")
 
 
+GROUP_SCALARS = 8                 # numbers a token and head that ``channel_delta_groups`` leaves beside its rows
+
+_groups_ok_memo: dict = {}
+
+
+def channel_delta_groups_ok(dk: int, dv: int) -> bool:
+    """True when the form by groups of four tokens takes heads of ``dk`` x ``dv``."""
+    ok = _groups_ok_memo.get((dk, dv))
+    if ok is None:
+        lib = build.load("delta_rule")
+        lib.si_channel_delta_groups_ok.restype = _c_int
+        ok = _groups_ok_memo[(dk, dv)] = bool(lib.si_channel_delta_groups_ok(_c_int(dk), _c_int(dv)))
+    return ok
+
+
+def channel_delta_groups(xc, ba, b_off: int, dec, a_log, dt_bias, rec, sc, row_seq, q_start, num_seqs: int, G: int, H: int, dk: int) -> None:
+    """``channel_delta_prepare`` for the recurrence in groups of four tokens (counted from each sequence's first row of the step). ``rec``
+    fp32 [T, H, 3, dk] receives, with c the product of the group's decays up to the token and s that of those behind it, c k, c q and s k;
+    ``sc`` fp32 [T, H, 8] beta and the token's inner products with the group's earlier tokens (k with k: 3, q with k, its own included: 4);
+    ``dec`` fp32 [T, H*dk] holds the raw decay values and, in the rows that start a group, receives the product of all its decays."""
+    _cuda(xc, ba, dec, a_log, dt_bias, rec, sc, row_seq, q_start)
+    _i32(row_seq, "row_seq"); _i32(q_start, "q_start")
+    T = xc.shape[0]
+    _need(xc.dtype == torch.float32 and xc.stride(1) == 1 and xc.shape[1] >= 2 * G * dk, "channel_delta_groups: xc must be fp32 rows")
+    _need(ba.shape[0] == T and ba.stride(1) == 1 and ba.shape[1] >= b_off + H, "channel_delta_groups: ba rows")
+    _need(dec.dtype == torch.float32 and dec.shape == (T, H * dk) and dec.stride(1) == 1, "channel_delta_groups: dec must be fp32 [T, H*dk]")
+    _f32v(rec, "rec", T * H * 3 * dk); _f32v(sc, "sc", T * H * GROUP_SCALARS)
+    _f32v(a_log, "a_log", H); _f32v(dt_bias, "dt_bias", H * dk)
+    f = _fn("delta_rule", "si_channel_delta_groups",
+            [_c_p, _c_ll, _c_p, _c_int, _c_ll, _c_int, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int,
+             _c_int, _c_p])
+    _check(f(_ptr(xc), xc.stride(0), _ptr(ba), _dt(ba), ba.stride(0), int(b_off), _ptr(dec), dec.stride(0), _ptr(a_log), _ptr(dt_bias),
+             _ptr(rec), _ptr(sc), _ptr(row_seq), _ptr(q_start), T, int(num_seqs), G, H, dk, _stream()), f"channel_delta_groups(heads={H}, dk={dk})")
+
+
+def channel_delta_group_scan(rec, sc, dec, xc, state, y, q_start, ctx_len, slots, num_seqs: int, G: int, H: int, dk: int, dv: int) -> None:
+    """``channel_delta_scan`` in groups of four tokens, from what ``channel_delta_groups`` leaves (``rec``, ``sc``, ``dec``) and the values in
+    ``xc`` (fp32 rows [q | k | v]); the same state, the same result up to the order of its sums."""
+    _cuda(rec, sc, dec, xc, state, y, q_start, ctx_len, slots)
+    for t, nm in ((q_start, "q_start"), (ctx_len, "ctx_len"), (slots, "slots")):
+        _i32(t, nm)
+    T = xc.shape[0]
+    _need(xc.dtype == torch.float32 and xc.stride(1) == 1 and xc.shape[1] >= 2 * G * dk + H * dv, "channel_delta_group_scan: xc must be fp32 [T, 2*G*dk + H*dv]")
+    _need(dec.dtype == torch.float32 and dec.shape == (T, H * dk) and dec.stride(1) == 1, "channel_delta_group_scan: dec must be fp32 [T, H*dk]")
+    _f32v(rec, "rec", T * H * 3 * dk); _f32v(sc, "sc", T * H * GROUP_SCALARS)
+    _need(y.dtype == torch.float32 and y.shape == (T, H * dv) and y.stride(1) == 1, "channel_delta_group_scan: y must be fp32 [T, H*dv]")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
+          and state.shape[1] >= H * delta_state_floats(dk, dv),
+          "channel_delta_group_scan: state must be fp32 [slots, >= H * delta_state_floats(dk, dv)]")
+    f = _fn("delta_rule", "si_channel_delta_group_scan",
+            [_c_p, _c_p, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_ll, _c_p, _c_p, _c_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_p])
+    _check(f(_ptr(rec), _ptr(sc), _ptr(dec), dec.stride(0), _ptr(xc), xc.stride(0), _ptr(state), state.stride(0), _ptr(y), y.stride(0),
+             _ptr(q_start), _ptr(ctx_len), _ptr(slots), int(num_seqs), G, H, dk, dv, _stream()),
+           f"channel_delta_group_scan(heads={H}, dk={dk}, dv={dv})")
+
+
 def gated_linear(u, z, bias_r, bias_i, rate, y, y_bias, state, out, q_start, ctx_len, slots, num_seqs: int, scale: float = 1.0,
                  kinds: int = 3) -> None:
     """The real-gated linear recurrence per channel, all fp32: r = sigmoid(zr + bias_r), i = sigmoid(zi + bias_i), a = exp(-rate * r),

@@ -37,7 +37,7 @@ KINDS = {
     "moe_route": "moe_route", "moe_plan": "moe_plan", "moe_gather": "moe_gather", "moe_gemm_tc05": "moe_gemm_tc05",
     "moe_gemm_tiles": "moe_gemm_tiles", "moe_combine": "moe_combine", "gated_add": "gated_add", "gemm_skinny_batched": "gemm_skinny_batched",
     "stream_norm": "stream_norm", "qkv_conv": "qkv_conv", "conv_rows": "conv_rows", "stream_add": "stream_add",
-    "channel_delta_prepare": "channel_delta_prepare", "channel_delta_scan": "channel_delta_scan", "gated_linear": "gated_linear",
+    "channel_delta_prepare": "channel_delta_prepare", "channel_delta_scan": "channel_delta_scan", "channel_delta_groups": "channel_delta_groups", "channel_delta_group_scan": "channel_delta_group_scan", "gated_linear": "gated_linear",
     "token_gate": "token_gate", "gemm_skinny_token_gate": "gemm_skinny_token_gate",
     "glu_limited": "glu_limited", "gemm_skinny_glu_limited": "gemm_skinny_glu_limited", "gemm_tc05_glu_limited": "gemm_tc05_glu_limited",
 }

@@ -55,6 +55,7 @@ import torch
 from ..csrc import ops
 from .base import CacheNeed, Mixer, StateNeed, first_visible_key, register_mixer
 from . import flex_plan
+from .step_rows import portions
 from . import linear as linear_mod
 from .linear import linear
 
@@ -515,19 +516,6 @@ class Attention(Mixer):
         if plan["por"] is not None:
             portion = ops.attn_portion_tc05 if plan["tc05"] else ops.attn_portion
             portion(q, cache.k, cache.v, cache.block_table, plan["por"], out, *args, status=ctx.status, **extra)
-
-
-def portions(ctx) -> int:
-    """What the step holds beside sequences of one row, as ``ops.qkv_conv`` and ``ops.conv_rows`` take it: 1 portions from position 0,
-    2 portions that go on, 3 both, 0 neither."""
-    if ctx.seq_cap is not None:                          # fixed shapes hold single rows
-        return 0
-    got = ctx.plans.get("portions")
-    if got is None:
-        n = np.diff(ctx.h_q_start)
-        fresh = np.asarray(ctx.h_ctx_len) == n
-        got = ctx.plans["portions"] = (1 if (fresh & (n > 1)).any() else 0) | (2 if (~fresh & (n > 1)).any() else 0)
-    return got
 
 
 def distance_bucket(n: int, rows: int, max_distance: float) -> int:

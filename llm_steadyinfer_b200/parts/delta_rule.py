@@ -23,7 +23,8 @@ With a decay per head and key channel (``channel_delta``), decay and read-out ga
     g = exp(-exp(A_log_h) * softplus(W_a2 (W_a1 x) + dt_bias)) [H, dk];   S <- diag(g_h) S, then as above
     o <- norm_w * o * rsqrt(mean(o^2) + eps) * sigmoid(W_g2 (W_g1 x))_h
 The convolutions, their silu and the unit norms are one launch behind the stacked projection (``conv_rows``); the second low-rank
-product of the decays leaves fp32.
+product of the decays leaves fp32. In steps with portions of several rows the recurrence runs in groups of four tokens where the
+sizes allow (``channel_delta_group_scan``), else token by token.
 Tensor names: q, k, v, q.conv, k.conv, v.conv, b, A_log, a1, a2, dt_bias, g1, g2, norm, o.
 """
 from __future__ import annotations
@@ -31,9 +32,9 @@ from __future__ import annotations
 import torch
 
 from ..csrc import ops
-from .attention import portions
 from .base import Mixer, StateNeed, register_mixer
 from .linear import linear
+from .step_rows import portions, row_kinds
 
 
 class GatedDeltaRule(Mixer):
@@ -118,6 +119,9 @@ class GatedDeltaRule(Mixer):
 
 
 register_mixer("gated_delta", GatedDeltaRule)
+
+
+USE_GROUPS = True        # portions: four tokens at a time where the sizes allow; False: token by token
 
 
 class ChannelDeltaRule(Mixer):
@@ -205,10 +209,16 @@ class ChannelDeltaRule(Mixer):
                       portions=portions(ctx), status=ctx.status)
         dec = ctx.buf("delta_decay", (T, self.nd), torch.float32)
         linear(u[:, self.a_cols[0]:self.a_cols[1]], self.w_a2, dec, ctx.status)
-        bg = ctx.buf("delta_bg", (T, H + G), torch.float32)
-        ops.channel_delta_prepare(xc, u, self.b_off, dec, self.a_log, self.dt_bias, bg, G, H, dk)
         y = ctx.buf("delta_y", (T, self.nv), torch.float32)
-        ops.channel_delta_scan(xc, dec, bg, state, y, ctx.q_start, ctx.ctx_len, ctx.slots, ctx.seq_slots, G, H, dk, dv)
+        if row_kinds(ctx) & 2 and USE_GROUPS and ops.channel_delta_groups_ok(dk, dv):
+            rec = ctx.buf("delta_groups", (T, H, 3, dk), torch.float32)
+            sc = ctx.buf("delta_scalars", (T, H, ops.GROUP_SCALARS), torch.float32)
+            ops.channel_delta_groups(xc, u, self.b_off, dec, self.a_log, self.dt_bias, rec, sc, ctx.row_seq, ctx.q_start, ctx.seq_slots, G, H, dk)
+            ops.channel_delta_group_scan(rec, sc, dec, xc, state, y, ctx.q_start, ctx.ctx_len, ctx.slots, ctx.seq_slots, G, H, dk, dv)
+        else:
+            bg = ctx.buf("delta_bg", (T, H + G), torch.float32)
+            ops.channel_delta_prepare(xc, u, self.b_off, dec, self.a_log, self.dt_bias, bg, G, H, dk)
+            ops.channel_delta_scan(xc, dec, bg, state, y, ctx.q_start, ctx.ctx_len, ctx.slots, ctx.seq_slots, G, H, dk, dv)
         gate = ctx.buf("delta_gate", (T, self.nv), self.dtype)
         linear(u[:, self.g_cols[0]:self.g_cols[1]], self.w_g2, gate, ctx.status)
         gated = ctx.buf("delta_gated", (T, self.nv), self.dtype)

@@ -19,10 +19,10 @@ import numpy as np
 import torch
 
 from ..csrc import ops
-from .attention import portions
 from .base import Mixer, StateNeed, register_mixer
 from .linear import linear
 from . import linear as linear_mod
+from .step_rows import portions, row_kinds
 
 DECAY_RATE = 8.0
 
@@ -122,17 +122,6 @@ class GatedRecurrence(Mixer):
         out = ctx.buf("delta", (T, self.hidden), self.dtype)
         linear(heads, self.output_weight, out, ctx.status)
         return out
-
-
-def row_kinds(ctx) -> int:
-    """What the step holds: 1 sequences of one row, 2 longer portions, 3 both."""
-    if ctx.seq_cap is not None:                          # fixed shapes hold single rows
-        return 1
-    got = ctx.plans.get("row_kinds")
-    if got is None:
-        n = np.diff(ctx.h_q_start)
-        got = ctx.plans["row_kinds"] = (1 if (n == 1).any() else 0) | (2 if (n > 1).any() else 0)
-    return got
 
 
 register_mixer("gated_recurrence", GatedRecurrence)

@@ -458,10 +458,15 @@ def test_rotation_between_convolution_and_norm(NQ, NK, NV, dk, dv, K, dims, time
 
 
 @pytest.mark.parametrize("H,G,dk,dv", [(4, 2, 24, 16), (3, 3, 64, 128), (2, 1, 5, 9), (8, 2, 128, 64), (2, 2, 160, 24), (16, 8, 128, 128), (1, 1, 512, 40),
-                                       (2, 2, 4, 4), (2, 1, 200, 36)])
-def test_channel_delta_kernels_in_portions(H, G, dk, dv):
-    """Preparation, recurrence and the read-out's norm with its sigmoid gate over three sequences in unequal portions."""
+                                       (2, 2, 4, 4), (2, 1, 200, 36), (9, 3, 64, 64), (2, 1, 96, 20)])
+@pytest.mark.parametrize("groups", [False, True], ids=["token_by_token", "by_groups"])
+def test_channel_delta_kernels_in_portions(H, G, dk, dv, groups):
+    """Preparation, recurrence and the read-out's norm with its sigmoid gate over three sequences in unequal portions, token by token and
+    in groups of four tokens (portions of 1 to 30 rows end at every place of a group)."""
     from llm_steadyinfer_b200.csrc import ops
+    if groups and not ops.channel_delta_groups_ok(dk, dv):
+        assert dk % 4 or dv % 4 or dk <= 32 or dk > 256
+        return
     torch.manual_seed(H * 100 + dk)
     C = 2 * G * dk + H * dv
     raw = [torch.randn(n, H * dk) for n in LENS]
@@ -486,8 +491,14 @@ def test_channel_delta_kernels_in_portions(H, G, dk, dv):
         xc, dec, rows = cat(x), cat(raw), cat(ba)
         R = xc.shape[0]
         bg, y = torch.zeros(R, H + G, device=DEV), torch.zeros(R, H * dv, device=DEV)
-        ops.channel_delta_prepare(xc, rows, 3, dec, a_log.to(DEV), dt_bias.to(DEV), bg, G, H, dk)
-        ops.channel_delta_scan(xc, dec, bg, state, y, starts, ctx, slots, len(live), G, H, dk, dv)
+        if groups:
+            seq = i32(*[i for i, (_, _, m) in enumerate(live) for _ in range(m)])
+            rec, sc_ = torch.full((R, H, 3, dk), 9.0, device=DEV), torch.full((R, H, ops.GROUP_SCALARS), 9.0, device=DEV)
+            ops.channel_delta_groups(xc, rows, 3, dec, a_log.to(DEV), dt_bias.to(DEV), rec, sc_, seq, starts, len(live), G, H, dk)
+            ops.channel_delta_group_scan(rec, sc_, dec, xc, state, y, starts, ctx, slots, len(live), G, H, dk, dv)
+        else:
+            ops.channel_delta_prepare(xc, rows, 3, dec, a_log.to(DEV), dt_bias.to(DEV), bg, G, H, dk)
+            ops.channel_delta_scan(xc, dec, bg, state, y, starts, ctx, slots, len(live), G, H, dk, dv)
         out = torch.zeros(R, H * dv, device=DEV)
         ops.head_norm_gate(y, cat(z), norm_w.to(DEV), out, H, dv, 1e-5, gate="sigmoid")
         r = 0
