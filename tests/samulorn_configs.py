@@ -219,6 +219,7 @@ def _tensors(cfg, seed):
             D = side["dim"]
             lin(p + "side.gate", D, W); lin(p + "side.proj", W, D); vec(p + "side.norm", W, 0.5, 0.2)
     norm("final.norm", 0.5)
+    vec("final.norm", W, 0.0, 1.0)                       # of both signs: the head is the embedding, and a token must not simply echo itself
     return out
 
 
